@@ -10,11 +10,13 @@
 //   second plane of the same pages at the place of position b.  Tokens and blocks share one softmax.
 //   score:  s = scale * q . k;   `softcap` = c > 0:  s <- c tanh(s / c);   `r1`, `r2` [H]:  s <- s - r1_h ln(1 + r2_h (p - j))
 //   (tokens only);  `sink` [H]: the softmax's denominator also holds exp(sink_h), a term without key or value;
-//   `gate` [T, H]: the head's output is multiplied by sigmoid(gate[t, h]).
+//   `gate` [T, H]: the head's output is multiplied by sigmoid(gate[t, h]), or, with one column per element ([T, H dv]), every
+//   element by its own;  `out_scale`: and by this constant.  Rows of the output may lie inside wider rows (`out_stride`).
 //
 //   Pages are [plane][kv head][slot][dk + dv] with 1 plane, or 2 when blocks are pooled (plane 1: the blocks' means).
 //
-//   masked_qkv_prep : from the packed projection row [q: H dk | k: G dk | v: G dv]: per-head RMS norm of q and k (one weight
+//   masked_qkv_prep : from the packed projection row [q: H dk | k: G dk | v: G dv], plus an optional bias of the same layout:
+//                     per-head RMS norm of q and k (one weight
 //                     vector for all heads, float arithmetic, one rounding), rotation of the first `rot` elements in pairs
 //                     (2i, 2i + 1) or (i, i + rot / 2), the value mixed with the same token's value of an earlier layer
 //                     (v <- (1 - lam) v + lam v_first), the entry's write, and the queries' write.  One warp per head.
@@ -43,13 +45,16 @@ __device__ __forceinline__ float2 load2(const __nv_bfloat16* p) { return __bfloa
 __device__ __forceinline__ void store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ void store2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
 
+// two floats of a vector that may start anywhere
+__device__ __forceinline__ float2 load2f(const float* p) { return make_float2(p[0], p[1]); }
+
 constexpr int kPrepPairs = 8;                            // pairs per lane: heads of up to 512 elements
 
 // The same epilogue two elements at a time, for even sizes and a rotation in pairs (2i, 2i + 1) (or none): a lane holds whole
 // pairs in registers from the load to the store, so neither shared memory nor a second pass is needed.
 template <typename T>
 __global__ void __launch_bounds__(kPrepWarps * 32)
-masked_qkv_prep_pairs_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int stride, const float* __restrict__ q_w,
+masked_qkv_prep_pairs_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int stride, const float* __restrict__ bias, const float* __restrict__ q_w,
                              const float* __restrict__ k_w, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                              const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ pages,
                              T* __restrict__ vfirst_out, const T* __restrict__ vfirst_in, const float* __restrict__ lam_p,
@@ -79,6 +84,7 @@ masked_qkv_prep_pairs_kernel(T* __restrict__ q_out, const T* __restrict__ packed
         const float lam = (vfirst_in != nullptr && lam_p != nullptr) ? lam_p[0] : 0.f;
         for (int e = lane * 2; e < dv; e += 64) {
             float2 v = load2(src + e);
+            if (bias != nullptr) { const float2 b = load2f(bias + H * dk + G * dk + g * dv + e); v.x += b.x; v.y += b.y; }
             if (vfirst_out != nullptr) store2(vfirst_out + t * G * dv + g * dv + e, v);
             if (vfirst_in != nullptr) {
                 const float2 f = load2(vfirst_in + t * G * dv + g * dv + e);
@@ -99,7 +105,12 @@ masked_qkv_prep_pairs_kernel(T* __restrict__ q_out, const T* __restrict__ packed
 #pragma unroll
     for (int k = 0; k < kPrepPairs; ++k) {
         const int i = lane + 32 * k;
-        if (i < np) { x[k] = load2(src + 2 * i); ss = fmaf(x[k].x, x[k].x, ss); ss = fmaf(x[k].y, x[k].y, ss); }
+        if (i < np) {
+            x[k] = load2(src + 2 * i);
+            if (bias != nullptr) { const float2 b = load2f(bias + task * dk + 2 * i); x[k].x += b.x; x[k].y += b.y; }   // key heads lie behind the query heads
+            ss = fmaf(x[k].x, x[k].x, ss);
+            ss = fmaf(x[k].y, x[k].y, ss);
+        }
     }
     if (w != nullptr) {
         ss = warp_sum(ss);
@@ -165,7 +176,7 @@ template <> struct Chunk16<__nv_bfloat16> {
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int stride, const float* __restrict__ q_w,
+masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int stride, const float* __restrict__ bias, const float* __restrict__ q_w,
                            const float* __restrict__ k_w, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                            const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ pages,
                            T* __restrict__ vfirst_out, const T* __restrict__ vfirst_in, const float* __restrict__ lam_p,
@@ -195,6 +206,10 @@ masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, 
         if (vi >= G * chv) return;
         const int g = vi / chv, e = (vi - g * chv) * N;
         Chunk16<T>::load(v, row + H * dk + G * dk + g * dv + e);
+        if (bias != nullptr) {
+#pragma unroll
+            for (int i = 0; i < N; ++i) v[i] += bias[H * dk + G * dk + g * dv + e + i];
+        }
         if (vfirst_out != nullptr) Chunk16<T>::store(vfirst_out + t * G * dv + g * dv + e, v);
         if (vfirst_in != nullptr) {
             const float lam = lam_p[0];
@@ -214,6 +229,10 @@ masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, 
     float ss = 0.f;
     if (live) {
         Chunk16<T>::load(v, row + task * dk + c * N);   // key heads lie behind the query heads in the row
+        if (bias != nullptr) {
+#pragma unroll
+            for (int i = 0; i < N; ++i) v[i] += bias[task * dk + c * N + i];
+        }
 #pragma unroll
         for (int i = 0; i < N; ++i) ss = fmaf(v[i], v[i], ss);
     }
@@ -251,7 +270,7 @@ masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, 
 
 template <typename T>
 __global__ void __launch_bounds__(kPrepWarps * 32)
-masked_qkv_prep_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int stride, const float* __restrict__ q_w,
+masked_qkv_prep_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int stride, const float* __restrict__ bias, const float* __restrict__ q_w,
                        const float* __restrict__ k_w, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                        const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ pages,
                        T* __restrict__ vfirst_out, const T* __restrict__ vfirst_in, const float* __restrict__ lam_p,
@@ -282,7 +301,8 @@ masked_qkv_prep_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int 
         const float lam = (vfirst_in != nullptr && lam_p != nullptr) ? lam_p[0] : 0.f;
         for (int e = lane; e < dv; e += 32) {
             float v = to_float(src[e]);
-            if (vfirst_out != nullptr) vfirst_out[t * G * dv + g * dv + e] = src[e];
+            if (bias != nullptr) v += bias[H * dk + G * dk + g * dv + e];
+            if (vfirst_out != nullptr) vfirst_out[t * G * dv + g * dv + e] = from_float<T>(v);
             if (vfirst_in != nullptr) v = (1.f - lam) * v + lam * to_float(vfirst_in[t * G * dv + g * dv + e]);
             if (entry >= 0) pages[entry + static_cast<int64_t>(g) * page_size * ew + dk + e] = from_float<T>(v);
         }
@@ -294,7 +314,12 @@ masked_qkv_prep_kernel(T* __restrict__ q_out, const T* __restrict__ packed, int 
     const float* w = is_q ? q_w : k_w;
     float* buf = smem + warp * dk;
     float ss = 0.f;
-    for (int e = lane; e < dk; e += 32) { const float x = to_float(src[e]); buf[e] = x; ss = fmaf(x, x, ss); }
+    for (int e = lane; e < dk; e += 32) {
+        float x = to_float(src[e]);
+        if (bias != nullptr) x += bias[task * dk + e];
+        buf[e] = x;
+        ss = fmaf(x, x, ss);
+    }
     if (w != nullptr) {
         ss = warp_sum(ss);
         const float inv = rsqrtf(ss / static_cast<float>(dk) + eps);
@@ -395,7 +420,8 @@ attn_masked_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T
                            const int* __restrict__ block_tables, int table_width, const int* __restrict__ seq_of_token,
                            const int* __restrict__ positions, int H, int G, int dk, int dv, int page_size, int planes,
                            MaskParams mp, const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
-                           const T* __restrict__ gate, int gate_stride, int num_pages, int* __restrict__ err) {
+                           const T* __restrict__ gate, int gate_stride, int gate_element, float out_scale, int out_stride, int num_pages,
+                           int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ int64_t smem64[];
@@ -465,11 +491,15 @@ attn_masked_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T
         }
     }
     float inv_l = l > 0.f ? 1.f / l : 0.f;
-    if (gate != nullptr) inv_l *= 1.f / (1.f + expf(-to_float(gate[t * gate_stride + h])));
+    inv_l *= out_scale;
+    if (gate != nullptr && !gate_element) inv_l *= 1.f / (1.f + expf(-to_float(gate[t * gate_stride + h])));
 #pragma unroll
     for (int i = 0; i < kMaskedDimsPerThread; ++i) {
         const int d = tid + i * kMaskedThreads;
-        if (d < dv) out[(t * H + h) * dv + d] = from_float<T>(acc[i] * inv_l);
+        if (d >= dv) continue;
+        float v = acc[i] * inv_l;
+        if (gate != nullptr && gate_element) v *= 1.f / (1.f + expf(-to_float(gate[t * gate_stride + h * dv + d])));
+        out[t * out_stride + h * dv + d] = from_float<T>(v);
     }
 }
 
@@ -481,17 +511,19 @@ constexpr int kMThreads = 128;
 constexpr float kLog2eM = 1.4426950408889634f;
 
 struct MaskedAttnParams {
-    __nv_bfloat16* out;                 // [T, H * dv]
+    __nv_bfloat16* out;                 // [T, H * dv] inside rows of out_stride
     const __nv_bfloat16* q;             // [T, H * dk]
     const __nv_bfloat16* pages;         // [num_pages, planes, G, page_size, dk + dv]
-    const __nv_bfloat16* gate;          // [T, gate_stride] or null
+    const __nv_bfloat16* gate;          // [T, gate_stride] or null: a column per head, or (gate_element) per element
     const float* r1;                    // [H] or null
     const float* r2;
     const float* sink;                  // [H] or null
     const int* block_tables;            // [S, table_width]
     const int* cu_seqlens;              // [S + 1]
     const int* positions;               // [T]
-    int gate_stride, table_width, S, H, G, dk, dv, page_size, page_shift, num_pages, planes;
+    int gate_stride, gate_element, out_stride;
+    float out_scale;
+    int table_width, S, H, G, dk, dv, page_size, page_shift, num_pages, planes;
     MaskParams mp;
     // decode form only: the tiles of a (request, kv head) are shared out among `splits` blocks (gridDim.z); with more than
     // one, a block leaves its part (unnormalised rows, maxima, sums) in `parts` and a second kernel merges them
@@ -715,14 +747,20 @@ attn_masked_kernel(const MaskedAttnParams p) {
         const int tok = r / g;
         if (tok >= n_tok) continue;
         const int head = kvh * g + r % g;
-        float inv = l[half] > 0.f ? 1.f / l[half] : 0.f;
-        if (p.gate != nullptr)
+        float inv = l[half] > 0.f ? p.out_scale / l[half] : 0.f;
+        if (p.gate != nullptr && !p.gate_element)
             inv *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<int64_t>(cu0 + q0 + tok) * p.gate_stride + head])));
-        __nv_bfloat16* dst = p.out + (static_cast<int64_t>(cu0 + q0 + tok) * p.H + head) * dv;
+        __nv_bfloat16* dst = p.out + static_cast<int64_t>(cu0 + q0 + tok) * p.out_stride + head * dv;
+        const __nv_bfloat16* eg = p.gate != nullptr && p.gate_element ? p.gate + static_cast<int64_t>(cu0 + q0 + tok) * p.gate_stride + head * dv : nullptr;
 #pragma unroll
         for (int dt = 0; dt < W / 8; ++dt) {
             const int d = dt * 8 + ((lane & 3) << 1);
             if (!EXACT && d >= dv) break;
+            if (eg != nullptr) {
+                const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(eg + d));
+                o[dt][half * 2] *= __fdividef(1.f, 1.f + __expf(-z.x));
+                o[dt][half * 2 + 1] *= __fdividef(1.f, 1.f + __expf(-z.y));
+            }
             *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(o[dt][half * 2] * inv, o[dt][half * 2 + 1] * inv);
         }
     }
@@ -760,9 +798,10 @@ __device__ __forceinline__ void masked_finish(const MaskedAttnParams& p, int t, 
         ll = ll * f + ex2(sk - top);
         acc *= f;
     }
-    float v = ll > 0.f ? acc / ll : 0.f;
-    if (p.gate != nullptr) v *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<int64_t>(t) * p.gate_stride + head])));
-    p.out[(static_cast<int64_t>(t) * p.H + head) * dv + d] = __float2bfloat16_rn(v);
+    float v = ll > 0.f ? acc / ll * p.out_scale : 0.f;
+    if (p.gate != nullptr)
+        v *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<int64_t>(t) * p.gate_stride + (p.gate_element ? head * dv + d : head)])));
+    p.out[static_cast<int64_t>(t) * p.out_stride + head * dv + d] = __float2bfloat16_rn(v);
 }
 
 template <int W, bool EXACT>
@@ -1054,7 +1093,7 @@ int launch_attn_masked_decode(const MaskedAttnParams& p, cudaStream_t stream) {
 
 using namespace cvb;
 
-extern "C" int cvb_masked_qkv_prep(void* q_out, const void* packed, int T, int stride, const float* q_w, const float* k_w,
+extern "C" int cvb_masked_qkv_prep(void* q_out, const void* packed, int T, int stride, const float* bias, const float* q_w, const float* k_w,
                                    const float* cos_t, const float* sin_t, const int* positions, const int* slots, void* pages,
                                    void* vfirst_out, const void* vfirst_in, const float* lam, int H, int G, int dk, int dv, int rot,
                                    int interleaved, int planes, int page_size, int max_pos, float eps, int64_t total_slots, int dtype,
@@ -1082,15 +1121,15 @@ extern "C" int cvb_masked_qkv_prep(void* q_out, const void* packed, int T, int s
     const dim3 grid16(static_cast<unsigned>(T), vec16 ? static_cast<unsigned>((qk_pad + G * (dv / n16) + 127) / 128) : 1u);
 #define CALL(TY)                                                                                                          \
     if (vec16)                                                                                                            \
-    launch_kernel(masked_qkv_prep_vec_kernel<TY>, grid16, dim3(128), 0, stream, (TY*)q_out, (const TY*)packed, stride, q_w,           \
+    launch_kernel(masked_qkv_prep_vec_kernel<TY>, grid16, dim3(128), 0, stream, (TY*)q_out, (const TY*)packed, stride, bias, q_w,           \
                   k_w, cos_t, sin_t, positions, slots, (TY*)pages, (TY*)vfirst_out, (const TY*)vfirst_in, lam, H, G, dk, dv, rot,    \
                   planes, page_size, max_pos, eps, total_slots, qk_pad, err_flag);                                        \
     else if (pairs)                                                                                                       \
-    launch_kernel(masked_qkv_prep_pairs_kernel<TY>, grid, dim3(kPrepWarps * 32), 0, stream, (TY*)q_out, (const TY*)packed, stride, q_w, \
+    launch_kernel(masked_qkv_prep_pairs_kernel<TY>, grid, dim3(kPrepWarps * 32), 0, stream, (TY*)q_out, (const TY*)packed, stride, bias, q_w, \
                   k_w, cos_t, sin_t, positions, slots, (TY*)pages, (TY*)vfirst_out, (const TY*)vfirst_in, lam, H, G, dk, dv, rot,    \
                   planes, page_size, max_pos, eps, total_slots, err_flag);                                                \
     else                                                                                                                  \
-    launch_kernel(masked_qkv_prep_kernel<TY>, grid, dim3(kPrepWarps * 32), smem, stream, (TY*)q_out, (const TY*)packed, stride, q_w, \
+    launch_kernel(masked_qkv_prep_kernel<TY>, grid, dim3(kPrepWarps * 32), smem, stream, (TY*)q_out, (const TY*)packed, stride, bias, q_w, \
                   k_w, cos_t, sin_t, positions, slots, (TY*)pages, (TY*)vfirst_out, (const TY*)vfirst_in, lam, H, G, dk, dv, rot,    \
                   interleaved, planes, page_size, max_pos, eps, total_slots, err_flag)
     CVB_DISPATCH_DTYPE(dtype, CALL);
@@ -1115,20 +1154,21 @@ extern "C" int cvb_attn_masked_general(void* out, const void* q, const void* pag
                                        const int* seq_of_token, const int* positions, int T, int H, int G, int dk, int dv,
                                        int page_size, int planes, int chunk, int window, int pool, float scale, float softcap,
                                        const float* r1, const float* r2, const float* sink, const void* gate, int gate_stride,
-                                       int num_pages, int dtype, int* err_flag, cudaStream_t stream) {
+                                       int gate_element, float out_scale, int out_stride, int num_pages, int dtype, int* err_flag, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
     if (T < 0 || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || page_size <= 0 || table_width <= 0 || num_pages <= 0) return CVB_E_SIZE;
     if (dv > kMaskedThreads * kMaskedDimsPerThread || H > 65535) return CVB_E_SIZE;
     if (H % G || chunk < 0 || window < 0 || pool < 0 || (planes != 1 && planes != 2) || (pool > 0 && (planes != 2 || window <= 0)))
         return CVB_E_SHAPE;
-    if ((r1 == nullptr) != (r2 == nullptr)) return CVB_E_SHAPE;
+    if ((r1 == nullptr) != (r2 == nullptr) || out_stride < H * dv) return CVB_E_SHAPE;
+    if (gate != nullptr && gate_stride < (gate_element ? H * dv : H)) return CVB_E_SHAPE;
     MaskParams mp{chunk, window, pool, scale, softcap};
     const size_t smem = kMaskedThreads * sizeof(int64_t) + (static_cast<size_t>(dk) + kMaskedThreads + 32) * sizeof(float);
     if (smem > 48 * 1024) return CVB_E_SIZE;
 #define CALL(TY)                                                                                                          \
     launch_kernel(attn_masked_general_kernel<TY>, dim3(T, H), dim3(kMaskedThreads), smem, stream, (TY*)out, (const TY*)q,           \
                   (const TY*)pages, block_tables, table_width, seq_of_token, positions, H, G, dk, dv, page_size, planes, mp, r1, r2, \
-                  sink, (const TY*)gate, gate_stride, num_pages, err_flag)
+                  sink, (const TY*)gate, gate_stride, gate_element, out_scale, out_stride, num_pages, err_flag)
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
     return launch_status();
@@ -1144,20 +1184,24 @@ extern "C" int cvb_attn_masked_bf16(void* out, const void* q, const void* pages,
                                     const int* cu_seqlens, const int* positions, int S, int num_tiles, int H, int G, int dk, int dv,
                                     int page_size, int planes, int chunk, int window, int pool, float scale, float softcap,
                                     const float* r1, const float* r2, const float* sink, const void* gate, int gate_stride,
-                                    int num_pages, int all_single, int splits, float* parts, int64_t parts_floats, int* err_flag,
+                                    int gate_element, float out_scale, int out_stride, int num_pages, int all_single, int splits, float* parts, int64_t parts_floats, int* err_flag,
                                     cudaStream_t stream) {
     if (num_tiles == 0 || S == 0) return CVB_OK;
     if (S < 0 || num_tiles < 0 || page_size <= 0 || table_width <= 0 || num_pages <= 0) return CVB_E_SIZE;
     if (!cvb_attn_masked_supported(H, G, dk, dv)) return CVB_E_UNSUPPORTED;
     if (chunk < 0 || window < 0 || pool < 0 || (planes != 1 && planes != 2) || (pool > 0 && (planes != 2 || window <= 0))) return CVB_E_SHAPE;
     if ((r1 == nullptr) != (r2 == nullptr)) return CVB_E_SHAPE;
-    if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(pages) | reinterpret_cast<uintptr_t>(out)) & 15) return CVB_E_ALIGN;
+    if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(pages)) & 15) return CVB_E_ALIGN;
+    if (out_stride < H * dv || (gate != nullptr && gate_stride < (gate_element ? H * dv : H))) return CVB_E_SHAPE;
+    if ((reinterpret_cast<uintptr_t>(out) & 3) || (out_stride & 1)) return CVB_E_ALIGN;                  // stores of element pairs
+    if (gate != nullptr && gate_element && ((reinterpret_cast<uintptr_t>(gate) & 3) || (gate_stride & 1))) return CVB_E_ALIGN;
     if (G > 65535) return CVB_E_SIZE;
     MaskedAttnParams p;
     p.out = static_cast<__nv_bfloat16*>(out);
     p.q = static_cast<const __nv_bfloat16*>(q);
     p.pages = static_cast<const __nv_bfloat16*>(pages);
-    p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_stride = gate_stride;
+    p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_stride = gate_stride; p.gate_element = gate_element;
+    p.out_scale = out_scale; p.out_stride = out_stride;
     p.r1 = r1; p.r2 = r2; p.sink = sink;
     p.block_tables = block_tables; p.cu_seqlens = cu_seqlens; p.positions = positions;
     p.table_width = table_width; p.S = S; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.page_size = page_size;

@@ -43,6 +43,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "moe": ["moe.cu"],
     "latent": ["latent.cu"],
     "recurrent": ["recurrent.cu"],
+    "lru": ["lru.cu"],
     "sandwich": ["sandwich.cu"],
     "hyper": ["hyper.cu"],
     "attn_masked": ["attention_masked.cu"],

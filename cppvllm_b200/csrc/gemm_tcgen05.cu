@@ -35,7 +35,10 @@ constexpr int kBK = 64;                       // one 128-byte swizzle span of bf
 constexpr int kGemmThreads = 192;
 constexpr int kBoxBytes = 32 * 64 * 2;        // what a warp of the epilogue hands to one TMA store: 32 rows of 64 bf16
 
-enum GemmEpilogue { kPlain = 0, kSwiglu = 1, kAddResidual = 2, kRelu2 = 3 };   // kRelu2: C = relu(T(A B^T))^2
+// kRelu2: C = relu(T(A B^T))^2.  kSwiglu, kClamped and kGeglu share the gated tile: C = f(T(G), T(U)) with f = silu(g) u;
+// min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1);  gelu_tanh(g) u.
+enum GemmEpilogue { kPlain = 0, kSwiglu = 1, kAddResidual = 2, kRelu2 = 3, kClamped = 4, kGeglu = 5 };
+constexpr bool gated_epilogue(int e) { return e == kSwiglu || e == kClamped || e == kGeglu; }
 
 struct GemmParams {
     __nv_bfloat16* out;       // [M, n_out]
@@ -49,7 +52,24 @@ struct GemmParams {
     // expert's matrix; a tile whose entry is negative holds no rows and is skipped by every role alike
     const int* tile_expert;
     int expert_rows;
+    float limit, alpha;       // kClamped
 };
+
+// One element of a gated epilogue, from the two products as T rounds them.
+template <int EPI>
+__device__ __forceinline__ float gated_value(float g, float u, float limit, float alpha) {
+    if constexpr (EPI == kClamped) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
+    } else if constexpr (EPI == kGeglu) {
+        // z / 2 (1 + tanh(s)) = z sigmoid(2 s)
+        const float s = 0.7978845608028654f * (g + 0.044715f * g * g * g);
+        return __fdividef(g, 1.f + __expf(-2.f * s)) * u;
+    } else {
+        return rnd<__nv_bfloat16>(__fdividef(g, 1.f + __expf(-g))) * u;
+    }
+}
 
 // Tile t of the walk: groups of kGroupM row tiles are finished one after the other, and within a group the row tile runs
 // fastest.  The blocks that run side by side then cover a patch of at most kGroupM row tiles by a few column tiles, whose
@@ -80,7 +100,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     const __grid_constant__ CUtensorMap map_out, const GemmParams p) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     using L = GemmSmem<BN, STAGES>;
-    constexpr bool SWIGLU = EPI == kSwiglu;
+    constexpr bool SWIGLU = gated_epilogue(EPI);       // gate and up rows in one tile
     static_assert(!SWIGLU || BN == 256, "gate and up rows share a tile of 256");
     pdl_trigger();
     const uint32_t raw_addr = smem_u32(smem_raw);
@@ -215,8 +235,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                 const float g0 = rnd<__nv_bfloat16>(y0), g1 = rnd<__nv_bfloat16>(y1);
                                 const float u0 = rnd<__nv_bfloat16>(__uint_as_float(u[j + 2 * k]));
                                 const float u1 = rnd<__nv_bfloat16>(__uint_as_float(u[j + 2 * k + 1]));
-                                y0 = rnd<__nv_bfloat16>(__fdividef(g0, 1.f + __expf(-g0))) * u0;
-                                y1 = rnd<__nv_bfloat16>(__fdividef(g1, 1.f + __expf(-g1))) * u1;
+                                y0 = gated_value<EPI>(g0, u0, p.limit, p.alpha);
+                                y1 = gated_value<EPI>(g1, u1, p.limit, p.alpha);
                             }
                             if constexpr (EPI == kRelu2) {
                                 y0 = fmaxf(rnd<__nv_bfloat16>(y0), 0.f); y0 *= y0;
@@ -280,7 +300,7 @@ static int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mw, const CUten
         if (e != cudaSuccess) return static_cast<int>(e);
         set = true;
     }
-    constexpr int OUT_COLS = EPI == kSwiglu ? BN / 2 : BN;
+    constexpr int OUT_COLS = gated_epilogue(EPI) ? BN / 2 : BN;
     p.tiles_m = (p.M + kBM - 1) / kBM;
     p.tiles_n = (p.n_out + OUT_COLS - 1) / OUT_COLS;
     const int64_t tiles = static_cast<int64_t>(p.tiles_m) * p.tiles_n;
@@ -296,7 +316,7 @@ static int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mw, const CUten
 using namespace cvb;
 
 // mode 0: C = A W^T.  mode 1: C = silu(A Wg^T) * (A Wu^T) with W = [Wg; Wu].  mode 2: C = rnd(A W^T) + resid (resid may
-// be C itself).  tile_n: 128 or 256 (modes 0 and 2).
+// be C itself).  mode 5: like 1 with gelu_tanh for silu.  tile_n: 128 or 256 (modes 0 and 2).
 extern "C" int cvb_gemm_bf16_tcgen05(void* out, const void* a, const void* w, const void* resid, int M, int N, int K, int mode,
                                      int tile_n, int* err_flag, cudaStream_t stream) {
     if (M == 0) return CVB_OK;
@@ -304,11 +324,12 @@ extern "C" int cvb_gemm_bf16_tcgen05(void* out, const void* a, const void* w, co
     if (K % 8) return CVB_E_ALIGN;                     // rows of A and W must start on 16-byte boundaries for TMA
     auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
     if (!al(out) || !al(a) || !al(w) || !al(resid)) return CVB_E_ALIGN;
-    if (mode == 1 && (N % 2)) return CVB_E_SHAPE;
+    const bool gated = mode == 1 || mode == 5;
+    if (gated && (N % 2)) return CVB_E_SHAPE;
     if (mode == 2 && !resid) return CVB_E_SHAPE;
     GemmParams p{};
     p.out = (__nv_bfloat16*)out; p.resid = (const __nv_bfloat16*)resid; p.M = M; p.N = N; p.K = K;
-    p.n_out = mode == 1 ? N / 2 : N; p.err = err_flag;
+    p.n_out = gated ? N / 2 : N; p.err = err_flag;
     if (p.n_out % 8) return CVB_E_ALIGN;               // 16-byte stores of output rows
     CUtensorMap ma, mw, mo;
     int rc = matrix_map(&ma, a, M, K);
@@ -318,6 +339,7 @@ extern "C" int cvb_gemm_bf16_tcgen05(void* out, const void* a, const void* w, co
     rc = cached_bf16_map(&mo, out, M, p.n_out, 64, 32);      // the epilogue stores boxes of 32 rows by 64 columns
     if (rc != CVB_OK) return rc;
     if (mode == 1) return launch_gemm<256, 4, kSwiglu>(ma, mw, mo, p, stream);
+    if (mode == 5) return launch_gemm<256, 4, kGeglu>(ma, mw, mo, p, stream);
     if (mode == 0) return tile_n == 256 ? launch_gemm<256, 4, kPlain>(ma, mw, mo, p, stream) : launch_gemm<128, 6, kPlain>(ma, mw, mo, p, stream);
     if (mode == 2) return tile_n == 256 ? launch_gemm<256, 4, kAddResidual>(ma, mw, mo, p, stream) : launch_gemm<128, 6, kAddResidual>(ma, mw, mo, p, stream);
     if (mode == 3) return tile_n == 256 ? launch_gemm<256, 4, kRelu2>(ma, mw, mo, p, stream) : launch_gemm<128, 6, kRelu2>(ma, mw, mo, p, stream);
@@ -327,20 +349,22 @@ extern "C" int cvb_gemm_bf16_tcgen05(void* out, const void* a, const void* w, co
 // The grouped form: A [M, K] holds the rows of E experts in segments that start on multiples of 128 rows; row tile i
 // belongs to expert tile_expert[i] (device memory, negative: no rows); W [E * N, K] holds the experts' matrices one below
 // the other.  mode 0: C[M, N] = A W_e^T per tile;  mode 1: C[M, N / 2] = silu(A Wg_e^T) * (A Wu_e^T), W_e = [Wg_e; Wu_e];
-// mode 3: C[M, N] = relu(A W_e^T)^2.
+// mode 3: C[M, N] = relu(A W_e^T)^2;  mode 4: like 1 with the clamped activation of `limit` and `alpha`.
 extern "C" int cvb_gemm_grouped_bf16_tcgen05(void* out, const void* a, const void* w, const int* tile_expert, int M, int N, int E,
-                                             int K, int mode, int tile_n, int* err_flag, cudaStream_t stream) {
+                                             int K, int mode, int tile_n, float limit, float alpha, int* err_flag, cudaStream_t stream) {
     if (M == 0) return CVB_OK;
     if (M < 0 || N <= 0 || K <= 0 || E <= 0 || tile_expert == nullptr) return CVB_E_SIZE;
     if (K % 8 || M % kBM) return CVB_E_ALIGN;
     auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
     if (!al(out) || !al(a) || !al(w)) return CVB_E_ALIGN;
-    if (mode != 0 && mode != 1 && mode != 3) return CVB_E_SHAPE;
-    if (mode == 1 && (N % 2)) return CVB_E_SHAPE;
+    if (mode != 0 && mode != 1 && mode != 3 && mode != 4) return CVB_E_SHAPE;
+    const bool gated = mode == 1 || mode == 4;
+    if (gated && (N % 2)) return CVB_E_SHAPE;
     if (static_cast<int64_t>(E) * N > 2147483647LL) return CVB_E_SIZE;
     GemmParams p{};
     p.out = (__nv_bfloat16*)out; p.resid = nullptr; p.M = M; p.N = N; p.K = K;
-    p.n_out = mode == 1 ? N / 2 : N; p.err = err_flag;
+    p.n_out = gated ? N / 2 : N; p.err = err_flag;
+    p.limit = limit; p.alpha = alpha;
     p.tile_expert = tile_expert; p.expert_rows = N;
     if (p.n_out % 8) return CVB_E_ALIGN;
     CUtensorMap ma, mw, mo;
@@ -351,6 +375,7 @@ extern "C" int cvb_gemm_grouped_bf16_tcgen05(void* out, const void* a, const voi
     rc = cached_bf16_map(&mo, out, M, p.n_out, 64, 32);
     if (rc != CVB_OK) return rc;
     if (mode == 1) return launch_gemm<256, 4, kSwiglu>(ma, mw, mo, p, stream);
+    if (mode == 4) return launch_gemm<256, 4, kClamped>(ma, mw, mo, p, stream);
     if (mode == 3) return tile_n == 256 ? launch_gemm<256, 4, kRelu2>(ma, mw, mo, p, stream) : launch_gemm<128, 6, kRelu2>(ma, mw, mo, p, stream);
     return tile_n == 256 ? launch_gemm<256, 4, kPlain>(ma, mw, mo, p, stream) : launch_gemm<128, 6, kPlain>(ma, mw, mo, p, stream);
 }

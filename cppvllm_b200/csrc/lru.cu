@@ -1,0 +1,370 @@
+// Gated linear recurrence over channels (one float per request and channel instead of a matrix per head):
+//
+//   p = (Wx h) + bx          u_t = sum_m c[ch, m] p_(t - K + 1 + m) + cb       causal, per channel, p = 0 before the sequence's start
+//   per part b of the channels (equal parts):  r = sg(Ra_b u_b + ra_b),  i = sg(Ri_b u_b + ri_b)
+//   l = r * nsp (nsp = -8 softplus(lam) per channel);  S_t = e^l S_(t-1) + sqrt(1 - e^(2 l)) i u;   out = T( S * gelu_tanh((Wy h) + by) )
+//
+// A request's state row holds S [W] and behind it, for K > 1 taps, a ring of the last K inputs p [K, W]: the input at position
+// q lies in row q mod K.  A ring of K rows (one more than the convolution looks back) lets the kernel for decoded tokens write its
+// input while other blocks still read the others; inputs before position 0 are zeros by their position, so a slot needs no
+// clearing for them.  Everything that enters the recurrence is float; u is rounded once to the activations' type T.
+//
+//   lru_conv   : u of every token of the step
+//   (the two gate products of every part are one batched library product into z [parts, T, 2 * part], float)
+//   lru_chunk  : per chunk of a request's tokens and channel: a = e^l and the weighted input, which replace the two products in z,
+//                and what the chunk does to a state: the product of its a and the state it leaves from zero.  A request's first
+//                chunk starts from the request's state instead and leaves that state beside the one it ends with.
+//   lru_finish : per chunk and channel: the state in front of the chunk from the summaries of the chunks before it, then the
+//                tokens one after the other; the gate; a request's last chunk leaves the new state and the ring.  Where no
+//                request has more than one chunk it works from the gate products directly and lru_chunk is not launched.
+//   lru_step   : a step of decoded tokens (one per request): all of it in one kernel.  A block owns a few channels of one part and up
+//                to eight requests: the part's convolutions into shared memory, the two rows of gate weights of a channel read once
+//                for all its requests, the recurrence, the gate, the ring.
+#include "common.cuh"
+
+namespace cvb {
+
+constexpr int kLruThreads = 128;
+
+__device__ __forceinline__ float lru_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float lru_gelu(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+struct LruShape {
+    int W, part, taps, stride;          // channels, channels per part, taps, elements per row of the packed projection
+    int y_off, x_off;                   // columns of the two projections
+    int64_t state_floats;
+    int num_slots;
+};
+
+// u of channel c for the token at packed row t: `local` tokens of its portion lie before it, it sits at position pos.
+template <typename T>
+__device__ __forceinline__ float lru_conv_of(const T* __restrict__ packed, const float* __restrict__ bias_x, const float* __restrict__ conv_w,
+                                             const float* __restrict__ conv_b, const float* __restrict__ ring, const LruShape& sh, int64_t t,
+                                             int local, int pos, int c) {
+    float acc = 0.f;
+    const float b = bias_x[c];
+    for (int m = 0; m < sh.taps; ++m) {
+        const int back = sh.taps - 1 - m;
+        float x = 0.f;
+        if (local >= back) x = to_float(packed[(t - back) * sh.stride + sh.x_off + c]) + b;
+        else if (pos >= back) x = ring[static_cast<int64_t>((pos - back) % sh.taps) * sh.W + c];
+        acc = fmaf(conv_w[static_cast<int64_t>(m) * sh.W + c], x, acc);
+    }
+    return acc + conv_b[c];
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kLruThreads)
+lru_conv_kernel(T* __restrict__ u, const T* __restrict__ packed, const float* __restrict__ bias_x, const float* __restrict__ conv_w,
+                const float* __restrict__ conv_b, const float* __restrict__ state, const int* __restrict__ seq_of_token,
+                const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, const int* __restrict__ positions, LruShape sh,
+                int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t t = blockIdx.x;
+    const int s = seq_of_token[t];
+    const int slot = state_slots[s];
+    if (slot < 0 || slot >= sh.num_slots) {
+        if (threadIdx.x == 0) atomicExch(err, 2);
+        return;
+    }
+    const int local = static_cast<int>(t) - cu_seqlens[s], pos = positions[t];
+    const float* ring = state + static_cast<int64_t>(slot) * sh.state_floats + sh.W;
+    for (int c = blockIdx.y * kLruThreads + threadIdx.x; c < sh.W; c += gridDim.y * kLruThreads)
+        u[t * sh.W + c] = from_float<T>(lru_conv_of(packed, bias_x, conv_w, conv_b, ring, sh, t, local, pos, c));
+}
+
+// Which chunk of which request block x works on: chunk k of request s holds its tokens k * len .. (at most len of them).
+__device__ __forceinline__ bool lru_locate(const int* __restrict__ cu_seqlens, int S, int len, int x, int& s_out, int& k, int& first_chunk) {
+    int base = 0;
+    for (int s = 0; s < S; ++s) {
+        const int n = cu_seqlens[s + 1] - cu_seqlens[s];
+        const int chunks = (n + len - 1) / len;
+        if (x < base + chunks) { s_out = s; k = x - base; first_chunk = base; return true; }
+        base += chunks;
+    }
+    return false;
+}
+
+__device__ __forceinline__ void lru_gate(float zr, float zi, float br, float bi, float nsp, float u, float& a, float& in) {
+    const float l = lru_sigmoid(zr + br) * nsp;
+    a = expf(l);
+    in = sqrtf(fmaxf(-expm1f(2.f * l), 0.f)) * lru_sigmoid(zi + bi) * u;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kLruThreads)
+lru_chunk_kernel(float* __restrict__ z, const T* __restrict__ u, const float* __restrict__ br, const float* __restrict__ bi,
+                 const float* __restrict__ nsp, const float* __restrict__ state, float* __restrict__ summary,
+                 const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, int S, int n_tokens, int len, LruShape sh,
+                 int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    int s, k, first_chunk;
+    if (!lru_locate(cu_seqlens, S, len, blockIdx.x, s, k, first_chunk)) return;
+    const int c = blockIdx.y * kLruThreads + threadIdx.x;
+    if (c >= sh.W) return;
+    const int slot = state_slots[s];
+    if (slot < 0 || slot >= sh.num_slots) {
+        if (threadIdx.x == 0) atomicExch(err, 2);
+        return;
+    }
+    const int t0 = cu_seqlens[s] + k * len, n = min(len, cu_seqlens[s + 1] - t0);
+    const int b = c / sh.part, o = c - b * sh.part;
+    float* zp = z + (static_cast<int64_t>(b) * n_tokens + t0) * 2 * sh.part + o;
+    const T* up = u + static_cast<int64_t>(t0) * sh.W + c;
+    const float rb = br[c], ib = bi[c], ns = nsp[c];
+    float A = 1.f, B = 0.f;
+    if (k == 0) { B = state[static_cast<int64_t>(slot) * sh.state_floats + c]; }
+    const float start = B;
+#pragma unroll 4
+    for (int i = 0; i < n; ++i) {
+        float a, in;
+        lru_gate(zp[static_cast<int64_t>(i) * 2 * sh.part], zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part], rb, ib, ns,
+                 to_float(up[static_cast<int64_t>(i) * sh.W]), a, in);
+        zp[static_cast<int64_t>(i) * 2 * sh.part] = a;
+        zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part] = in;
+        A *= a;
+        B = fmaf(a, B, in);
+    }
+    float* out = summary + static_cast<int64_t>(blockIdx.x) * 2 * sh.W + c;
+    out[0] = k == 0 ? start : A;
+    out[sh.W] = B;
+}
+
+template <typename T, bool GATED>
+__global__ void __launch_bounds__(kLruThreads)
+lru_finish_kernel(T* __restrict__ out, const float* __restrict__ z, const T* __restrict__ u, const T* __restrict__ packed,
+                  const float* __restrict__ bias_y, const float* __restrict__ bias_x, const float* __restrict__ br,
+                  const float* __restrict__ bi, const float* __restrict__ nsp, float* __restrict__ state, const float* __restrict__ summary,
+                  const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, const int* __restrict__ positions, int S,
+                  int n_tokens, int len, LruShape sh, int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    int s, k, first_chunk;
+    if (!lru_locate(cu_seqlens, S, len, blockIdx.x, s, k, first_chunk)) return;
+    const int c = blockIdx.y * kLruThreads + threadIdx.x;
+    if (c >= sh.W) return;
+    const int slot = state_slots[s];
+    if (slot < 0 || slot >= sh.num_slots) {
+        if (threadIdx.x == 0) atomicExch(err, 2);
+        return;
+    }
+    const int begin = cu_seqlens[s], end = cu_seqlens[s + 1];
+    const int t0 = begin + k * len, n = min(len, end - t0);
+    const int b = c / sh.part, o = c - b * sh.part;
+    const float* zp = z + (static_cast<int64_t>(b) * n_tokens + t0) * 2 * sh.part + o;
+    const T* up = u + static_cast<int64_t>(t0) * sh.W + c;
+    const T* yp = packed + static_cast<int64_t>(t0) * sh.stride + sh.y_off + c;
+    T* op = out + static_cast<int64_t>(t0) * sh.W + c;
+    float* row = state + static_cast<int64_t>(slot) * sh.state_floats;
+    float st;
+    if (GATED) {
+        st = row[c];
+    } else {
+        const float* sm = summary + static_cast<int64_t>(first_chunk) * 2 * sh.W + c;
+        if (k == 0) {
+            st = sm[0];
+        } else {
+            st = sm[sh.W];
+#pragma unroll 4
+            for (int j = 1; j < k; ++j) st = fmaf(sm[static_cast<int64_t>(j) * 2 * sh.W], st, sm[static_cast<int64_t>(j) * 2 * sh.W + sh.W]);
+        }
+    }
+    const float rb = GATED ? br[c] : 0.f, ib = GATED ? bi[c] : 0.f, ns = GATED ? nsp[c] : 0.f, yb = bias_y[c];
+#pragma unroll 4
+    for (int i = 0; i < n; ++i) {
+        float a = zp[static_cast<int64_t>(i) * 2 * sh.part], in = zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part];
+        if (GATED) lru_gate(a, in, rb, ib, ns, to_float(up[static_cast<int64_t>(i) * sh.W]), a, in);
+        st = fmaf(a, st, in);
+        op[static_cast<int64_t>(i) * sh.W] = from_float<T>(st * lru_gelu(to_float(yp[static_cast<int64_t>(i) * sh.stride]) + yb));
+    }
+    if (t0 + n == end) {
+        row[c] = st;
+        if (sh.taps > 1) {
+            const float xb = bias_x[c];
+            for (int t = max(begin, end - sh.taps); t < end; ++t)
+                row[sh.W + static_cast<int64_t>(positions[t] % sh.taps) * sh.W + c] = to_float(packed[static_cast<int64_t>(t) * sh.stride + sh.x_off + c]) + xb;
+        }
+    }
+}
+
+constexpr int kStepThreads = 256;
+constexpr int kStepTokens = 8;          // requests per block
+constexpr int kStepChannels = 16;       // channels per block: two per warp
+
+__device__ __forceinline__ void fma8(const __nv_bfloat16* w, float (&f)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(w);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const float2 v = __bfloat1622float2(h[i]); f[2 * i] = v.x; f[2 * i + 1] = v.y; }
+}
+__device__ __forceinline__ void fma8(const float* w, float (&f)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(w), b = *reinterpret_cast<const float4*>(w + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
+// gates [parts, 2 * part, part]: the rows of Ra over the rows of Ri
+template <typename T, int NT>
+__global__ void __launch_bounds__(kStepThreads)
+lru_step_kernel(T* __restrict__ out, const T* __restrict__ packed, const float* __restrict__ bias_y, const float* __restrict__ bias_x,
+                const float* __restrict__ conv_w, const float* __restrict__ conv_b, const T* __restrict__ gates, const float* __restrict__ br,
+                const float* __restrict__ bi, const float* __restrict__ nsp, float* __restrict__ state, const int* __restrict__ cu_seqlens,
+                const int* __restrict__ state_slots, const int* __restrict__ positions, int S, LruShape sh, int vec, int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float us[];         // [NT][ld]
+    const int per_part = (sh.part + kStepChannels - 1) / kStepChannels;
+    const int b = blockIdx.x / per_part, o0 = (blockIdx.x - b * per_part) * kStepChannels;
+    const int s0 = blockIdx.y * NT, nt = min(NT, S - s0);
+    const int ld = (sh.part + 7) / 8 * 8;
+    for (int i = threadIdx.x; i < NT * sh.part; i += kStepThreads) {
+        const int k = i / sh.part, ch = i - k * sh.part;
+        float v = 0.f;
+        if (k < nt) {
+            const int t = cu_seqlens[s0 + k], slot = state_slots[s0 + k];
+            if (slot >= 0 && slot < sh.num_slots)
+                v = rnd<T>(lru_conv_of(packed, bias_x, conv_w, conv_b, state + static_cast<int64_t>(slot) * sh.state_floats + sh.W, sh, t, 0,
+                                       positions[t], b * sh.part + ch));
+            else atomicExch(err, 2);
+        }
+        us[k * ld + ch] = v;
+    }
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int o = o0 + warp; o < min(o0 + kStepChannels, sh.part); o += kStepThreads / 32) {
+        const T* wr = gates + (static_cast<int64_t>(b) * 2 * sh.part + o) * sh.part;
+        const T* wi = wr + static_cast<int64_t>(sh.part) * sh.part;
+        float zr[NT], zi[NT];
+#pragma unroll
+        for (int k = 0; k < NT; ++k) zr[k] = zi[k] = 0.f;
+        if (vec) {
+            for (int e = lane * 8; e < sh.part; e += 256) {
+                float fr[8], fi[8];
+                fma8(wr + e, fr);
+                fma8(wi + e, fi);
+#pragma unroll
+                for (int k = 0; k < NT; ++k) {
+                    const float4 x0 = *reinterpret_cast<const float4*>(us + k * ld + e), x1 = *reinterpret_cast<const float4*>(us + k * ld + e + 4);
+                    const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) { zr[k] = fmaf(x[j], fr[j], zr[k]); zi[k] = fmaf(x[j], fi[j], zi[k]); }
+                }
+            }
+        } else {
+            for (int e = lane; e < sh.part; e += 32) {
+                const float fr = to_float(wr[e]), fi = to_float(wi[e]);
+#pragma unroll
+                for (int k = 0; k < NT; ++k) { const float x = us[k * ld + e]; zr[k] = fmaf(x, fr, zr[k]); zi[k] = fmaf(x, fi, zi[k]); }
+            }
+        }
+        float mr = 0.f, mi = 0.f;                       // lane k keeps request k's pair
+#pragma unroll
+        for (int k = 0; k < NT; ++k) {
+            const float a = warp_sum(zr[k]), d = warp_sum(zi[k]);
+            if (lane == k) { mr = a; mi = d; }
+        }
+        if (lane < nt) {
+            const int t = cu_seqlens[s0 + lane], slot = state_slots[s0 + lane], c = b * sh.part + o;
+            if (slot >= 0 && slot < sh.num_slots) {
+                float* row = state + static_cast<int64_t>(slot) * sh.state_floats;
+                float a, in;
+                lru_gate(mr, mi, br[c], bi[c], nsp[c], us[lane * ld + o], a, in);
+                const float st = fmaf(a, row[c], in);
+                row[c] = st;
+                out[static_cast<int64_t>(t) * sh.W + c] =
+                    from_float<T>(st * lru_gelu(to_float(packed[static_cast<int64_t>(t) * sh.stride + sh.y_off + c]) + bias_y[c]));
+                if (sh.taps > 1)
+                    row[sh.W + static_cast<int64_t>(positions[t] % sh.taps) * sh.W + c] = to_float(packed[static_cast<int64_t>(t) * sh.stride + sh.x_off + c]) + bias_x[c];
+            }
+        }
+    }
+}
+
+}  // namespace cvb
+
+using namespace cvb;
+
+static int lru_shape(LruShape& sh, int W, int parts, int taps, int stride, int y_off, int x_off, int64_t state_floats, int num_slots) {
+    if (W <= 0 || parts <= 0 || taps <= 0 || num_slots <= 0) return CVB_E_SIZE;
+    if (W % parts || y_off < 0 || x_off < 0 || stride < y_off + W || stride < x_off + W) return CVB_E_SHAPE;
+    if (state_floats < static_cast<int64_t>(W) * (taps > 1 ? taps + 1 : 1)) return CVB_E_SHAPE;
+    sh = LruShape{W, W / parts, taps, stride, y_off, x_off, state_floats, num_slots};
+    return CVB_OK;
+}
+
+extern "C" int cvb_lru_conv(void* u, const void* packed, const float* bias_x, const float* conv_w, const float* conv_b, const float* state,
+                            int64_t state_floats, int num_slots, const int* seq_of_token, const int* cu_seqlens, const int* state_slots,
+                            const int* positions, int T, int W, int parts, int taps, int stride, int y_off, int x_off, int dtype, int* err_flag,
+                            cudaStream_t stream) {
+    if (T == 0) return CVB_OK;
+    LruShape sh;
+    const int rc = lru_shape(sh, W, parts, taps, stride, y_off, x_off, state_floats, num_slots);
+    if (rc != CVB_OK || T < 0) return rc != CVB_OK ? rc : CVB_E_SIZE;
+    const dim3 grid(T, min((W + kLruThreads - 1) / kLruThreads, 8));
+#define CALL(TY)                                                                                                              \
+    launch_kernel(lru_conv_kernel<TY>, grid, dim3(kLruThreads), 0, stream, (TY*)u, (const TY*)packed, bias_x, conv_w, conv_b, state, \
+                  seq_of_token, cu_seqlens, state_slots, positions, sh, err_flag)
+    CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+    return launch_status();
+}
+
+// `chunks`: how many chunks of `len` tokens the step's requests have together; `single`: no request has more than one (then
+// `summary` is not used), otherwise `summary` holds 2 * W floats per chunk.
+extern "C" int cvb_lru_scan(void* out, float* z, const void* u, const void* packed, const float* bias_y, const float* bias_x, const float* br,
+                            const float* bi, const float* nsp, float* state, int64_t state_floats, int num_slots, float* summary,
+                            int64_t summary_floats, const int* cu_seqlens, const int* state_slots, const int* positions, int S, int T,
+                            int len, int chunks, int single, int W, int parts, int taps, int stride, int y_off, int x_off, int dtype,
+                            int* err_flag, cudaStream_t stream) {
+    if (T == 0 || S == 0) return CVB_OK;
+    LruShape sh;
+    const int rc = lru_shape(sh, W, parts, taps, stride, y_off, x_off, state_floats, num_slots);
+    if (rc != CVB_OK) return rc;
+    if (T < 0 || S < 0 || len <= 0 || chunks <= 0) return CVB_E_SIZE;
+    if (!single && (summary == nullptr || summary_floats < static_cast<int64_t>(chunks) * 2 * W)) return CVB_E_SCRATCH;
+    const dim3 grid(chunks, (W + kLruThreads - 1) / kLruThreads);
+    if (grid.y > 65535) return CVB_E_SIZE;
+#define CALL(TY)                                                                                                              \
+    if (single) {                                                                                                             \
+        launch_kernel(lru_finish_kernel<TY, true>, grid, dim3(kLruThreads), 0, stream, (TY*)out, z, (const TY*)u, (const TY*)packed, bias_y, \
+                      bias_x, br, bi, nsp, state, summary, cu_seqlens, state_slots, positions, S, T, len, sh, err_flag);       \
+    } else {                                                                                                                  \
+        launch_kernel(lru_chunk_kernel<TY>, grid, dim3(kLruThreads), 0, stream, z, (const TY*)u, br, bi, nsp, state, summary,  \
+                      cu_seqlens, state_slots, S, T, len, sh, err_flag);                                                      \
+        launch_kernel(lru_finish_kernel<TY, false>, grid, dim3(kLruThreads), 0, stream, (TY*)out, z, (const TY*)u, (const TY*)packed, bias_y, \
+                      bias_x, br, bi, nsp, state, summary, cu_seqlens, state_slots, positions, S, T, len, sh, err_flag);       \
+    }
+    CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+    return launch_status();
+}
+
+extern "C" int cvb_lru_step(void* out, const void* packed, const float* bias_y, const float* bias_x, const float* conv_w, const float* conv_b,
+                            const void* gates, const float* br, const float* bi, const float* nsp, float* state, int64_t state_floats,
+                            int num_slots, const int* cu_seqlens, const int* state_slots, const int* positions, int S, int W, int parts,
+                            int taps, int stride, int y_off, int x_off, int dtype, int* err_flag, cudaStream_t stream) {
+    if (S == 0) return CVB_OK;
+    LruShape sh;
+    const int rc = lru_shape(sh, W, parts, taps, stride, y_off, x_off, state_floats, num_slots);
+    if (rc != CVB_OK) return rc;
+    if (S < 0) return CVB_E_SIZE;
+    const int per_part = (sh.part + kStepChannels - 1) / kStepChannels;
+    const int nt = S <= 1 ? 1 : (S <= 2 ? 2 : (S <= 4 ? 4 : kStepTokens));
+    const dim3 grid(parts * per_part, (S + nt - 1) / nt);
+    const size_t smem = static_cast<size_t>(nt) * ((sh.part + 7) / 8 * 8) * sizeof(float);
+    if (smem > 200 * 1024 || grid.y > 65535) return CVB_E_SIZE;
+    const int vec = sh.part % 8 == 0 && (reinterpret_cast<uintptr_t>(gates) & 15) == 0;
+#define CALL_N(TY, NT)                                                                                                        \
+    do {                                                                                                                      \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(lru_step_kernel<TY, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
+        launch_kernel(lru_step_kernel<TY, NT>, grid, dim3(kStepThreads), smem, stream, (TY*)out, (const TY*)packed, bias_y, bias_x,     \
+                      conv_w, conv_b, (const TY*)gates, br, bi, nsp, state, cu_seqlens, state_slots, positions, S, sh, vec, err_flag);  \
+    } while (0)
+#define CALL(TY)                                                                                                              \
+    if (nt == 1) { CALL_N(TY, 1); } else if (nt == 2) { CALL_N(TY, 2); } else if (nt == 4) { CALL_N(TY, 4); } else { CALL_N(TY, 8); }
+    CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+#undef CALL_N
+    return launch_status();
+}

@@ -7,9 +7,15 @@
 //                    winners).  Rows of Wr behind the E experts' (`extra` of them) are not experts: their raw products
 //                    leave as extra_out[t, :] (a gate per token that shares the router's pass over x).
 //                    `mode` 2: weights sigmoid(z_e) of the winners, each on its own (no sum over experts at all).
+//                    `mode` 3: scores s = softmax(z) over all experts; the choice goes by s + bias (a correction that the weights
+//                    do not see) among the experts of the `keep` groups (of `groups` equal groups of neighbours) whose largest
+//                    choice score is largest; weights s_e / (sum over the winners of s_c + 1e-20).
+//   Router outputs behind the E experts that have weights (`identity` of them) stand for the input itself: such a pair adds
+//   weights[t, k] * x[t], touches no weights and gets no row in the sorted order.
 //   With `on_input` = 1 a pair's weight multiplies the expert's INPUT instead of its output: y[t] = sum_k expert_e(T(w_k x[t])).
-//   With `gated` = 0 an expert is  Wd_e ( T(relu(T(Wu_e x))^2) )  and Wgu holds [E, ff, D].
-//   An expert is  Wd_e ( T(act(Wg_e x) * (Wu_e x)) ),  act(z) = z * sigmoid(z);  the layer's output is
+//   With `act` = 0 an expert is  Wd_e ( T(relu(T(Wu_e x))^2) )  and Wgu holds [E, ff, D];  with `act` = 2 it is
+//   Wd_e ( T(g sigmoid(alpha g) (u + 1)) ),  g = min(Wg_e x, limit),  u = clamp(Wu_e x, -limit, limit).
+//   An expert (`act` = 1) is  Wd_e ( T(silu(Wg_e x) * (Wu_e x)) ),  silu(z) = z * sigmoid(z);  the layer's output is
 //   y[t] = T( sum_k weights[t, k] * expert_{ids[t, k]}(x[t]) ).  Wgu is [E, 2 ff, D] (gate rows over up rows), Wd is
 //   [E, D, ff].  Products and the weighted sum are float; the gated activation is rounded to T once, as the input of a
 //   product.
@@ -33,14 +39,14 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x, const float* __restrict__ wr,
                   const float* __restrict__ bias, int n_tokens, int D, int E, int top, int mode, float scale, int extra,
-                  float* __restrict__ extra_out) {
+                  float* __restrict__ extra_out, int groups, int keep) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ float smem[];                     // [kRouteWarps][E]
+    extern __shared__ float smem[];                     // [kRouteWarps][E], mode 3: [kRouteWarps][2 E + groups]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t t = static_cast<int64_t>(blockIdx.x) * kRouteWarps + warp;
     if (t >= n_tokens) return;
-    float* z = smem + warp * E;
+    float* z = smem + warp * (mode == 3 ? 2 * E + groups : E);
     const T* xr = x + t * D;
     // four rows of Wr at a time, each with a sum of its own (a row's sum runs over the same elements in the same order as
     // alone): four independent loads in flight per lane and step instead of one chain
@@ -68,19 +74,45 @@ route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* _
             const float v = warp_sum(d[q]);
             const int e = e0 + q;
             if (lane == 0) {
-                if (e < E) z[e] = v + (bias ? bias[e] : 0.f);
+                if (e < E) z[e] = v + (bias && mode != 3 ? bias[e] : 0.f);
                 else extra_out[t * extra + (e - E)] = v;
             }
         }
     }
     __syncwarp();
-    float all = 0.f;                                    // mode 1: the sum over all experts, against the largest logit
-    if (mode == 1) {
+    float all = 0.f;                                    // modes 1 and 3: the sum over all experts, against the largest logit
+    if (mode == 1 || mode == 3) {
         float big = -INFINITY;
         for (int e = lane; e < E; e += 32) big = fmaxf(big, z[e]);
         big = warp_max(big);
         for (int e = lane; e < E; e += 32) all += expf(z[e] - big);
         all = warp_sum(all);
+        if (mode == 3) {
+            float* s = z + E;                           // the scores; z becomes the choice scores
+            float* best_of = s + E;                     // [groups] the largest choice score of each
+            for (int e = lane; e < E; e += 32) {
+                const float v = expf(z[e] - big) / all;
+                s[e] = v;
+                z[e] = v + (bias ? bias[e] : 0.f);
+            }
+            __syncwarp();
+            const int per = E / groups;
+            for (int g = lane; g < groups; g += 32) {
+                float b = -INFINITY;
+                for (int i = 0; i < per; ++i) b = fmaxf(b, z[g * per + i]);
+                best_of[g] = b;
+            }
+            __syncwarp();
+            // a group is left out if `keep` groups come before it (larger, or equal and in front)
+            for (int e = lane; e < E; e += 32) {
+                const int g = e / per;
+                const float mine = best_of[g];
+                int before = 0;
+                for (int o = 0; o < groups; ++o) before += (best_of[o] > mine || (best_of[o] == mine && o < g)) ? 1 : 0;
+                if (before >= keep) z[e] = -INFINITY;
+            }
+            __syncwarp();
+        }
     }
     float z_first = 0.f, sum = 0.f;
     for (int k = 0; k < top; ++k) {
@@ -97,7 +129,8 @@ route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* _
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
         if (k == 0) z_first = best;
-        const float p = mode == 2 ? best : expf(best - z_first);      // mode 2 keeps the logit itself
+        if (mode == 3 && at >= E) at = 0;               // not reached: the kept groups hold `top` experts or more
+        const float p = mode == 3 ? z[E + at] : (mode == 2 ? best : expf(best - z_first));      // mode 2 keeps the logit itself
         sum += p;
         if (lane == 0) {
             ids[t * top + k] = at;
@@ -110,7 +143,7 @@ route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* _
         for (int k = lane; k < top; k += 32) weights[t * top + k] = scale / (1.f + expf(-weights[t * top + k]));
         return;
     }
-    const float inv = mode == 1 ? scale / all : 1.f / sum;
+    const float inv = mode == 1 ? scale / all : (mode == 3 ? scale / (sum + 1e-20f) : 1.f / sum);
     for (int k = lane; k < top; k += 32) weights[t * top + k] *= inv;     // lane 0's writes are visible after the syncwarp
 }
 
@@ -141,12 +174,23 @@ template <> __device__ __forceinline__ bool rows_by_16_bytes<__nv_bfloat16>(cons
 template <typename T> __device__ __forceinline__ float dot8_of(const T*, const float*, float acc) { return acc; }
 template <> __device__ __forceinline__ float dot8_of<__nv_bfloat16>(const __nv_bfloat16* w, const float* xs, float acc) { return dot8(w, xs, acc); }
 
+constexpr int kActRelu2 = 0, kActClamped = 2;            // 1: silu
+
+__device__ __forceinline__ float gated_of(float g, float u, int act, float limit, float alpha) {
+    if (act == kActClamped) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g * (1.f / (1.f + expf(-alpha * g))) * (u + 1.f);
+    }
+    return silu_exact<float>(g) * u;
+}
+
 // hid[pair, f] = T(silu(Wg_e[f] . x) * (Wu_e[f] . x)) for the block's slice of f; pair = t * top + k, e = ids[pair]
 template <typename T>
 __global__ void __launch_bounds__(kExpertThreads)
 expert_hidden_kernel(T* __restrict__ hid, const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ wgu,
-                     int D, int F, int E, int top, int per_block, int gated, const float* __restrict__ in_weights,
-                     int* __restrict__ err) {
+                     int D, int F, int E, int top, int per_block, int act, const float* __restrict__ in_weights,
+                     int identity, float limit, float alpha, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float smem[];
@@ -155,10 +199,12 @@ expert_hidden_kernel(T* __restrict__ hid, const T* __restrict__ x, const int* __
     const int64_t t = pair / top;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     int e = ids[pair];
+    if (e >= E && e < E + identity) return;             // the input itself: nothing to compute here
     if (e < 0 || e >= E) {
         if (threadIdx.x == 0) atomicExch(err, 7);
         e = 0;
     }
+    const bool gated = act != kActRelu2;
     const float wi = in_weights != nullptr ? in_weights[pair] : 1.f;
     if (in_weights != nullptr) {
         for (int i = threadIdx.x; i < D; i += kExpertThreads) xs[i] = rnd<T>(wi * to_float(x[t * D + i]));
@@ -175,14 +221,18 @@ expert_hidden_kernel(T* __restrict__ hid, const T* __restrict__ x, const int* __
         const T* ur = u_rows + static_cast<int64_t>(f) * D;
         float g = 0.f, u = 0.f;
         if (gated) {
-            for (int i = lane; i < D; i += 32) {
-                const float xv = xs[i];
-                g = fmaf(xv, to_float(gr[i]), g);
-                u = fmaf(xv, to_float(ur[i]), u);
+            if (wide) {
+                for (int i = lane * 8; i < D; i += 256) { g = dot8_of<T>(gr + i, xs + i, g); u = dot8_of<T>(ur + i, xs + i, u); }
+            } else {
+                for (int i = lane; i < D; i += 32) {
+                    const float xv = xs[i];
+                    g = fmaf(xv, to_float(gr[i]), g);
+                    u = fmaf(xv, to_float(ur[i]), u);
+                }
             }
             g = warp_sum(g);
             u = warp_sum(u);
-            if (lane == 0) hid[pair * F + f] = from_float<T>(silu_exact<T>(g) * u);
+            if (lane == 0) hid[pair * F + f] = from_float<T>(gated_of(g, u, act, limit, alpha));
         } else {
             if (wide) {
                 for (int i = lane * 8; i < D; i += 256) g = dot8_of<T>(gr + i, xs + i, g);
@@ -198,8 +248,9 @@ expert_hidden_kernel(T* __restrict__ hid, const T* __restrict__ x, const int* __
 // y[t, d] = T(sum_k weights[t, k] * (Wd_e[d] . hid[t * top + k])) for the block's slice of d
 template <typename T>
 __global__ void __launch_bounds__(kExpertThreads)
-expert_down_kernel(T* __restrict__ y, const T* __restrict__ hid, const int* __restrict__ ids, const float* __restrict__ weights,
-                   const T* __restrict__ wd, int D, int F, int E, int top, int per_block, int on_input) {
+expert_down_kernel(T* __restrict__ y, const T* __restrict__ hid, const T* __restrict__ x, const int* __restrict__ ids,
+                   const float* __restrict__ weights, const T* __restrict__ wd, int D, int F, int E, int top, int per_block, int on_input,
+                   int identity) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float smem[];
@@ -209,11 +260,17 @@ expert_down_kernel(T* __restrict__ y, const T* __restrict__ hid, const int* __re
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int d0 = blockIdx.y * per_block, d1 = min(D, d0 + per_block);
     for (int i = threadIdx.x; i < per_block; i += kExpertThreads) acc[i] = 0.f;
+    __syncthreads();                                    // an identity expert adds before any other barrier
     const bool wide = rows_by_16_bytes<T>(wd, F);
     for (int k = 0; k < top; ++k) {
         int e = ids[t * top + k];
-        if (e < 0 || e >= E) e = 0;                      // reported by the kernel in front
         const float wk = on_input ? 1.f : weights[t * top + k];
+        if (e >= E && e < E + identity) {                // the input itself, times the weight
+            for (int d = d0 + warp; d < d1; d += kExpertWarps)
+                if (lane == 0) acc[d - d0] = fmaf(weights[t * top + k], to_float(x[t * D + d]), acc[d - d0]);
+            continue;
+        }
+        if (e < 0 || e >= E) e = 0;                      // reported by the kernel in front
         __syncthreads();
         for (int i = threadIdx.x; i < F; i += kExpertThreads) hs[i] = to_float(hid[(t * top + k) * F + i]);
         __syncthreads();
@@ -242,10 +299,11 @@ constexpr int kSortThreads = 1024;
 // grouped product's row tiles are 128 rows of ONE expert).  One block.  The order of an expert's rows among themselves
 // is not fixed; no result depends on it.  tile_expert[i]: the expert of row tile i, -1 for tiles behind the last segment (max_tiles
 // entries).  row_token[slot]: the token whose row goes to sorted row `slot` (0 for the padding rows: they are computed
-// and never read).  slot_of[pair]: where the pair's row lies.
+// and never read).  slot_of[pair]: where the pair's row lies; -1 for a pair whose expert is the input itself.
 __global__ void __launch_bounds__(kSortThreads)
 sort_pairs_padded_kernel(int* __restrict__ tile_expert, int* __restrict__ row_token, int* __restrict__ slot_of,
-                         const int* __restrict__ ids, int n_pairs, int E, int top, int pad, int max_tiles, int* __restrict__ err) {
+                         const int* __restrict__ ids, int n_pairs, int E, int top, int pad, int max_tiles, int identity,
+                         int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ int ismem[];
@@ -256,6 +314,7 @@ sort_pairs_padded_kernel(int* __restrict__ tile_expert, int* __restrict__ row_to
     __syncthreads();
     for (int i = threadIdx.x; i < n_pairs; i += kSortThreads) {
         int e = ids[i];
+        if (e >= E && e < E + identity) continue;
         if (e < 0 || e >= E) { atomicExch(err, 7); e = 0; }
         atomicAdd(&count[e], 1);
     }
@@ -283,6 +342,7 @@ sort_pairs_padded_kernel(int* __restrict__ tile_expert, int* __restrict__ row_to
     __syncthreads();
     for (int i = threadIdx.x; i < n_pairs; i += kSortThreads) {
         int e = ids[i];
+        if (e >= E && e < E + identity) { slot_of[i] = -1; continue; }
         if (e < 0 || e >= E) e = 0;
         const int slot = start[e] + atomicAdd(&count[e], 1);
         row_token[slot] = i / top;
@@ -298,21 +358,24 @@ __global__ void scatter_pairs_scaled_kernel(__nv_bfloat16* __restrict__ xs, cons
     pdl_wait();
     const int64_t pair = blockIdx.x;
     const float w = weights[pair];
+    if (slot_of[pair] < 0) return;
     const __nv_bfloat16* src = x + pair / top * D;
     __nv_bfloat16* dst = xs + static_cast<int64_t>(slot_of[pair]) * D;
     for (int d = threadIdx.x; d < D; d += blockDim.x) dst[d] = __float2bfloat16_rn(w * __bfloat162float(src[d]));
 }
 
-// y[t, :] = sum_k weights[t, k] * rows[slot_of[t * top + k], :]   (weights = nullptr: all 1)
-__global__ void combine_pairs_kernel(__nv_bfloat16* __restrict__ y, const __nv_bfloat16* __restrict__ rows, const int* __restrict__ slot_of,
-                                     const float* __restrict__ weights, int D, int top) {
+// y[t, :] = sum_k weights[t, k] * rows[slot_of[t * top + k], :]   (weights = nullptr: all 1; a negative slot: x[t, :] instead)
+__global__ void combine_pairs_kernel(__nv_bfloat16* __restrict__ y, const __nv_bfloat16* __restrict__ rows, const __nv_bfloat16* __restrict__ x,
+                                     const int* __restrict__ slot_of, const float* __restrict__ weights, int D, int top) {
     pdl_trigger();
     pdl_wait();
     const int64_t t = blockIdx.x;
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
         float s = 0.f;
-        for (int k = 0; k < top; ++k)
-            s = fmaf(weights != nullptr ? weights[t * top + k] : 1.f, __bfloat162float(rows[static_cast<int64_t>(slot_of[t * top + k]) * D + d]), s);
+        for (int k = 0; k < top; ++k) {
+            const int64_t slot = slot_of[t * top + k];
+            s = fmaf(weights != nullptr ? weights[t * top + k] : 1.f, __bfloat162float(slot >= 0 ? rows[slot * D + d] : x[t * D + d]), s);
+        }
         y[t * D + d] = __float2bfloat16_rn(s);
     }
 }
@@ -322,24 +385,28 @@ __global__ void combine_pairs_kernel(__nv_bfloat16* __restrict__ y, const __nv_b
 using namespace cvb;
 
 extern "C" int cvb_route_topk(int* ids, float* weights, const void* x, const float* wr, const float* bias, int T, int D, int E,
-                              int top, int mode, float scale, int extra, float* extra_out, int dtype, cudaStream_t stream) {
+                              int top, int mode, float scale, int extra, float* extra_out, int groups, int keep, int dtype,
+                              cudaStream_t stream) {
     if (T == 0) return CVB_OK;
     if (T < 0 || D <= 0 || E <= 0 || top <= 0 || extra < 0 || (extra > 0 && extra_out == nullptr)) return CVB_E_SIZE;
-    if (mode < 0 || mode > 2) return CVB_E_SHAPE;
+    if (mode < 0 || mode > 3) return CVB_E_SHAPE;
     if (top > E || E > 2048) return CVB_E_SHAPE;
-    const size_t smem = static_cast<size_t>(kRouteWarps) * E * sizeof(float);
+    if (mode == 3 && (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups))) return CVB_E_SHAPE;
+    const size_t smem = static_cast<size_t>(kRouteWarps) * (mode == 3 ? 2 * E + groups : E) * sizeof(float);
+    if (smem > 48 * 1024) return CVB_E_SIZE;
 #define CALL(TY) launch_kernel(route_topk_kernel<TY>, dim3((T + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), smem, \
-                               stream, ids, weights, (const TY*)x, wr, bias, T, D, E, top, mode, scale, extra, extra_out)
+                               stream, ids, weights, (const TY*)x, wr, bias, T, D, E, top, mode, scale, extra, extra_out, groups, keep)
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
     return launch_status();
 }
 
 extern "C" int cvb_expert_rows(void* y, void* hid, const void* x, const int* ids, const float* weights, const void* wgu,
-                               const void* wd, int T, int D, int F, int E, int top, int gated, int on_input, int dtype, int* err_flag,
-                               cudaStream_t stream) {
+                               const void* wd, int T, int D, int F, int E, int top, int act, int on_input, int identity, float limit,
+                               float alpha, int dtype, int* err_flag, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
-    if (T < 0 || D <= 0 || F <= 0 || E <= 0 || top <= 0) return CVB_E_SIZE;
+    if (T < 0 || D <= 0 || F <= 0 || E <= 0 || top <= 0 || identity < 0) return CVB_E_SIZE;
+    if (act < kActRelu2 || act > kActClamped) return CVB_E_SHAPE;
     if (static_cast<size_t>(D) * sizeof(float) > 160 * 1024 || static_cast<size_t>(F) * sizeof(float) > 160 * 1024) return CVB_E_SIZE;
     // slices sized so that a step of one token still gives every SM a block or two
     const int64_t pairs = static_cast<int64_t>(T) * top;
@@ -357,9 +424,9 @@ extern "C" int cvb_expert_rows(void* y, void* hid, const void* x, const int* ids
         if (smem2 > 48 * 1024)                                                                                           \
             cudaFuncSetAttribute(expert_down_kernel<TY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);       \
         launch_kernel(expert_hidden_kernel<TY>, dim3((unsigned)pairs, (F + f_per - 1) / f_per), dim3(kExpertThreads), smem1,  \
-                      stream, (TY*)hid, (const TY*)x, ids, (const TY*)wgu, D, F, E, top, f_per, gated, on_input ? weights : nullptr, err_flag);                \
+                      stream, (TY*)hid, (const TY*)x, ids, (const TY*)wgu, D, F, E, top, f_per, act, on_input ? weights : nullptr, identity, limit, alpha, err_flag); \
         launch_kernel(expert_down_kernel<TY>, dim3(T, (D + d_per - 1) / d_per), dim3(kExpertThreads), smem2, stream,      \
-                      (TY*)y, (const TY*)hid, ids, weights, (const TY*)wd, D, F, E, top, d_per, on_input);                          \
+                      (TY*)y, (const TY*)hid, (const TY*)x, ids, weights, (const TY*)wd, D, F, E, top, d_per, on_input, identity);    \
     } while (0)
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
@@ -368,12 +435,12 @@ extern "C" int cvb_expert_rows(void* y, void* hid, const void* x, const int* ids
 
 // Sorts the pairs for the tcgen05 grouped product (see sort_pairs_padded_kernel); max_tiles * 128 rows of scratch.
 extern "C" int cvb_sort_pairs_padded(int* tile_expert, int* row_token, int* slot_of, const int* ids, int T, int E, int top,
-                                     int max_tiles, int* err_flag, cudaStream_t stream) {
+                                     int max_tiles, int identity, int* err_flag, cudaStream_t stream) {
     if (T <= 0 || E <= 0 || top <= 0 || max_tiles <= 0 || E > 4096) return CVB_E_SIZE;
     const int64_t pairs = static_cast<int64_t>(T) * top;
     if (pairs > (1 << 30) || (pairs + 127) / 128 + E > max_tiles) return CVB_E_SCRATCH;
     launch_kernel(sort_pairs_padded_kernel, dim3(1), dim3(kSortThreads), (2 * static_cast<size_t>(E) + 1) * sizeof(int), stream,
-                  tile_expert, row_token, slot_of, ids, static_cast<int>(pairs), E, top, 128, max_tiles, err_flag);
+                  tile_expert, row_token, slot_of, ids, static_cast<int>(pairs), E, top, 128, max_tiles, identity, err_flag);
     return launch_status();
 }
 
@@ -385,10 +452,10 @@ extern "C" int cvb_scatter_pairs_scaled_bf16(void* xs, const void* x, const int*
     return launch_status();
 }
 
-extern "C" int cvb_combine_pairs_bf16(void* y, const void* rows, const int* slot_of, const float* weights, int T, int D, int top,
+extern "C" int cvb_combine_pairs_bf16(void* y, const void* rows, const void* x, const int* slot_of, const float* weights, int T, int D, int top,
                                       cudaStream_t stream) {
     if (T <= 0 || D <= 0 || top <= 0) return CVB_E_SIZE;
     launch_kernel(combine_pairs_kernel, dim3(T), dim3(D >= 1024 ? 256 : 128), 0, stream, (__nv_bfloat16*)y,
-                  (const __nv_bfloat16*)rows, slot_of, weights, D, top);
+                  (const __nv_bfloat16*)rows, (const __nv_bfloat16*)x, slot_of, weights, D, top);
     return launch_status();
 }

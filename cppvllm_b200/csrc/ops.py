@@ -327,17 +327,17 @@ def bias_act(out: torch.Tensor, x: torch.Tensor, bias: Optional[torch.Tensor], a
 def gated_norm(out: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, groups: int, eps: float,
                gate_act: str = "sigmoid") -> torch.Tensor:
     """out[t, g, :] = RMSNorm(o[t, g, :]) * weight * sigmoid(gate[t, g, :]) (or * silu(gate): `gate_act` = "silu") over `groups` groups of weight.numel() elements;
-    o float32 [T, groups * G]; gate a view of [T, groups * G] columns inside rows of gate.stride(0) elements."""
-    _cuda(out, o, gate, weight); _contig(out, o, weight)
+    o float32 [T, groups * G]; out may be a column range of wider rows; gate a view of [T, groups * G] columns inside rows of gate.stride(0) elements."""
+    _cuda(out, o, gate, weight); _contig(o, weight)
     T = o.shape[0]
     G = weight.numel()
     if gate_act not in ("sigmoid", "silu"):
         raise KernelError("gated_norm: gate_act is sigmoid or silu")
     if (o.dtype != torch.float32 or o.shape[1] != groups * G or out.shape != o.shape or gate.dtype != out.dtype or gate.dim() != 2
-            or gate.shape != o.shape or gate.stride(1) != 1 or weight.dtype != torch.float32):
+            or gate.shape != o.shape or gate.stride(1) != 1 or out.stride(1) != 1 or weight.dtype != torch.float32):
         raise KernelError("gated_norm: o float32 [T, groups * G]; out and gate [T, groups * G] of the activations' type; weight float32 [G]")
     _check(_resid32_lib().cvb_gated_norm(_ptr(out), _ptr(o), _ptr(gate), c_int(gate.stride(0)), _ptr(weight), c_int(T), c_int(groups),
-                                         c_int(G), c_float(eps), c_int(1 if gate_act == "silu" else 0), c_int(dtype_code(out.dtype)), _stream()), "gated_norm")
+                                         c_int(G), c_float(eps), c_int(1 if gate_act == "silu" else 0), c_int(out.stride(0)), c_int(dtype_code(out.dtype)), _stream()), "gated_norm")
     return out
 
 
@@ -350,7 +350,7 @@ def _sandwich_lib():
     global _sandwich
     if _sandwich is None:
         lib = load_library("sandwich")
-        for name in ("cvb_input_conv", "cvb_gated_norm_add", "cvb_glu_clamped", "cvb_add_gated_rows", "cvb_wide_qk_prep"):
+        for name in ("cvb_input_conv", "cvb_gated_norm_add", "cvb_glu_act", "cvb_add_gated_rows", "cvb_wide_qk_prep"):
             getattr(lib, name).restype = c_int
         _sandwich = lib
     return _sandwich
@@ -408,8 +408,19 @@ def glu_clamped(out: torch.Tensor, gate_up: torch.Tensor, limit: float, alpha: f
     T, I = out.shape
     if gate_up.shape != (T, 2 * I) or gate_up.dtype != out.dtype:
         raise KernelError("glu_clamped: gate_up must be [T, 2I] for out [T, I]")
-    _check(_sandwich_lib().cvb_glu_clamped(_ptr(out), _ptr(gate_up), c_int(T), c_int(I), c_float(limit), c_float(alpha),
-                                           c_int(dtype_code(out.dtype)), _stream()), "glu_clamped")
+    _check(_sandwich_lib().cvb_glu_act(_ptr(out), _ptr(gate_up), c_int(T), c_int(I), c_int(0), c_float(limit), c_float(alpha),
+                                       c_int(dtype_code(out.dtype)), _stream()), "glu_clamped")
+    return out
+
+
+def geglu(out: torch.Tensor, gate_up: torch.Tensor) -> torch.Tensor:
+    """out = gelu_tanh(gate) * up; gate_up [T, 2 I] (gate columns, then up)."""
+    _cuda(out, gate_up); _contig(out, gate_up)
+    T, I = out.shape
+    if gate_up.shape != (T, 2 * I) or gate_up.dtype != out.dtype:
+        raise KernelError("geglu: gate_up must be [T, 2I] for out [T, I]")
+    _check(_sandwich_lib().cvb_glu_act(_ptr(out), _ptr(gate_up), c_int(T), c_int(I), c_int(1), c_float(0.0), c_float(0.0),
+                                       c_int(dtype_code(out.dtype)), _stream()), "geglu")
     return out
 
 
@@ -603,7 +614,8 @@ def _recurrent_lib():
     global _recurrent
     if _recurrent is None:
         lib = load_library("recurrent")
-        for name in ("cvb_lightning_prep", "cvb_lightning_scan", "cvb_delta_prep", "cvb_conv_history", "cvb_delta_scan"):
+        for name in ("cvb_lightning_prep", "cvb_lightning_scan", "cvb_linear_prep", "cvb_linear_scan", "cvb_linear_step", "cvb_delta_prep",
+                     "cvb_conv_history", "cvb_delta_scan"):
             getattr(lib, name).restype = c_int
         _recurrent = lib
     return _recurrent
@@ -643,6 +655,180 @@ def lightning_scan(out: torch.Tensor, qf: torch.Tensor, kf: torch.Tensor, vf: to
     _check(_recurrent_lib().cvb_lightning_scan(
         _ptr(out), _ptr(qf), _ptr(kf), _ptr(vf), sp, sf, _ptr(decay), _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs),
         c_int(num_heads), c_int(dim), c_int(vdim), _ptr(error_flag(out.device)), _stream()), "lightning_scan")
+    return out
+
+
+def linear_prep(qf: torch.Tensor, kf: torch.Tensor, vf: torch.Tensor, gg: torch.Tensor, packed: torch.Tensor, q_off: int, k_off: int,
+                v_off: int, z: torch.Tensor, bias: torch.Tensor, qk_scale: float, tau: float) -> None:
+    """qf = qk_scale * q, kf = k [T, H * dim] and vf = v [T, H * vdim] (float32) from the packed projection's column ranges, and the decays
+    gg = sigmoid(z + bias)^(1 / tau) [T, H * dim] from the float32 product z (gg may be z itself)."""
+    _cuda(qf, kf, vf, gg, packed, z, bias); _contig(qf, kf, vf, gg, z, bias)
+    T = packed.shape[0]
+    if (any(t.dtype != torch.float32 for t in (qf, kf, vf, gg, z, bias)) or kf.shape != qf.shape or gg.shape != qf.shape or z.shape != qf.shape
+            or qf.shape[0] != T or vf.shape[0] != T or bias.numel() != qf.shape[1] or packed.stride(1) != 1):
+        raise KernelError("linear_prep: q, k, decays and z float32 [T, H * dim], v float32 [T, H * vdim], bias float32 [H * dim]")
+    _check(_recurrent_lib().cvb_linear_prep(_ptr(qf), _ptr(kf), _ptr(vf), _ptr(gg), _ptr(packed), c_int(T), c_int(packed.stride(0)), c_int(q_off),
+                                            c_int(k_off), c_int(v_off), _ptr(z), _ptr(bias), c_float(qk_scale), c_float(1.0 / tau),
+                                            c_int(qf.shape[1]), c_int(vf.shape[1]), c_int(dtype_code(packed.dtype)), _stream()), "linear_prep")
+
+
+def linear_scan(out: torch.Tensor, qf: torch.Tensor, kf: torch.Tensor, vf: torch.Tensor, gg: torch.Tensor, state: torch.Tensor,
+                cu_seqlens: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, num_heads: int, dim: int, vdim: int) -> torch.Tensor:
+    """Per request and head, over the request's tokens of this step: S <- diag(g) S + k v^T, out = S^T q; q, k, g [T, H * dim] and v
+    [T, H * vdim] float32; S [dim, vdim] float32 at the front of the request's state row.  out float32 [T, H * vdim]."""
+    _cuda(out, qf, kf, vf, gg, state, cu_seqlens, state_slots); _contig(out, qf, kf, vf, gg, cu_seqlens, state_slots)
+    sp, sf, n_slots = _state_args(state)
+    T = qf.shape[0]
+    if (any(t.dtype != torch.float32 for t in (out, qf, kf, vf, gg)) or out.shape != (T, num_heads * vdim) or qf.shape != (T, num_heads * dim)
+            or kf.shape != qf.shape or gg.shape != qf.shape or vf.shape != out.shape or cu_seqlens.dtype != torch.int32
+            or state_slots.dtype != torch.int32):
+        raise KernelError("linear_scan: q, k, g float32 [T, H * dim]; v, out float32 [T, H * vdim]; cu_seqlens, state_slots int32")
+    _check(_recurrent_lib().cvb_linear_scan(
+        _ptr(out), _ptr(qf), _ptr(kf), _ptr(vf), _ptr(gg), sp, sf, _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs),
+        c_int(num_heads), c_int(dim), c_int(vdim), _ptr(error_flag(out.device)), _stream()), "linear_scan")
+    return out
+
+
+def linear_step_supported(dim: int, vdim: int, rank: int) -> bool:
+    """Whether the one-kernel form of a step of decoded tokens holds a head's vectors in shared memory."""
+    return (3 * dim + rank + max(1024, vdim)) * 4 <= 48 * 1024
+
+
+def linear_step(out: torch.Tensor, packed: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, a_off: int, w_a2: torch.Tensor,
+                a2_bias: torch.Tensor, qk_scale: float, tau: float, norm_weight: torch.Tensor, eps: float, out_scale: float,
+                state: torch.Tensor, cu_seqlens: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, num_heads: int, dim: int,
+                vdim: int) -> torch.Tensor:
+    """A step of one token per request: decays sigmoid(w_a2 a + bias)^(1 / tau), S <- diag(g) S + k v^T, o = S^T (qk_scale q), out =
+    out_scale * RMSNorm(o_h) * norm_weight * silu(gate_h), in `packed`'s element type; all inputs are column ranges of `packed`."""
+    _cuda(out, packed, w_a2, a2_bias, norm_weight, state, cu_seqlens, state_slots)
+    _contig(w_a2, a2_bias, norm_weight, cu_seqlens, state_slots)
+    sp, sf, n_slots = _state_args(state)
+    rank = w_a2.shape[1]
+    if (out.dtype != packed.dtype or w_a2.dtype != packed.dtype or w_a2.shape[0] != num_heads * dim or out.shape[1] != num_heads * vdim
+            or out.stride(1) != 1 or packed.stride(1) != 1 or out.shape[0] < num_seqs or packed.shape[0] < num_seqs
+            or a2_bias.dtype != torch.float32 or a2_bias.numel() != num_heads * dim or norm_weight.dtype != torch.float32
+            or norm_weight.numel() != vdim or cu_seqlens.dtype != torch.int32 or state_slots.dtype != torch.int32):
+        raise KernelError("linear_step: out [S, H * vdim], w_a2 [H * dim, rank] of packed's element type; bias, norm weight float32")
+    _check(_recurrent_lib().cvb_linear_step(
+        _ptr(out), c_int(out.stride(0)), _ptr(packed), c_int(packed.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), c_int(g_off),
+        c_int(a_off), c_int(rank), _ptr(w_a2), _ptr(a2_bias), c_float(qk_scale), c_float(1.0 / tau), _ptr(norm_weight), c_float(eps),
+        c_float(out_scale), sp, sf, _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs), c_int(num_heads), c_int(dim),
+        c_int(vdim), c_int(dtype_code(packed.dtype)), _ptr(error_flag(packed.device)), _stream()), "linear_step")
+    return out
+
+
+# ---- gated linear recurrence over channels (csrc/lru.cu) ---------------------------------------------------------------------
+
+_lru = None
+
+
+def _lru_lib():
+    global _lru
+    if _lru is None:
+        lib = load_library("lru")
+        for name in ("cvb_lru_conv", "cvb_lru_scan", "cvb_lru_step"):
+            getattr(lib, name).restype = c_int
+        _lru = lib
+    return _lru
+
+
+def _lru_check(packed, width, parts, y_off, x_off, vectors, ints):
+    if packed.stride(1) != 1 or width % parts or packed.shape[1] < max(y_off, x_off) + width:
+        raise KernelError("lru: the packed rows hold both projections of `width` channels, in equal parts")
+    for t, n in vectors:
+        if t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous():
+            raise KernelError("lru: biases, convolution and decay vectors are contiguous float32 of the channels' sizes")
+    for t in ints:
+        if t.dtype != torch.int32 or not t.is_contiguous():
+            raise KernelError("lru: index tensors are int32")
+
+
+def lru_chunk_tokens(num_tokens: int) -> int:
+    """Tokens per chunk of a request's portion: short enough that a long prompt's chunks fill the SMs, long enough that the chunks
+    before a chunk are few."""
+    return 32 if num_tokens <= 1024 else (64 if num_tokens <= 4096 else 128)
+
+
+def lru_conv(u: torch.Tensor, packed: torch.Tensor, y_off: int, x_off: int, parts: int, bias_x, conv_w, conv_b, state, seq_of_token, cu_seqlens,
+             state_slots, positions) -> torch.Tensor:
+    """u [T, W]: the causal convolution over time of (packed's x columns + bias_x), taps conv_w float32 [taps, W] (oldest first), plus
+    conv_b; inputs before the portion come from the ring behind S in the request's state row."""
+    T, W = u.shape
+    taps = conv_w.shape[0]
+    _cuda(u, packed, bias_x, conv_w, conv_b, state, seq_of_token, cu_seqlens, state_slots, positions)
+    _lru_check(packed, W, parts, y_off, x_off, ((bias_x, W), (conv_w, taps * W), (conv_b, W)), (seq_of_token, cu_seqlens, state_slots, positions))
+    sp, sf, n_slots = _state_args(state)
+    if u.dtype != packed.dtype or packed.shape[0] != T or not u.is_contiguous():
+        raise KernelError("lru_conv: u [T, W] of packed's element type")
+    _check(_lru_lib().cvb_lru_conv(_ptr(u), _ptr(packed), _ptr(bias_x), _ptr(conv_w), _ptr(conv_b), sp, sf, c_int(n_slots), _ptr(seq_of_token),
+                                   _ptr(cu_seqlens), _ptr(state_slots), _ptr(positions), c_int(T), c_int(W), c_int(parts), c_int(taps),
+                                   c_int(packed.stride(0)), c_int(y_off), c_int(x_off), c_int(dtype_code(packed.dtype)),
+                                   _ptr(error_flag(packed.device)), _stream()), "lru_conv")
+    return u
+
+
+def lru_gates(z: torch.Tensor, u: torch.Tensor, gates: torch.Tensor) -> torch.Tensor:
+    """z [parts, T, 2 * part] (float32) = u's parts times gates [parts, 2 * part, part]^T: one batched library product."""
+    _cuda(z, u, gates); _contig(z, u, gates)
+    parts, two, part = gates.shape
+    T = u.shape[0]
+    if u.dtype != gates.dtype or u.shape[1] != parts * part or two != 2 * part or z.dtype != torch.float32 or z.numel() != T * parts * two:
+        raise KernelError("lru_gates: u [T, parts * part], gates [parts, 2 * part, part] of one element type, z float32 [parts, T, 2 * part]")
+    a = u.view(T, parts, part).transpose(0, 1)
+    if u.dtype == torch.float32:
+        torch.bmm(a, gates.transpose(1, 2), out=z.view(parts, T, two))
+    else:
+        torch.bmm(a, gates.transpose(1, 2), out_dtype=torch.float32, out=z.view(parts, T, two))
+    return z
+
+
+def lru_scan(out: torch.Tensor, z: torch.Tensor, u: torch.Tensor, packed: torch.Tensor, y_off: int, x_off: int, parts: int, taps: int, bias_y, bias_x,
+             bias_r, bias_i, neg_softplus, state, cu_seqlens, state_slots, positions, q_lens, chunk_tokens: int,
+             summary: Optional[torch.Tensor]) -> torch.Tensor:
+    """out [T, W] = S_t * gelu_tanh(y + bias_y) over every request's tokens, from the gate products z (overwritten), u and the packed
+    projection; S and the ring in the state rows move on.  `q_lens`: the requests' portion lengths; portions longer than
+    `chunk_tokens` are worked on in chunks side by side through `summary` (float32, 2 * W per chunk)."""
+    T, W = out.shape
+    _cuda(out, z, u, packed, bias_y, bias_x, bias_r, bias_i, neg_softplus, state, cu_seqlens, state_slots, positions, summary)
+    _contig(out, z, u, summary)
+    _lru_check(packed, W, parts, y_off, x_off, tuple((v, W) for v in (bias_y, bias_x, bias_r, bias_i, neg_softplus)),
+               (cu_seqlens, state_slots, positions))
+    sp, sf, n_slots = _state_args(state)
+    if (out.dtype != packed.dtype or u.dtype != out.dtype or u.shape != out.shape or packed.shape[0] != T or z.dtype != torch.float32
+            or z.numel() != 2 * T * W or (summary is not None and summary.dtype != torch.float32)):
+        raise KernelError("lru_scan: out, u [T, W] of packed's element type, z float32 [parts, T, 2 * part], summary float32")
+    chunks = sum((n + chunk_tokens - 1) // chunk_tokens for n in q_lens)
+    single = max(q_lens) <= chunk_tokens
+    _check(_lru_lib().cvb_lru_scan(
+        _ptr(out), _ptr(z), _ptr(u), _ptr(packed), _ptr(bias_y), _ptr(bias_x), _ptr(bias_r), _ptr(bias_i), _ptr(neg_softplus), sp, sf,
+        c_int(n_slots), _ptr(summary), c_int64(summary.numel() if summary is not None else 0), _ptr(cu_seqlens), _ptr(state_slots),
+        _ptr(positions), c_int(len(q_lens)), c_int(T), c_int(chunk_tokens), c_int(chunks), c_int(1 if single else 0), c_int(W), c_int(parts),
+        c_int(taps), c_int(packed.stride(0)), c_int(y_off), c_int(x_off), c_int(dtype_code(packed.dtype)), _ptr(error_flag(out.device)),
+        _stream()), "lru_scan", kernels=1 if single else 2)
+    return out
+
+
+LRU_STEP_MAX = 32       # requests up to which reading the gate weights per eight of them beats the batched product
+
+
+def lru_step(out: torch.Tensor, packed: torch.Tensor, y_off: int, x_off: int, bias_y, bias_x, conv_w, conv_b, gates: torch.Tensor, bias_r, bias_i,
+             neg_softplus, state, cu_seqlens, state_slots, positions, num_seqs: int) -> torch.Tensor:
+    """A step of one token per request: convolution, both gate products, the recurrence, the output gate and the ring in one kernel."""
+    W = out.shape[1]
+    parts, two, part = gates.shape
+    taps = conv_w.shape[0]
+    _cuda(out, packed, bias_y, bias_x, conv_w, conv_b, gates, bias_r, bias_i, neg_softplus, state, cu_seqlens, state_slots, positions)
+    _contig(out, gates)
+    _lru_check(packed, W, parts, y_off, x_off, tuple((v, W) for v in (bias_y, bias_x, conv_b, bias_r, bias_i, neg_softplus)) + ((conv_w, taps * W),),
+               (cu_seqlens, state_slots, positions))
+    sp, sf, n_slots = _state_args(state)
+    if out.dtype != packed.dtype or gates.dtype != out.dtype or two != 2 * part or parts * part != W or out.shape[0] < num_seqs:
+        raise KernelError("lru_step: out [S, W], gates [parts, 2 * part, part] of packed's element type")
+    _check(_lru_lib().cvb_lru_step(
+        _ptr(out), _ptr(packed), _ptr(bias_y), _ptr(bias_x), _ptr(conv_w), _ptr(conv_b), _ptr(gates), _ptr(bias_r), _ptr(bias_i),
+        _ptr(neg_softplus), sp, sf, c_int(n_slots), _ptr(cu_seqlens), _ptr(state_slots), _ptr(positions), c_int(num_seqs), c_int(W), c_int(parts),
+        c_int(taps), c_int(packed.stride(0)), c_int(y_off), c_int(x_off), c_int(dtype_code(packed.dtype)), _ptr(error_flag(out.device)),
+        _stream()), "lru_step")
     return out
 
 
@@ -786,11 +972,13 @@ def _moe_lib():
 
 def route_topk(ids: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router: torch.Tensor,
                bias: Optional[torch.Tensor], over_all: bool = False, scale: float = 1.0,
-               extra_out: Optional[torch.Tensor] = None, logistic: bool = False) -> None:
+               extra_out: Optional[torch.Tensor] = None, logistic: bool = False, groups: int = 0, keep: int = 0) -> None:
     """ids, weights [T, top]: the `top` largest of x @ router^T + bias (float32 arithmetic) and the softmax over them; with
     `over_all` the weights are `scale` times the winners' shares of the softmax over ALL experts instead.  `extra_out`
     float32 [T, n]: the last n rows of `router` are not experts, their products with x leave there unchanged.  `logistic`: the
-    weights are `scale` times the winners' own sigmoid(z), with no sum over experts."""
+    weights are `scale` times the winners' own sigmoid(z), with no sum over experts.  `groups` > 0: scores are the softmax over all
+    outputs, the choice goes by score + bias inside the `keep` groups with the largest such sum, and the weights are the
+    chosen scores (without bias) over their sum."""
     _cuda(ids, weights, x, router, bias, extra_out); _contig(ids, weights, x, router, bias, extra_out)
     T, D = x.shape
     extra = 0 if extra_out is None else extra_out.shape[1]
@@ -802,19 +990,34 @@ def route_topk(ids: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router
             or ids.shape != (T, top) or weights.shape != (T, top) or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != E))):
         raise KernelError("route_topk: ids int32 and weights float32 [T, top]; router float32 [E, D]; bias float32 [E]")
     _check(_moe_lib().cvb_route_topk(_ptr(ids), _ptr(weights), _ptr(x), _ptr(router), _ptr(bias), c_int(T), c_int(D), c_int(E),
-                                     c_int(top), c_int(2 if logistic else (1 if over_all else 0)), c_float(scale), c_int(extra), _ptr(extra_out),
+                                     c_int(top), c_int(3 if groups else (2 if logistic else (1 if over_all else 0))), c_float(scale), c_int(extra), _ptr(extra_out),
+                                     c_int(groups), c_int(keep),
                                      c_int(dtype_code(x.dtype)), _stream()), "route_topk")
 
 
+EXPERT_ACTS = {"relu2": 0, "silu": 1, "clamped": 2}
+
+
+def _expert_gated(activation: str, identity: int, weight_on_input: bool) -> bool:
+    if activation not in EXPERT_ACTS:
+        raise KernelError(f"experts: activation '{activation}' is not built; built: {sorted(EXPERT_ACTS)}")
+    if identity and weight_on_input:
+        raise KernelError("experts: an identity expert takes its weight on the output")
+    return activation != "relu2"
+
+
 def expert_rows(y: torch.Tensor, hid: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                w_gate_up: torch.Tensor, w_down: torch.Tensor, gated: bool = True, weight_on_input: bool = False) -> torch.Tensor:
+                w_gate_up: torch.Tensor, w_down: torch.Tensor, activation: str = "silu", weight_on_input: bool = False, identity: int = 0,
+                limit: float = 0.0, alpha: float = 1.702) -> torch.Tensor:
     """y[t] = sum_k weights[t, k] * down_e(silu(gate_e x) * up_e x), e = ids[t, k]; w_gate_up [E, 2 ff, D], w_down [E, D, ff];
     with `weight_on_input` y[t] = sum_k expert_e(weights[t, k] * x) instead;
     `hid` [T * top, ff] is scratch.  Two kernels that read only the chosen experts' weights: for a few tokens, and for
-    float32.  `gated=False`: an expert is down_e(relu(up_e x)^2) and w_gate_up holds [E, ff, D]."""
+    float32.  `activation` = "relu2": an expert is down_e(relu(up_e x)^2) and w_gate_up holds [E, ff, D]; "clamped": gated with
+    g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit).  Ids E .. E + identity - 1 stand for the input itself."""
     _cuda(y, hid, x, ids, weights, w_gate_up, w_down); _contig(y, hid, x, ids, weights, w_gate_up, w_down)
     T, D = x.shape
     E, F2, _ = w_gate_up.shape
+    gated = _expert_gated(activation, identity, weight_on_input)
     F = F2 // 2 if gated else F2
     top = ids.shape[1]
     if (y.shape != x.shape or y.dtype != x.dtype or w_gate_up.dtype != x.dtype or w_down.dtype != x.dtype or hid.dtype != x.dtype
@@ -823,8 +1026,8 @@ def expert_rows(y: torch.Tensor, hid: torch.Tensor, x: torch.Tensor, ids: torch.
         raise KernelError("expert_rows: x, y [T, D], hid [T * top, ff], w_gate_up [E, 2 ff, D] and w_down [E, D, ff] of one element "
                           "type; ids int32 and weights float32 [T, top]")
     _check(_moe_lib().cvb_expert_rows(_ptr(y), _ptr(hid), _ptr(x), _ptr(ids), _ptr(weights), _ptr(w_gate_up), _ptr(w_down), c_int(T),
-                                      c_int(D), c_int(F), c_int(E), c_int(top), c_int(1 if gated else 0), c_int(1 if weight_on_input else 0),
-                                      c_int(dtype_code(x.dtype)), _ptr(error_flag(x.device)), _stream()), "expert_rows", kernels=2)
+                                      c_int(D), c_int(F), c_int(E), c_int(top), c_int(EXPERT_ACTS[activation]), c_int(1 if weight_on_input else 0),
+                                      c_int(identity), c_float(limit), c_float(alpha), c_int(dtype_code(x.dtype)), _ptr(error_flag(x.device)), _stream()), "expert_rows", kernels=2)
     return y
 
 
@@ -839,7 +1042,8 @@ def grouped_rows_tcgen05(num_tokens: int, top: int, num_experts: int) -> int:
 
 
 def experts_grouped_tcgen05(y, x, ids, weights, w_gate_up, w_down, tile_expert, row_token, slot_of, xs, hid, rows,
-                            gated: bool = True, weight_on_input: bool = False) -> torch.Tensor:
+                            activation: str = "silu", weight_on_input: bool = False, identity: int = 0, limit: float = 0.0,
+                            alpha: float = 1.702) -> torch.Tensor:
     """More tokens on the tcgen05 tensor cores: the pairs are sorted by expert into segments that start on multiples of
     128 rows (device side), the tokens' rows are gathered into that order, and two grouped products (the first with the
     gated activation as its epilogue) run on csrc/gemm_tcgen05.cu's kernel; the last kernel adds a token's expert outputs
@@ -850,6 +1054,7 @@ def experts_grouped_tcgen05(y, x, ids, weights, w_gate_up, w_down, tile_expert, 
     _contig(y, x, ids, weights, w_gate_up, w_down, tile_expert, row_token, slot_of, xs, hid, rows)
     T, D = x.shape
     E, F2, _ = w_gate_up.shape
+    gated = _expert_gated(activation, identity, weight_on_input)
     F, top = (F2 // 2 if gated else F2), ids.shape[1]
     R = grouped_rows_tcgen05(T, top, E)
     bf = torch.bfloat16
@@ -865,7 +1070,7 @@ def experts_grouped_tcgen05(y, x, ids, weights, w_gate_up, w_down, tile_expert, 
     _gemm.cvb_gemm_grouped_bf16_tcgen05.restype = c_int
     err = _ptr(error_flag(x.device))
     _check(_moe_lib().cvb_sort_pairs_padded(_ptr(tile_expert), _ptr(row_token), _ptr(slot_of), _ptr(ids), c_int(T), c_int(E), c_int(top),
-                                            c_int(R // 128), err, _stream()), "sort_pairs_padded")
+                                            c_int(R // 128), c_int(identity), err, _stream()), "sort_pairs_padded")
     xs2, hid2, rows2 = xs.view(-1)[:R * D].view(R, D), hid.view(-1)[:R * F].view(R, F), rows.view(-1)[:R * D].view(R, D)
     if weight_on_input:     # a pair's weight scales its row on the way in; the rows behind a segment keep what they held (finite)
         _moe_lib().cvb_scatter_pairs_scaled_bf16.restype = c_int
@@ -875,17 +1080,18 @@ def experts_grouped_tcgen05(y, x, ids, weights, w_gate_up, w_down, tile_expert, 
         gather_rows(xs2, x, row_token.view(-1)[:R])
     if gated:
         _check(_gemm.cvb_gemm_grouped_bf16_tcgen05(_ptr(hid2), _ptr(xs2), _ptr(w_gate_up), _ptr(tile_expert), c_int(R), c_int(2 * F), c_int(E),
-                                                   c_int(D), c_int(1), c_int(256), err, _stream()), "gemm_grouped_bf16_tcgen05")
+                                                   c_int(D), c_int(4 if activation == "clamped" else 1), c_int(256), c_float(limit), c_float(alpha),
+                                                   err, _stream()), "gemm_grouped_bf16_tcgen05")
     else:           # the squared relu is the epilogue
         up_256 = (T * top // 128 + 1) * ((F + 255) // 256)
         _check(_gemm.cvb_gemm_grouped_bf16_tcgen05(_ptr(hid2), _ptr(xs2), _ptr(w_gate_up), _ptr(tile_expert), c_int(R), c_int(F), c_int(E),
-                                                   c_int(D), c_int(3), c_int(256 if up_256 >= 120 else 128), err, _stream()),
+                                                   c_int(D), c_int(3), c_int(256 if up_256 >= 120 else 128), c_float(0.0), c_float(0.0), err, _stream()),
                "gemm_grouped_bf16_tcgen05")
     tiles_256 = (T * top // 128 + 1) * ((D + 255) // 256)
     _check(_gemm.cvb_gemm_grouped_bf16_tcgen05(_ptr(rows2), _ptr(hid2), _ptr(w_down), _ptr(tile_expert), c_int(R), c_int(D), c_int(E),
-                                               c_int(F), c_int(0), c_int(256 if tiles_256 >= 120 else 128), err, _stream()),
+                                               c_int(F), c_int(0), c_int(256 if tiles_256 >= 120 else 128), c_float(0.0), c_float(0.0), err, _stream()),
            "gemm_grouped_bf16_tcgen05")
-    _check(_moe_lib().cvb_combine_pairs_bf16(_ptr(y), _ptr(rows2), _ptr(slot_of), _ptr(None if weight_on_input else weights), c_int(T),
+    _check(_moe_lib().cvb_combine_pairs_bf16(_ptr(y), _ptr(rows2), _ptr(x), _ptr(slot_of), _ptr(None if weight_on_input else weights), c_int(T),
                                              c_int(D), c_int(top), _stream()),
            "combine_pairs")
     return y
@@ -901,14 +1107,15 @@ def grouped_experts_preferred(num_pairs: int, num_experts: int, expert_bytes: in
             or (num_pairs >= 3 and expert_bytes >= (64 << 20)))
 
 
-def routed_experts(y, x, ids, weights, w_gate_up, w_down, workspace=None, kernel: str = "", gated: bool = True,
-                   weight_on_input: bool = False) -> torch.Tensor:
+def routed_experts(y, x, ids, weights, w_gate_up, w_down, workspace=None, kernel: str = "", activation: str = "silu",
+                   weight_on_input: bool = False, identity: int = 0, limit: float = 0.0, alpha: float = 1.702) -> torch.Tensor:
     """The experts' outputs added up with the router's weights, by the kernels that suit the step: one or two tokens (and
     float32, and sizes that are no multiples of 8) read the chosen experts' weights pair by pair; more go through the
     grouped tcgen05 products (see grouped_experts_preferred).  `workspace` (parts.base.Workspace) lends the scratch;
     without it the scratch is allocated.  `kernel` = "rows" | "tcgen05" fixes the choice (where the shape allows it)."""
     T, D = x.shape
     E, F2, _ = w_gate_up.shape
+    gated = _expert_gated(activation, identity, weight_on_input)
     F, top = (F2 // 2 if gated else F2), ids.shape[1]
     expert_bytes = (3 if gated else 2) * D * F * x.element_size()
     grouped = kernel == "tcgen05" or (kernel == "" and grouped_experts_preferred(T * top, E, expert_bytes))
@@ -923,13 +1130,14 @@ def routed_experts(y, x, ids, weights, w_gate_up, w_down, workspace=None, kernel
         slot_of = workspace.rows("moe_slot_of", T, top, torch.int32) if workspace is not None else torch.empty(T * top, dtype=torch.int32, device=x.device)
         return experts_grouped_tcgen05(y, x, ids, weights, w_gate_up, w_down, buf("moe_tile_expert", R, torch.int32),
                                        buf("moe_row_token", R, torch.int32), slot_of, buf(f"moe_xs{D}", R * D, x.dtype),
-                                       buf(f"moe_hid{F}", R * F, x.dtype), buf(f"moe_rows{D}", R * D, x.dtype), gated=gated,
-                                       weight_on_input=weight_on_input)
+                                       buf(f"moe_hid{F}", R * F, x.dtype), buf(f"moe_rows{D}", R * D, x.dtype), activation=activation,
+                                       weight_on_input=weight_on_input, identity=identity, limit=limit, alpha=alpha)
     if workspace is not None:
         hid = workspace.rows("moe_hidden", T, top * F, x.dtype)
     else:
         hid = torch.empty((T, top * F), dtype=x.dtype, device=x.device)
-    return expert_rows(y, hid, x, ids, weights, w_gate_up, w_down, gated=gated, weight_on_input=weight_on_input)
+    return expert_rows(y, hid, x, ids, weights, w_gate_up, w_down, activation=activation, weight_on_input=weight_on_input,
+                       identity=identity, limit=limit, alpha=alpha)
 
 
 # ---- several residual streams read and written through learned weights (csrc/hyper.cu) ------------------------------------
@@ -1014,16 +1222,19 @@ def masked_qkv_prep(q_out: torch.Tensor, packed: torch.Tensor, num_heads: int, n
                     positions: Optional[torch.Tensor] = None, pages: Optional[torch.Tensor] = None,
                     slots: Optional[torch.Tensor] = None, page_size: int = 1, planes: int = 1,
                     v_first_out: Optional[torch.Tensor] = None, v_first_in: Optional[torch.Tensor] = None,
-                    lam: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """From rows [q: H dim | k: G dim | v: G vdim] of `packed`: q_out [T, H, dim] = turn(norm(q)); the entry [turn(norm(k)) | v']
+                    lam: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """From rows [q: H dim | k: G dim | v: G vdim] of `packed` (a column range of wider rows will do), plus `bias` (float32, the same
+    layout; None: none): q_out [T, H, dim] = turn(norm(q)); the entry [turn(norm(k)) | v']
     of every kv head into the token's cache slot of `pages` ([page, planes, G, slot, dim + vdim], plane 0), with
     v' = (1 - lam) v + lam v_first_in (v itself without v_first_in); `v_first_out` [T, G * vdim] receives v as projected."""
-    _cuda(q_out, packed, q_weight, k_weight, cos, sin, positions, pages, slots, v_first_out, v_first_in, lam)
-    _contig(q_out, packed, q_weight, k_weight, cos, sin, positions, pages, slots, v_first_out, v_first_in, lam)
+    _cuda(q_out, packed, q_weight, k_weight, cos, sin, positions, pages, slots, v_first_out, v_first_in, lam, bias)
+    _contig(q_out, q_weight, k_weight, cos, sin, positions, pages, slots, v_first_out, v_first_in, lam, bias)
     T = packed.shape[0]
     H, G = num_heads, num_kv_heads
-    if q_out.dtype != packed.dtype or q_out.numel() != T * H * dim or packed.shape[1] < H * dim + G * (dim + vdim):
+    if q_out.dtype != packed.dtype or q_out.numel() != T * H * dim or packed.shape[1] < H * dim + G * (dim + vdim) or packed.stride(1) != 1:
         raise KernelError("masked_qkv_prep: packed [T, H dim + G (dim + vdim)] and q_out [T, H, dim] of one element type")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != H * dim + G * (dim + vdim)):
+        raise KernelError("masked_qkv_prep: bias float32 [H dim + G (dim + vdim)]")
     for w in (q_weight, k_weight):
         if w is not None and (w.dtype != torch.float32 or w.numel() != dim):
             raise KernelError("masked_qkv_prep: norm weights are float32 [dim]")
@@ -1045,7 +1256,7 @@ def masked_qkv_prep(q_out: torch.Tensor, packed: torch.Tensor, num_heads: int, n
             raise KernelError("masked_qkv_prep: positions and slots are int32 [T]")
     total_slots = pages.numel() // (planes * G * (dim + vdim)) if pages is not None else 0
     _check(_attn_masked_lib().cvb_masked_qkv_prep(
-        _ptr(q_out), _ptr(packed), c_int(T), c_int(packed.shape[1]), _ptr(q_weight), _ptr(k_weight), _ptr(cos if rot else None),
+        _ptr(q_out), _ptr(packed), c_int(T), c_int(packed.stride(0)), _ptr(bias), _ptr(q_weight), _ptr(k_weight), _ptr(cos if rot else None),
         _ptr(sin if rot else None), _ptr(positions), _ptr(slots), _ptr(pages), _ptr(v_first_out), _ptr(v_first_in), _ptr(lam),
         c_int(H), c_int(G), c_int(dim), c_int(vdim), c_int(rot), c_int(1 if interleaved else 0), c_int(planes), c_int(page_size),
         c_int(max_pos), c_float(eps), c_int64(total_slots), c_int(dtype_code(packed.dtype)), _ptr(error_flag(packed.device)),
@@ -1071,28 +1282,31 @@ def attn_masked_general(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor,
                         seq_of_token: torch.Tensor, positions: torch.Tensor, num_tokens: int, num_heads: int, num_kv_heads: int,
                         dim: int, vdim: int, page_size: int, scale: float, planes: int = 1, chunk: int = 0, window: int = 0,
                         pool: int = 0, softcap: float = 0.0, r1: Optional[torch.Tensor] = None, r2: Optional[torch.Tensor] = None,
-                        sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out [T, H, vdim]: one block per (token, query head), any sizes, float32 or bf16 (see csrc/attention_masked.cu).
-    `gate` [T, H] (a view with unit column stride): the head's output is multiplied by sigmoid(gate[t, h])."""
+                        sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
+    """out [T, H * vdim] (a column range of wider rows will do): one block per (token, query head), any sizes, float32 or bf16 (see csrc/attention_masked.cu).
+    `gate` [T, H] (a view with unit column stride): the head's output is multiplied by sigmoid(gate[t, h]); a gate of H * vdim columns
+    gates every element by itself.  `out_scale` multiplies the output."""
     _cuda(out, q, pages, block_tables, seq_of_token, positions, r1, r2, sink, gate)
-    _contig(out, q, pages, block_tables, seq_of_token, positions, r1, r2, sink)
+    _contig(q, pages, block_tables, seq_of_token, positions, r1, r2, sink)
     T, H, G = num_tokens, num_heads, num_kv_heads
-    if q.dtype != pages.dtype or out.dtype != q.dtype or q.numel() < T * H * dim or out.numel() < T * H * vdim:
+    if (q.dtype != pages.dtype or out.dtype != q.dtype or q.numel() < T * H * dim or out.dim() != 2 or out.shape[0] < T
+            or out.shape[1] != H * vdim or out.stride(1) != 1):
         raise KernelError("attn_masked: q [T, H, dim], out [T, H, vdim] and the pages share one element type")
     if block_tables.dtype != torch.int32 or block_tables.dim() != 2 or seq_of_token.dtype != torch.int32 or positions.dtype != torch.int32:
         raise KernelError("attn_masked: block_tables int32 [S, W]; seq_of_token and positions int32")
     for t in (r1, r2, sink):
         if t is not None and (t.dtype != torch.float32 or t.numel() != H):
             raise KernelError("attn_masked: r1, r2 and sink are float32 [H]")
-    if gate is not None and (gate.dtype != q.dtype or gate.shape[1] != H or gate.stride(1) != 1 or gate.shape[0] < T):
-        raise KernelError("attn_masked: gate [T, H] of the queries' element type")
+    if gate is not None and (gate.dtype != q.dtype or gate.shape[1] not in (H, H * vdim) or gate.stride(1) != 1 or gate.shape[0] < T):
+        raise KernelError("attn_masked: gate [T, H] or [T, H * vdim] of the queries' element type")
+    per_element = gate is not None and gate.shape[1] != H
     num_pages = pages.numel() // (planes * G * page_size * (dim + vdim))
     _check(_attn_masked_lib().cvb_attn_masked_general(
         _ptr(out), _ptr(q), _ptr(pages), _ptr(block_tables), c_int(block_tables.shape[1]), _ptr(seq_of_token), _ptr(positions),
         c_int(T), c_int(H), c_int(G), c_int(dim), c_int(vdim), c_int(page_size), c_int(planes), c_int(chunk), c_int(window),
         c_int(pool), c_float(scale), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate),
-        c_int(gate.stride(0) if gate is not None else 0), c_int(num_pages), c_int(dtype_code(q.dtype)),
-        _ptr(error_flag(q.device)), _stream()), "attn_masked_general")
+        c_int(gate.stride(0) if gate is not None else 0), c_int(1 if per_element else 0), c_float(out_scale), c_int(out.stride(0)),
+        c_int(num_pages), c_int(dtype_code(q.dtype)), _ptr(error_flag(q.device)), _stream()), "attn_masked_general")
     return out
 
 
@@ -1102,6 +1316,12 @@ def attn_masked_supported(dtype: torch.dtype, num_heads: int, num_kv_heads: int,
     of 16, up to 64 query heads per kv head."""
     return (dtype == torch.bfloat16 and dim % 16 == 0 and 16 <= dim <= 128 and vdim % 16 == 0 and 16 <= vdim <= 128
             and num_kv_heads > 0 and num_heads % num_kv_heads == 0 and num_heads // num_kv_heads <= 64)
+
+
+def attn_masked_pairs(out: torch.Tensor, gate: Optional[torch.Tensor], num_heads: int) -> bool:
+    """Whether rows of the output (and of a gate per element) start on the pairs of elements the tensor-core kernel handles."""
+    even = lambda t: t.stride(0) % 2 == 0 and t.data_ptr() % 4 == 0          # noqa: E731
+    return even(out) and (gate is None or gate.shape[1] == num_heads or even(gate))
 
 
 def attn_masked_decode_splits(num_seqs: int, num_kv_heads: int, visible_keys: int, sms: int = 148) -> int:
@@ -1121,13 +1341,13 @@ def attn_masked_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, bl
                      page_size: int, scale: float, planes: int = 1, chunk: int = 0, window: int = 0, pool: int = 0,
                      softcap: float = 0.0, r1: Optional[torch.Tensor] = None, r2: Optional[torch.Tensor] = None,
                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, all_single: bool = False,
-                     splits: int = 1, scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     splits: int = 1, scratch: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
     """The tensor-core form of attn_masked_general for prompt portions and decoded tokens alike; `num_tiles` as
     attn_keys_tiles gives it (blocks of 64 // group tokens of one request).  `all_single`: every request brings exactly one
     token (the form for decoded tokens, up to 16 query heads per kv head); with `splits` > 1 that many blocks share a
     (request, kv head), through `scratch` (float32, attn_keys_scratch_floats with vdim as the head size) and a merge kernel."""
     _cuda(out, q, pages, block_tables, cu_seqlens, positions, r1, r2, sink, gate)
-    _contig(out, q, pages, block_tables, cu_seqlens, positions, r1, r2, sink)
+    _contig(q, pages, block_tables, cu_seqlens, positions, r1, r2, sink)
     H = num_heads
     if q.dtype != torch.bfloat16 or pages.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("attn_masked_bf16 takes bf16 queries, pages and output")
@@ -1136,8 +1356,11 @@ def attn_masked_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, bl
     for t in (r1, r2, sink):
         if t is not None and (t.dtype != torch.float32 or t.numel() != H):
             raise KernelError("attn_masked_bf16: r1, r2 and sink are float32 [H]")
-    if gate is not None and (gate.dtype != torch.bfloat16 or gate.shape[1] != H or gate.stride(1) != 1):
-        raise KernelError("attn_masked_bf16: gate bf16 [T, H]")
+    if out.dim() != 2 or out.shape[1] != H * vdim or out.stride(1) != 1:
+        raise KernelError("attn_masked_bf16: out bf16 [T, H * vdim]")
+    if gate is not None and (gate.dtype != torch.bfloat16 or gate.shape[1] not in (H, H * vdim) or gate.stride(1) != 1):
+        raise KernelError("attn_masked_bf16: gate bf16 [T, H] or [T, H * vdim]")
+    per_element = gate is not None and gate.shape[1] != H
     num_pages = pages.numel() // (planes * num_kv_heads * page_size * (dim + vdim))
     if splits > 1 and (scratch is None or scratch.dtype != torch.float32 or not scratch.is_cuda or not scratch.is_contiguous()):
         raise KernelError("attn_masked_bf16: splits need a contiguous float32 CUDA scratch")
@@ -1145,7 +1368,8 @@ def attn_masked_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, bl
         _ptr(out), _ptr(q), _ptr(pages), _ptr(block_tables), c_int(block_tables.shape[1]), _ptr(cu_seqlens), _ptr(positions),
         c_int(num_seqs), c_int(num_tiles), c_int(H), c_int(num_kv_heads), c_int(dim), c_int(vdim), c_int(page_size), c_int(planes),
         c_int(chunk), c_int(window), c_int(pool), c_float(scale), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate),
-        c_int(gate.stride(0) if gate is not None else 0), c_int(num_pages), c_int(1 if all_single else 0), c_int(splits), _ptr(scratch),
+        c_int(gate.stride(0) if gate is not None else 0), c_int(1 if per_element else 0), c_float(out_scale), c_int(out.stride(0)),
+        c_int(num_pages), c_int(1 if all_single else 0), c_int(splits), _ptr(scratch),
         c_int64(scratch.numel() if scratch is not None else 0), _ptr(error_flag(q.device)), _stream()), "attn_masked_bf16",
         kernels=2 if all_single and splits > 1 else 1)
     return out
@@ -1691,9 +1915,9 @@ def gemm_tcgen05_supported(x_dtype: torch.dtype, weight: torch.Tensor, swiglu: b
 
 
 def gemm_bf16_tcgen05(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, swiglu: bool = False, tile_n: int = 0,
-                      resid: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      resid: Optional[torch.Tensor] = None, geglu: bool = False) -> torch.Tensor:
     """out = x @ weight^T on the tcgen05 tensor cores; with `swiglu`, weight holds gate rows over up rows and
-    out = silu(x @ gate^T) * (x @ up^T); with `resid` (which may be `out`), out = round(x @ weight^T) + resid.
+    out = silu(x @ gate^T) * (x @ up^T); `geglu`: the same with gelu_tanh for silu; with `resid` (which may be `out`), out = round(x @ weight^T) + resid.
     `tile_n` (128 or 256) picks the tile width; 0 chooses by the number of tiles it gives."""
     global _gemm
     if _gemm is None:
@@ -1703,9 +1927,10 @@ def gemm_bf16_tcgen05(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, 
     _cuda(out, x, weight, resid); _contig(out, x, weight, resid)
     M, K = x.shape
     N = weight.shape[0]
-    n_out = N // 2 if swiglu else N
+    gated = swiglu or geglu
+    n_out = N // 2 if gated else N
     if x.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or weight.shape[1] != K \
-            or out.shape != (M, n_out) or (swiglu and resid is not None) \
+            or out.shape != (M, n_out) or (gated and resid is not None) or (swiglu and geglu) \
             or (resid is not None and (resid.dtype != torch.bfloat16 or resid.shape != out.shape)):
         raise KernelError("gemm_bf16_tcgen05: x [M, K], weight [N, K], out [M, N] (or [M, N / 2] with swiglu), resid like out, "
                           "all bf16")
@@ -1713,7 +1938,7 @@ def gemm_bf16_tcgen05(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, 
         # tiles of 256 columns halve the traffic of A; take them when they still fill the SMs
         tiles_256 = ((M + 127) // 128) * ((N + 255) // 256)
         tile_n = 256 if tiles_256 >= 120 else 128
-    mode = 1 if swiglu else (2 if resid is not None else 0)
+    mode = 1 if swiglu else (5 if geglu else (2 if resid is not None else 0))
     _check(_gemm.cvb_gemm_bf16_tcgen05(_ptr(out), _ptr(x), _ptr(weight), _ptr(resid), c_int(M), c_int(N), c_int(K), c_int(mode),
                                        c_int(tile_n), _ptr(error_flag(x.device)), _stream()), "gemm_bf16_tcgen05")
     return out

@@ -11,7 +11,8 @@
 //                     new row is still on the chip.  With a history it also replaces the request's convolution history by the
 //                     last K - 1 rows of `a` (the block of a request's first token does that; the convolution that read the
 //                     history ran in an earlier kernel).
-//   glu_clamped     : g = min(gu[t, i], L), u = clamp(gu[t, I + i], -L, L);  out = T( g * sigmoid(alpha g) * (u + 1) )
+//   glu_act         : act 0: g = min(gu[t, i], L), u = clamp(gu[t, I + i], -L, L);  out = T( g * sigmoid(alpha g) * (u + 1) )
+//                     act 1: out = T( gelu_tanh(gu[t, i]) * gu[t, I + i] )
 //   add_gated_rows  : y[t, :] = T( y[t, :] + sigmoid(z[t]) * s[t, :] )   (a shared expert joins the routed ones through one
 //                     gate per token)
 //   wide_qk_prep    : q[t, :] = T( q / sqrt(mean(q^2) + eps) * wq * (1 + coef * ln(floor((p + 1) / every) + 1)) ) over the WHOLE
@@ -153,23 +154,32 @@ gated_norm_add_kernel(float* __restrict__ h, const T* __restrict__ y, const T* _
     }
 }
 
-template <typename T>
-__global__ void glu_clamped_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n, int I, float limit, float alpha) {
+template <int ACT>
+__device__ __forceinline__ float glu_of(float g, float u, float limit, float alpha) {
+    if constexpr (ACT == 0) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g * sigmoid_f(alpha * g) * (u + 1.f);
+    } else {
+        return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    }
+}
+
+template <typename T, int ACT>
+__global__ void glu_act_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n, int I, float limit, float alpha) {
     pdl_trigger();
     pdl_wait();
     for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
          i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
         const int64_t t = i / I;
         const int c = static_cast<int>(i - t * I);
-        const float g = fminf(to_float(gu[t * 2 * I + c]), limit);
-        const float u = fminf(fmaxf(to_float(gu[t * 2 * I + I + c]), -limit), limit);
-        out[i] = from_float<T>(g * sigmoid_f(alpha * g) * (u + 1.f));
+        out[i] = from_float<T>(glu_of<ACT>(to_float(gu[t * 2 * I + c]), to_float(gu[t * 2 * I + I + c]), limit, alpha));
     }
 }
 
 // 16 bytes of gate and of up per thread: I is a multiple of the chunk and all rows start on 16 bytes
-template <typename T>
-__global__ void glu_clamped_vec_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n_chunks, int I, float limit, float alpha) {
+template <typename T, int ACT>
+__global__ void glu_act_vec_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n_chunks, int I, float limit, float alpha) {
     pdl_trigger();
     pdl_wait();
     constexpr int N = 16 / sizeof(T);
@@ -182,11 +192,7 @@ __global__ void glu_clamped_vec_kernel(T* __restrict__ out, const T* __restrict_
     *reinterpret_cast<uint4*>(g) = *reinterpret_cast<const uint4*>(gu + t * 2 * I + c);
     *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(gu + t * 2 * I + I + c);
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-        const float gi = fminf(to_float(g[i]), limit);
-        const float ui = fminf(fmaxf(to_float(u[i]), -limit), limit);
-        o[i] = from_float<T>(gi * sigmoid_f(alpha * gi) * (ui + 1.f));
-    }
+    for (int i = 0; i < N; ++i) o[i] = from_float<T>(glu_of<ACT>(to_float(g[i]), to_float(u[i]), limit, alpha));
     *reinterpret_cast<uint4*>(out + t * I + c) = *reinterpret_cast<const uint4*>(o);
 }
 
@@ -287,21 +293,25 @@ extern "C" int cvb_gated_norm_add(float* h, const void* y, const void* z, const 
     return launch_status();
 }
 
-extern "C" int cvb_glu_clamped(void* out, const void* gate_up, int T, int I, float limit, float alpha, int dtype, cudaStream_t stream) {
+extern "C" int cvb_glu_act(void* out, const void* gate_up, int T, int I, int act, float limit, float alpha, int dtype, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
     if (T < 0 || I <= 0) return CVB_E_SIZE;
+    if (act < 0 || act > 1) return CVB_E_SHAPE;
     const int64_t n = static_cast<int64_t>(T) * I, want = (n + 255) / 256;
     const unsigned blocks = static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16);
     const bool aligned = ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(gate_up)) & 15) == 0;
-#define CALL(TY)                                                                                                                          \
+#define CALL_ACT(TY, ACT)                                                                                                                 \
     if (aligned && I % (16 / (int)sizeof(TY)) == 0) {                                                                                     \
         const int64_t nc = n / (16 / (int)sizeof(TY));                                                                                    \
-        launch_kernel(glu_clamped_vec_kernel<TY>, dim3(static_cast<unsigned>((nc + 255) / 256)), dim3(256), 0, stream, (TY*)out,          \
+        launch_kernel(glu_act_vec_kernel<TY, ACT>, dim3(static_cast<unsigned>((nc + 255) / 256)), dim3(256), 0, stream, (TY*)out,         \
                       (const TY*)gate_up, nc, I, limit, alpha);                                                                           \
     } else                                                                                                                                \
-        launch_kernel(glu_clamped_kernel<TY>, dim3(blocks), dim3(256), 0, stream, (TY*)out, (const TY*)gate_up, n, I, limit, alpha)
+        launch_kernel(glu_act_kernel<TY, ACT>, dim3(blocks), dim3(256), 0, stream, (TY*)out, (const TY*)gate_up, n, I, limit, alpha)
+#define CALL(TY)                                                                                                                          \
+    if (act == 0) { CALL_ACT(TY, 0); } else { CALL_ACT(TY, 1); }
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
+#undef CALL_ACT
     return launch_status();
 }
 

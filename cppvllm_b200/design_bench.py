@@ -655,7 +655,7 @@ def lorulix_kernel_pairs(s, pk):
     w_up, w_dn = rnd(EXPERTS, F, D, scale=0.02), rnd(EXPERTS, D, F, scale=0.02)
     w_gu = rnd(EXPERTS, 2 * F, D, scale=0.02)
     y = torch.empty(T, D, dtype=bf, device=d)
-    new = _us(lambda i: ops.routed_experts(y, x, ids, wts, w_up, w_dn, workspace=ws, gated=False))
+    new = _us(lambda i: ops.routed_experts(y, x, ids, wts, w_up, w_dn, workspace=ws, activation="relu2"))
     like = _us(lambda i: ops.routed_experts(y, x, ids2, wts2, w_gu, w_dn, workspace=ws))
     pair("experts_2048_tokens", new, 2.0 * T * TOP * 2 * D * F, like, 2.0 * T * TOP * 3 * D * F, "flops", "Givirax gated experts")
     ws8 = Workspace(d, 8)
@@ -665,7 +665,7 @@ def lorulix_kernel_pairs(s, pk):
     dns = [w_dn] + [rnd(EXPERTS, D, F, scale=0.02) for _ in range(copies - 1)]
     x8, y8 = x[:8].contiguous(), torch.empty(8, D, dtype=bf, device=d)
     ids8, wts8, ids28, wts28 = ids[:8].contiguous(), wts[:8].contiguous(), ids2[:8].contiguous(), wts2[:8].contiguous()
-    new = _us(lambda i: ops.routed_experts(y8, x8, ids8, wts8, ups[i % copies], dns[i % copies], workspace=ws8, gated=False))
+    new = _us(lambda i: ops.routed_experts(y8, x8, ids8, wts8, ups[i % copies], dns[i % copies], workspace=ws8, activation="relu2"))
     like = _us(lambda i: ops.routed_experts(y8, x8, ids28, wts28, gus[i % copies], dns[i % copies], workspace=ws8))
     used, used2 = len(set(ids8.flatten().tolist())), len(set(ids28.flatten().tolist()))
     pair("experts_8_decoded_tokens", new, used * 2.0 * D * F * 2, like, used2 * 3.0 * D * F * 2, "bytes", "Givirax gated experts")

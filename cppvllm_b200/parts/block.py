@@ -5,7 +5,8 @@
 The reference fuses every residual add with the norm that follows it (kernels/fused_ops.cu:70-87,
 model_architecture.cpp:180,187).  The block keeps that fusion without knowing its neighbours: it receives the
 residual stream `h` together with a `pending` delta that has not been added yet, folds it into its first
-norm, and hands its own feed-forward output on as the next pending delta."""
+norm, and hands its own feed-forward output on as the next pending delta.  A layer may have no feed-forward: its mixer's
+output is then what it hands on."""
 from __future__ import annotations
 
 
@@ -17,12 +18,12 @@ from .base import Block, build_part, register_part
 class PreNormBlock(Block):
     def __init__(self, runtime, prefix="", names=None, *, mixer, ffn, mixer_norm, ffn_norm):
         super().__init__(runtime, prefix, names)
-        if ffn is None or ffn_norm is None:
-            raise ValueError("a pre-norm block needs a feed-forward and a norm in front of it")
+        if (ffn is None) != (ffn_norm is None):
+            raise ValueError("a feed-forward and the norm in front of it come together")
         self.mixer, self.ffn, self.mixer_norm, self.ffn_norm = mixer, ffn, mixer_norm, ffn_norm
 
     def parts(self):
-        return (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn)
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
 
     def forward(self, h, pending, ctx, cache, state):
         # A part may offer to take the norm in front of it (and the residual add in front of that) into its own
@@ -39,6 +40,8 @@ class PreNormBlock(Block):
         else:
             x = self.mixer_norm.forward(h) if pending is None else self.mixer_norm.add_forward(h, pending)
             a = self.mixer.forward(x, ctx, cache, state)
+        if self.ffn is None:
+            return h, a
         fuse = getattr(self.ffn, "can_fuse_norm", None)
         if fuse is not None and fuse(self.ffn_norm, ctx):
             m, h = self.ffn.forward_fused(h, a, self.ffn_norm, ctx, ws.other_of_pair("residual", h, T, D, h.dtype) if a is not None else None)

@@ -1,5 +1,11 @@
-"""Dense gated feed-forward (reference model/model_architecture.cpp:106-112,182-185; kernels/fused_ops.cu:210-220):
-gu = x Wgu^T with Wgu = rows(gate_proj) over rows(up_proj); act = T( rnd(silu(g)) * u ); y = act Wdown^T; no biases."""
+"""Dense gated feed-forwards.
+
+``swiglu`` (reference model/model_architecture.cpp:106-112,182-185; kernels/fused_ops.cu:210-220):
+gu = x Wgu^T with Wgu = rows(gate_proj) over rows(up_proj); act = T( rnd(silu(g)) * u ); y = act Wdown^T; no biases.
+
+``gated_mlp``: y = Wdown (act(Wgate x) * (Wup x)), act = "gelu_tanh" (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))); tensors
+``gate|up|down`` (the names are parameters), no biases.  Prompt portions that fill the SMs take the product whose tcgen05 epilogue is
+the gated activation."""
 from __future__ import annotations
 
 from typing import Dict
@@ -75,3 +81,44 @@ class SwiGLUMLP(FeedForward):
             ops.gemv_stream_bf16(h_new, act, self.w_down, T, add_to=h_new)              # h <- rnd(h + rnd(act Wdown^T)), in place
             return None, h_new
         return self._down(act, T), h_new
+
+
+@register_part("ffn", "gated_mlp")
+class GatedMLP(FeedForward):
+    def __init__(self, runtime, prefix="", names=None, *, hidden_size: int, intermediate_size: int, activation: str = "gelu_tanh",
+                 gate_name: str = "gate", up_name: str = "up", down_name: str = "down"):
+        super().__init__(runtime, prefix, names)
+        if activation != "gelu_tanh":
+            raise ValueError(f"activation '{activation}' is not built; built: gelu_tanh")
+        self.hidden_size, self.intermediate_size, self.activation = int(hidden_size), int(intermediate_size), activation
+        self.gate_name, self.up_name, self.down_name = gate_name, up_name, down_name
+        self.w_gate_up = self.w_down = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        D, I = self.hidden_size, self.intermediate_size
+        return {self.full_name(self.gate_name): WeightSpec((I, D)), self.full_name(self.up_name): WeightSpec((I, D)),
+                self.full_name(self.down_name): WeightSpec((D, I))}
+
+    def bind(self, tensors) -> None:
+        g, u = tensors[self.full_name(self.gate_name)], tensors[self.full_name(self.up_name)]
+        if g.dtype != u.dtype:
+            g, u = g.float(), u.float()
+        self.w_gate_up = torch.cat([g, u], dim=0).contiguous()
+        self.w_down = tensors[self.full_name(self.down_name)]
+
+    def weight_bytes(self) -> int:
+        return sum(w.numel() * w.element_size() for w in (self.w_gate_up, self.w_down))
+
+    def _project(self, x, w, out, rows):
+        return ops.linear(x, w, out=out) if self.rt.plain_kernels else ops.project_rows(x, w, out, rows)
+
+    def forward(self, x, ctx):
+        T = x.shape[0]
+        ws = self.rt.workspace
+        act = ws.rows("ffn_act", T, self.intermediate_size, x.dtype)
+        if not self.rt.plain_kernels and ops.gated_product_fused(x.dtype, self.w_gate_up, T):
+            ops.gemm_bf16_tcgen05(act, x, self.w_gate_up, geglu=True)        # gate and up never travel through memory
+        else:
+            gu = self._project(x, self.w_gate_up, ws.rows("ffn_gate_up", T, 2 * self.intermediate_size, x.dtype), T)
+            ops.geglu(act, gu)
+        return self._project(act, self.w_down, ws.rows("ffn_out", T, self.hidden_size, x.dtype), T)

@@ -25,15 +25,7 @@ class CausalLM:
         self.embedding = build_part("embedding", spec.embedding, runtime)
         self.blocks = []
         for ls in spec.layers:
-            mixer_extra = {}
-            mparams = dict(ls.mixer.params)
-            pos_name = mparams.pop("position", None)
-            mixer_cls = part_class("mixer", ls.mixer.kind)
-            if pos_name is not None:
-                if pos_name not in self.positions:
-                    raise ValueError(f"mixer names position encoding '{pos_name}', which the spec does not define")
-                mixer_extra["position"] = self.positions[pos_name]
-            mixer = mixer_cls(runtime, prefix=ls.mixer.prefix, names=dict(ls.mixer.names), **mparams, **mixer_extra)
+            mixer = self._build_mixer(ls.mixer)
             ffn = build_part("ffn", ls.ffn, runtime) if ls.ffn is not None else None
             mixer_norm = build_part("norm", ls.mixer_norm, runtime)
             ffn_norm = build_part("norm", ls.ffn_norm, runtime) if ls.ffn_norm is not None else None
@@ -45,6 +37,18 @@ class CausalLM:
         self.head = build_part("head", spec.lm_head, runtime)
         self.run_order: List[RunEntry] = spec.resolved_run_order()
         self._check_shared_caches()
+
+    def _build_mixer(self, spec):
+        """A mixer from its spec: a position encoding it names is handed over, and mixers it is made of (``members``) are built first."""
+        params = dict(spec.params)
+        pos_name = params.pop("position", None)
+        if pos_name is not None:
+            if pos_name not in self.positions:
+                raise ValueError(f"mixer names position encoding '{pos_name}', which the spec does not define")
+            params["position"] = self.positions[pos_name]
+        if "members" in params:
+            params["members"] = [self._build_mixer(m) for m in params["members"]]
+        return part_class("mixer", spec.kind)(self.rt, prefix=spec.prefix, names=dict(spec.names), **params)
 
     @property
     def capturable(self) -> bool:

@@ -12,7 +12,10 @@
   stay capturable.  Options: ``score = "sigmoid"``: the chosen experts' weights are their own sigmoid(z_e), not renormalised;
   ``weight_on_input``: the weight multiplies the expert's input, y = sum_e expert_e(w_e x); ``router_bias = False``: no bias
   tensor; ``shared_size`` > 0: a shared expert of the same gated form (``<prefix>shared.gate|up|down``) runs for every token
-  and is added.
+  and is added.  ``score = "softmax_all"``: s = softmax(z) over all router outputs, the choice goes by s (plus a ``correction`` tensor
+  that the weights do not see) among the outputs of the ``keep_groups`` best of ``groups`` equal groups of neighbours (a group counts
+  as its best output), and the weights are the chosen s over their sum + 1e-20.  ``identity`` > 0: that many router outputs behind
+  the experts' stand for the input itself.  ``activation = "clamped"``: experts of the form of ``clamped_glu`` below.
 * ``clamped_glu``: dense and gated with clamps: g = min(Wgate x, L), u = clamp(Wup x, -L, L); y = Wdown (g sigmoid(alpha g) (u + 1)).
 * ``routed_act``: a mixture of ungated experts Wdown act(Wup x) (act = relu2) whose weights are `scale` times the chosen experts'
   shares of the softmax over ALL experts (not renormalised over the winners); no router bias.  Optionally a shared expert of
@@ -81,14 +84,30 @@ class ActMLP(FeedForward):
 class RoutedGLU(FeedForward):
     def __init__(self, runtime, prefix="", names=None, *, hidden_size: int, intermediate_size: int, num_experts: int, top: int,
                  router_name: str = "router", router_bias_name: str = "router.b", expert_prefix: str = "e", score: str = "softmax",
-                 weight_on_input: bool = False, router_bias: bool = True, shared_size: int = 0, shared_prefix: str = "shared."):
+                 weight_on_input: bool = False, router_bias: bool = True, shared_size: int = 0, shared_prefix: str = "shared.",
+                 activation: str = "silu", limit: float = 0.0, alpha: float = 1.702, correction: bool = False,
+                 correction_name: str = "correction", groups: int = 1, keep_groups: int = 1, identity: int = 0):
         super().__init__(runtime, prefix, names)
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.num_experts, self.top = int(num_experts), int(top)
-        if not (0 < self.top <= self.num_experts):
-            raise ValueError(f"a token cannot use {self.top} of {self.num_experts} experts")
-        if score not in ("softmax", "sigmoid"):
-            raise ValueError(f"score is 'softmax' (over the chosen experts) or 'sigmoid', got {score!r}")
+        self.outputs = self.num_experts + int(identity)
+        if not (0 < self.top <= self.outputs):
+            raise ValueError(f"a token cannot use {self.top} of {self.outputs} experts")
+        if score not in ("softmax", "sigmoid", "softmax_all"):
+            raise ValueError(f"score is 'softmax' (over the chosen experts), 'sigmoid' or 'softmax_all', got {score!r}")
+        if score != "softmax_all" and (correction or int(groups) != 1 or int(identity)):
+            raise ValueError("a correction, groups and identity experts go with the score 'softmax_all'")
+        if score == "softmax_all" and router_bias:
+            raise ValueError("the score 'softmax_all' takes no router bias")
+        if self.outputs % int(groups) or not (0 < int(keep_groups) <= int(groups)) or self.top > int(keep_groups) * (self.outputs // int(groups)):
+            raise ValueError(f"{self.top} experts out of {keep_groups} of {groups} groups over {self.outputs} outputs")
+        if activation not in ("silu", "clamped"):
+            raise ValueError(f"activation '{activation}' is not built for gated experts; built: silu, clamped")
+        if activation == "clamped" and shared_size:
+            raise ValueError("a shared expert goes with silu")
+        self.activation, self.limit, self.alpha = activation, float(limit), float(alpha)
+        self.correction, self.correction_name = bool(correction), correction_name
+        self.groups, self.keep_groups, self.identity = int(groups), int(keep_groups), int(identity)
         self.router_name, self.router_bias_name, self.expert_prefix = router_name, router_bias_name, expert_prefix
         self.score, self.weight_on_input, self.router_bias = score, bool(weight_on_input), bool(router_bias)
         self.shared_size, self.shared_prefix = int(shared_size), shared_prefix
@@ -99,9 +118,11 @@ class RoutedGLU(FeedForward):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         D, I, E = self.hidden_size, self.intermediate_size, self.num_experts
-        specs = {self.full_name(self.router_name): WeightSpec((E, D), role="vector")}
+        specs = {self.full_name(self.router_name): WeightSpec((self.outputs, D), role="vector")}
         if self.router_bias:
             specs[self.full_name(self.router_bias_name)] = WeightSpec((E,), role="vector")
+        if self.correction:
+            specs[self.full_name(self.correction_name)] = WeightSpec((self.outputs,), role="vector")
         for e in range(E):
             specs[self._expert(e, "gate")] = WeightSpec((I, D))
             specs[self._expert(e, "up")] = WeightSpec((I, D))
@@ -117,6 +138,8 @@ class RoutedGLU(FeedForward):
         E = self.num_experts
         self.w_router = tensors[self.full_name(self.router_name)]
         self.b_router = tensors[self.full_name(self.router_bias_name)] if self.router_bias else None
+        if self.correction:
+            self.b_router = tensors[self.full_name(self.correction_name)]
         if self.shared_size:
             sp = self.shared_prefix
             g, u = tensors[self.full_name(sp + "gate")], tensors[self.full_name(sp + "up")]
@@ -132,7 +155,7 @@ class RoutedGLU(FeedForward):
         """What a decoded token reads: the router, `top` of the experts and the shared expert."""
         per_expert = (self.w_gate_up.numel() + self.w_down.numel()) * self.w_down.element_size() // self.num_experts
         shared = sum(w.numel() * w.element_size() for w in (self.shared_gate_up, self.shared_down)) if self.shared_size else 0
-        return self.w_router.numel() * 4 + (self.b_router.numel() * 4 if self.router_bias else 0) + self.top * per_expert + shared
+        return self.w_router.numel() * 4 + (self.b_router.numel() * 4 if self.b_router is not None else 0) + self.top * per_expert + shared
 
     def _project(self, x, w, out, rows):
         return ops.linear(x, w, out=out) if self.rt.plain_kernels else ops.project_rows(x, w, out, rows)
@@ -142,10 +165,12 @@ class RoutedGLU(FeedForward):
         ws = self.rt.workspace
         ids = ws.rows("moe_ids", T, self.top, torch.int32)
         weights = ws.rows("moe_weights", T, self.top, torch.float32)
-        ops.route_topk(ids, weights, x, self.w_router, self.b_router, logistic=self.score == "sigmoid")
+        ops.route_topk(ids, weights, x, self.w_router, self.b_router, logistic=self.score == "sigmoid",
+                       groups=self.groups if self.score == "softmax_all" else 0, keep=self.keep_groups)
         y = ws.rows("ffn_out", T, self.hidden_size, x.dtype)
         ops.routed_experts(y, x, ids, weights, self.w_gate_up, self.w_down, workspace=ws,
-                           kernel="rows" if self.rt.plain_kernels else "", weight_on_input=self.weight_on_input)
+                           kernel="rows" if self.rt.plain_kernels else "", weight_on_input=self.weight_on_input,
+                           activation=self.activation, identity=self.identity, limit=self.limit, alpha=self.alpha)
         if self.shared_size:
             gu = self._project(x, self.shared_gate_up, ws.rows("ffn_gate_up", T, 2 * self.shared_size, x.dtype), T)
             act = ops.swiglu(ws.rows("ffn_act", T, self.shared_size, x.dtype), gu)
@@ -253,7 +278,7 @@ class RoutedAct(FeedForward):
         ops.route_topk(ids, weights, x, self.w_router, None, over_all=True, scale=self.scale, extra_out=gate)
         y = ws.rows("ffn_out", T, self.hidden_size, x.dtype)
         ops.routed_experts(y, x, ids, weights, self.w_up, self.w_down, workspace=ws, kernel="rows" if self.rt.plain_kernels else "",
-                           gated=False)
+                           activation="relu2")
         if self.shared_size:
             up = self._project(x, self.shared_up, ws.rows("ffn_up", T, self.shared_size, x.dtype), T)
             ops.bias_act(up, up, None, "relu2")

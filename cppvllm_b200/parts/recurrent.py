@@ -14,6 +14,10 @@ type; only the projections around them are products in the activations' type.
 * ``head_delta``: the same rule with ONE decay per head and token, g = exp(-exp(A_h) * softplus(Wa x + dt_h)), S <- g S, full-rank
   projections for the decay (Wa [H, D]) and the output gate (Wg [H * vdim, D]), and the gate through silu instead of the
   logistic function: y = Wo concat_h(RMSNorm(o_h) * w * silu(Wg x)_h).
+* ``gated_linear``: q = Wq x * dim^-1/2, k = Wk x, v = Wv x; g = sigmoid(Wa2 Wa1 x + b)^(1 / tau) per head and key channel;
+  S <- diag(g) S + k v^T;  o = S^T q;  y = Wo concat_h(RMSNorm(o_h) * w * silu(Wg x)_h), w shared by the heads.  State per request:
+  [H, dim, vdim].  A step of decoded tokens is one kernel between the projections.  The inner size of the low-rank projection is
+  whatever the checkpoint holds.
 """
 from __future__ import annotations
 
@@ -210,3 +214,69 @@ class HeadDeltaMixer(Mixer):
         y = ops.gated_norm(ws.rows("rec_y", T, H * dv, x.dtype), o, packed[:, self.g_off:self.g_off + H * dv], self.w_norm, H, self.eps,
                            gate_act="silu")
         return _project(self.rt, y, self.w_o, ws.rows("attn_proj", T, self.hidden_size, x.dtype), T)
+
+
+@register_part("mixer", "gated_linear")
+class GatedLinearMixer(Mixer):
+    def __init__(self, runtime, prefix="", names=None, *, hidden_size: int, num_heads: int, dim: int, vdim: int, tau: float, eps: float,
+                 decay_rank: Optional[int] = None):
+        super().__init__(runtime, prefix, names)
+        self.hidden_size, self.num_heads, self.dim, self.vdim = int(hidden_size), int(num_heads), int(dim), int(vdim)
+        self.tau, self.eps = float(tau), float(eps)
+        self.decay_rank = int(decay_rank) if decay_rank else -1
+        if self.dim > 512:
+            raise ValueError("the scan kernel keeps at most 512 key channels per head")
+        self.core_width = self.num_heads * self.vdim
+        self.w_in = self.w_o = self.w_a2 = None
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec((self.num_heads * self.dim * self.vdim,), torch.float32)
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        D, H, dk, dv, R = self.hidden_size, self.num_heads, self.dim, self.vdim, self.decay_rank
+        f = self.full_name
+        return {f("q"): WeightSpec((H * dk, D)), f("k"): WeightSpec((H * dk, D)), f("v"): WeightSpec((H * dv, D)), f("g"): WeightSpec((H * dv, D)),
+                f("a1"): WeightSpec((R, D)), f("a2"): WeightSpec((H * dk, R)), f("a2.b"): WeightSpec((H * dk,), role="vector"),
+                f("norm"): WeightSpec((dv,), role="vector", init="norm"), f("o"): WeightSpec((D, H * dv))}
+
+    def bind(self, tensors) -> None:
+        t = lambda n: tensors[self.full_name(n)]          # noqa: E731
+        self.decay_rank = t("a1").shape[0]
+        if t("a2").shape[1] != self.decay_rank:
+            raise ValueError(f"{self.prefix}: the two halves of the low-rank projection disagree about its inner size")
+        self.w_in = _cat_rows([t("q"), t("k"), t("v"), t("g"), t("a1")])
+        self.w_a2, self.b_a2, self.w_norm, self.w_o = t("a2"), t("a2.b").contiguous(), t("norm").contiguous(), t("o")
+        self._scaled = (1.0, self.w_norm)
+
+    def inner_weight_bytes(self) -> int:
+        return self.w_a2.numel() * self.w_a2.element_size()
+
+    def weight_bytes(self) -> int:
+        return self.inner_weight_bytes() + sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o))
+
+    def forward(self, x, ctx, cache, state):
+        T = x.shape[0]
+        ws = self.rt.workspace
+        packed = _project(self.rt, x, self.w_in, ws.rows("rec_in", T, self.w_in.shape[0], x.dtype), T)
+        y = self.core(packed, ws.rows("rec_y", T, self.core_width, x.dtype), 1.0, ctx, cache, state)
+        return _project(self.rt, y, self.w_o, ws.rows("attn_proj", T, self.hidden_size, x.dtype), T)
+
+    def core(self, packed, out, scale, ctx, cache, state):
+        T, S = packed.shape[0], ctx.num_seqs
+        H, dk, dv, R = self.num_heads, self.dim, self.vdim, self.decay_rank
+        q_off, k_off, v_off, g_off, a_off = 0, H * dk, 2 * H * dk, 2 * H * dk + H * dv, 2 * H * dk + 2 * H * dv
+        qk_scale = dk ** -0.5
+        if (ctx.all_decode and T == S and not self.rt.plain_kernels and self.w_a2.dtype == packed.dtype
+                and ops.linear_step_supported(dk, dv, R)):
+            return ops.linear_step(out, packed, q_off, k_off, v_off, g_off, a_off, self.w_a2, self.b_a2, qk_scale, self.tau, self.w_norm,
+                                   self.eps, scale, state, ctx.cu_seqlens, ctx.state_slots, S, H, dk, dv)
+        ws, f32 = self.rt.workspace, torch.float32
+        # the decay's logits leave their product unrounded and become the decays in place
+        z = ops.linear(packed[:, a_off:a_off + R], self.w_a2, out=ws.rows("linear_g", T, H * dk, f32), out_dtype=f32)
+        qf, kf, vf = ws.rows("delta_q", T, H * dk, f32), ws.rows("delta_k", T, H * dk, f32), ws.rows("delta_v", T, H * dv, f32)
+        ops.linear_prep(qf, kf, vf, z, packed, q_off, k_off, v_off, z, self.b_a2, qk_scale, self.tau)
+        o = ws.rows("rec_o", T, H * dv, f32)
+        ops.linear_scan(o, qf, kf, vf, z, state, ctx.cu_seqlens, ctx.state_slots, S, H, dk, dv)
+        if self._scaled[0] != scale:                      # the constant rides on the norm's weight
+            self._scaled = (scale, (self.w_norm * scale).contiguous())
+        return ops.gated_norm(out, o, packed[:, g_off:g_off + H * dv], self._scaled[1], H, self.eps, gate_act="silu")

@@ -1,0 +1,89 @@
+"""Mixer ``side_by_side``: several mixers that read the same input, their outputs added up with a constant each:
+
+    y = sum_m scale_m mixer_m(x)
+
+A member keeps its own tensors, cache entries and state, and offers its middle part, ``core(packed, out, scale, ctx, cache,
+state)``: from the columns of its input projection (``w_in``) to ``core_width`` columns in front of its output projection
+(``w_o``), times `scale`.  The members' input projections are one product (their rows one below the other), the scaled cores lie
+side by side in one buffer, and their output projections are one product too (their columns side by side), whose sum over
+the inner dimension is the sum over the members: two products for the layer, and no kernel adds anything up.
+At most one member may keep cache entries and at most one per-request state.
+"""
+from __future__ import annotations
+
+from typing import Dict, Sequence
+
+import torch
+
+from .base import Mixer, WeightSpec, register_part
+from .recurrent import _cat_rows, _project
+
+ROW_STEP = 8        # the joined input projection's rows are padded to whole 16-byte chunks of bf16 outputs
+
+
+@register_part("mixer", "side_by_side")
+class SideBySideMixer(Mixer):
+    def __init__(self, runtime, prefix="", names=None, *, hidden_size: int, members: Sequence[Mixer], scales: Sequence[float]):
+        super().__init__(runtime, prefix, names)
+        self.hidden_size, self.members, self.scales = int(hidden_size), tuple(members), tuple(float(s) for s in scales)
+        if not self.members or len(self.members) != len(self.scales):
+            raise ValueError("one scale per mixer")
+        for m in self.members:
+            if not hasattr(m, "core"):
+                raise ValueError(f"{type(m).__name__} does not offer what lies between its projections")
+        if sum(m.cache_spec() is not None for m in self.members) > 1 or sum(m.state_spec() is not None for m in self.members) > 1:
+            raise ValueError("at most one of the mixers keeps cache entries, and at most one per-request state")
+        self.core_width = sum(m.core_width for m in self.members)
+        self.w_in = self.w_o = None
+
+    @property
+    def capturable(self) -> bool:
+        return all(m.capturable for m in self.members)
+
+    def _only(self, specs):
+        return next((s for s in specs if s is not None), None)
+
+    def cache_spec(self):
+        return self._only(m.cache_spec() for m in self.members)
+
+    def state_spec(self):
+        return self._only(m.state_spec() for m in self.members)
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        specs: Dict[str, WeightSpec] = {}
+        for m in self.members:
+            specs.update(m.weight_specs())
+        return specs
+
+    def bind(self, tensors) -> None:
+        self.in_cols = []
+        col = 0
+        for m in self.members:
+            m.bind(tensors)
+            self.in_cols.append((col, col + m.w_in.shape[0]))
+            col += m.w_in.shape[0]
+        rows = [m.w_in for m in self.members]
+        pad = -col % ROW_STEP
+        if pad:
+            rows.append(torch.zeros(pad, self.hidden_size, dtype=rows[0].dtype, device=rows[0].device))
+        self.w_in = _cat_rows(rows)
+        outs = [m.w_o for m in self.members]
+        if len({o.dtype for o in outs}) > 1:
+            outs = [o.float() for o in outs]
+        self.w_o = torch.cat(outs, dim=1).contiguous()
+        for m in self.members:                # the joined matrices are the ones that are read
+            m.w_in = m.w_o = None
+
+    def weight_bytes(self) -> int:
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o)) + sum(getattr(m, "inner_weight_bytes", int)() for m in self.members)
+
+    def forward(self, x, ctx, cache, state):
+        T = x.shape[0]
+        ws = self.rt.workspace
+        packed = _project(self.rt, x, self.w_in, ws.rows("pair_in", T, self.w_in.shape[0], x.dtype), T)
+        joined = ws.rows("pair_out", T, self.core_width, x.dtype)
+        o0 = 0
+        for m, scale, (c0, c1) in zip(self.members, self.scales, self.in_cols):
+            m.core(packed[:, c0:c1], joined[:, o0:o0 + m.core_width], scale, ctx, cache, state)
+            o0 += m.core_width
+        return _project(self.rt, joined, self.w_o, ws.rows("attn_proj", T, self.hidden_size, x.dtype), T)

@@ -4,7 +4,7 @@ where a norm hands it to a matrix product.
 
 * embedding ``scaled_positions``: h = table[token] * scale + pos_table[position] (a learned vector per position; the
   position table is optional, the scale defaults to 1).
-* norm ``rmsnorm_wide``: y = T(x / sqrt(mean(x^2) + eps) * w), one rounding, at the store.  ``add_forward`` takes one
+* norm ``rmsnorm_wide``: y = T(x / sqrt(mean(x^2) + eps) * w), one rounding, at the store (``gain`` multiplies w).  ``add_forward`` takes one
   delta or a tuple of two, adds them to the stream in float (h + (d1 + d2)) and norms the sum, one kernel.
   With ``offset`` the stored weight is a distance from it (w_used = offset + w_stored; 1 for weights stored around zero).
   ``add_normed`` is the norm behind a sublayer: h <- h + norm(y [+ bias]); only the normed output joins the stream.
@@ -87,10 +87,10 @@ class WideRMSNorm(Norm):
     plain_rms = True          # y = x / rms(x) * self.weight with self.eps: a kernel that holds the row may apply it ahead of time
 
     def __init__(self, runtime, prefix="", names=None, *, size: int, eps: float, buffer: str = "normed",
-                 weight_name: str = "weight", offset: float = 0.0):
+                 weight_name: str = "weight", offset: float = 0.0, gain: float = 1.0):
         super().__init__(runtime, prefix, names)
         self.size, self.eps, self.buffer, self.weight_name = int(size), float(eps), buffer, weight_name
-        self.offset = float(offset)
+        self.offset, self.gain = float(offset), float(gain)
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -100,6 +100,8 @@ class WideRMSNorm(Norm):
         self.weight = tensors[self.full_name(self.weight_name)]
         if self.offset:
             self.weight = (self.weight + self.offset).contiguous()
+        if self.gain != 1.0:
+            self.weight = (self.weight * self.gain).contiguous()
 
     def add_normed(self, h, y, ctx, bias=None):
         """h <- h + norm(y + bias) * w, in place; returns the new stream in the activations' type."""
