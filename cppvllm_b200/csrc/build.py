@@ -44,6 +44,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "latent": ["latent.cu"],
     "recurrent": ["recurrent.cu"],
     "lru": ["lru.cu"],
+    "linear": ["linear.cu"],
     "sandwich": ["sandwich.cu"],
     "hyper": ["hyper.cu"],
     "attn_masked": ["attention_masked.cu"],

@@ -2,7 +2,7 @@
 //
 //   route_topk     : z = x Wr^T + b in float (x may be bf16; Wr and b are float); top-k by z
 //                    (of equal z the lower index first), weights exp(z_e) / sum over the k winners of exp(z_c):
-//                    ids[t, k], weights[t, k], k in order of falling logit.  One warp per token.
+//                    ids[t, k], weights[t, k], k in order of falling logit.
 //                    `mode` 1: weights scale * exp(z_e) / sum over ALL experts of exp(z_c) instead (not renormalised over the
 //                    winners).  Rows of Wr behind the E experts' (`extra` of them) are not experts: their raw products
 //                    leave as extra_out[t, :] (a gate per token that shares the router's pass over x).
@@ -33,53 +33,13 @@
 
 namespace cvb {
 
-constexpr int kRouteWarps = 4;
+constexpr int kRouteWarps = 4;          // many tokens: warps per block, kRouteTokens tokens each
+constexpr int kRouteTokens = 4;
+constexpr int kRouteFewWarps = 8;       // few tokens: the warps of a block share one token's router outputs out
 
-template <typename T>
-__global__ void __launch_bounds__(kRouteWarps * 32)
-route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x, const float* __restrict__ wr,
-                  const float* __restrict__ bias, int n_tokens, int D, int E, int top, int mode, float scale, int extra,
-                  float* __restrict__ extra_out, int groups, int keep) {
-    pdl_trigger();
-    pdl_wait();
-    extern __shared__ float smem[];                     // [kRouteWarps][E], mode 3: [kRouteWarps][2 E + groups]
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int64_t t = static_cast<int64_t>(blockIdx.x) * kRouteWarps + warp;
-    if (t >= n_tokens) return;
-    float* z = smem + warp * (mode == 3 ? 2 * E + groups : E);
-    const T* xr = x + t * D;
-    // four rows of Wr at a time, each with a sum of its own (a row's sum runs over the same elements in the same order as
-    // alone): four independent loads in flight per lane and step instead of one chain
-    for (int e0 = 0; e0 < E + extra; e0 += 4) {
-        const int ne = min(4, E + extra - e0);
-        const float* w = wr + static_cast<int64_t>(e0) * D;
-        float d[4] = {0.f, 0.f, 0.f, 0.f};
-        if (ne == 4) {
-            for (int i = lane; i < D; i += 32) {
-                const float xv = to_float(xr[i]);
-#pragma unroll
-                for (int q = 0; q < 4; ++q) d[q] = fmaf(xv, w[static_cast<int64_t>(q) * D + i], d[q]);
-            }
-        } else {
-            for (int i = lane; i < D; i += 32) {
-                const float xv = to_float(xr[i]);
-#pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    if (q < ne) d[q] = fmaf(xv, w[static_cast<int64_t>(q) * D + i], d[q]);
-            }
-        }
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-            if (q >= ne) break;
-            const float v = warp_sum(d[q]);
-            const int e = e0 + q;
-            if (lane == 0) {
-                if (e < E) z[e] = v + (bias && mode != 3 ? bias[e] : 0.f);
-                else extra_out[t * extra + (e - E)] = v;
-            }
-        }
-    }
-    __syncwarp();
+// The choice from the logits z [E] (shared memory of the calling warp; in mode 3 with 2 E + groups floats): see the top of this file.
+__device__ __forceinline__ void route_select(float* z, int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ bias,
+                                             int64_t t, int E, int top, int mode, float scale, int groups, int keep, int lane) {
     float all = 0.f;                                    // modes 1 and 3: the sum over all experts, against the largest logit
     if (mode == 1 || mode == 3) {
         float big = -INFINITY;
@@ -145,6 +105,107 @@ route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* _
     }
     const float inv = mode == 1 ? scale / all : (mode == 3 ? scale / (sum + 1e-20f) : 1.f / sum);
     for (int k = lane; k < top; k += 32) weights[t * top + k] *= inv;     // lane 0's writes are visible after the syncwarp
+}
+
+// V elements of a row as floats: 16 bytes of weights, the matching activations
+template <int V> __device__ __forceinline__ void route_load(const float* p, float (&f)[V]) {
+    if constexpr (V == 4) { const float4 v = *reinterpret_cast<const float4*>(p); f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
+    else f[0] = p[0];
+}
+template <int V> __device__ __forceinline__ void route_load(const __nv_bfloat16* p, float (&f)[V]) {
+    if constexpr (V == 4) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+    } else f[0] = __bfloat162float(p[0]);
+}
+
+// Many tokens: a warp holds kRouteTokens tokens by four router outputs in registers, so a weight it loads serves four tokens and
+// an activation four outputs.
+template <typename T, int V>
+__global__ void __launch_bounds__(kRouteWarps * 32)
+route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x, const float* __restrict__ wr,
+                  const float* __restrict__ bias, int n_tokens, int D, int E, int top, int mode, float scale, int extra,
+                  float* __restrict__ extra_out, int groups, int keep) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ float smem[];                     // [kRouteWarps][kRouteTokens][E], mode 3: [..][2 E + groups]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int64_t t0 = (static_cast<int64_t>(blockIdx.x) * kRouteWarps + warp) * kRouteTokens;
+    if (t0 >= n_tokens) return;
+    const int nt = static_cast<int>(n_tokens - t0 < kRouteTokens ? n_tokens - t0 : kRouteTokens);
+    const int per = mode == 3 ? 2 * E + groups : E;
+    float* z = smem + static_cast<int64_t>(warp) * kRouteTokens * per;
+    const T* xr[kRouteTokens];
+#pragma unroll
+    for (int k = 0; k < kRouteTokens; ++k) xr[k] = x + (t0 + min(k, nt - 1)) * D;       // rows past the end repeat the last one
+    for (int e0 = 0; e0 < E + extra; e0 += 4) {
+        const float* w[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) w[q] = wr + static_cast<int64_t>(min(e0 + q, E + extra - 1)) * D;
+        float d[kRouteTokens][4];
+#pragma unroll
+        for (int k = 0; k < kRouteTokens; ++k) { d[k][0] = d[k][1] = d[k][2] = d[k][3] = 0.f; }
+        for (int i = lane * V; i < D; i += 32 * V) {
+            float wv[4][V], xv[kRouteTokens][V];
+#pragma unroll
+            for (int q = 0; q < 4; ++q) route_load<V>(w[q] + i, wv[q]);
+#pragma unroll
+            for (int k = 0; k < kRouteTokens; ++k) route_load<V>(xr[k] + i, xv[k]);
+#pragma unroll
+            for (int k = 0; k < kRouteTokens; ++k)
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+#pragma unroll
+                    for (int v = 0; v < V; ++v) d[k][q] = fmaf(xv[k][v], wv[q][v], d[k][q]);
+        }
+#pragma unroll
+        for (int k = 0; k < kRouteTokens; ++k)
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+                const float v = warp_sum(d[k][q]);
+                const int e = e0 + q;
+                if (lane == 0 && k < nt && e < E + extra) {
+                    if (e < E) z[k * per + e] = v + (bias && mode != 3 ? bias[e] : 0.f);
+                    else extra_out[(t0 + k) * extra + (e - E)] = v;
+                }
+            }
+    }
+    __syncwarp();
+    for (int k = 0; k < nt; ++k) route_select(z + k * per, ids, weights, bias, t0 + k, E, top, mode, scale, groups, keep, lane);
+}
+
+// Few tokens: a block per token; its warps take the router outputs in turn.
+template <typename T, int V>
+__global__ void __launch_bounds__(kRouteFewWarps * 32)
+route_topk_few_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x, const float* __restrict__ wr,
+                      const float* __restrict__ bias, int D, int E, int top, int mode, float scale, int extra,
+                      float* __restrict__ extra_out, int groups, int keep) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ float smem[];                     // [E], mode 3: [2 E + groups]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int64_t t = blockIdx.x;
+    const T* xr = x + t * D;
+    for (int e = warp; e < E + extra; e += kRouteFewWarps) {
+        const float* w = wr + static_cast<int64_t>(e) * D;
+        float d = 0.f;
+#pragma unroll 8
+        for (int i = lane * V; i < D; i += 32 * V) {
+            float wv[V], xv[V];
+            route_load<V>(w + i, wv);
+            route_load<V>(xr + i, xv);
+#pragma unroll
+            for (int v = 0; v < V; ++v) d = fmaf(xv[v], wv[v], d);
+        }
+        d = warp_sum(d);
+        if (lane == 0) {
+            if (e < E) smem[e] = d + (bias && mode != 3 ? bias[e] : 0.f);
+            else extra_out[t * extra + (e - E)] = d;
+        }
+    }
+    __syncthreads();
+    if (warp == 0) route_select(smem, ids, weights, bias, t, E, top, mode, scale, groups, keep, lane);
 }
 
 constexpr int kExpertThreads = 256;
@@ -392,12 +453,27 @@ extern "C" int cvb_route_topk(int* ids, float* weights, const void* x, const flo
     if (mode < 0 || mode > 3) return CVB_E_SHAPE;
     if (top > E || E > 2048) return CVB_E_SHAPE;
     if (mode == 3 && (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups))) return CVB_E_SHAPE;
-    const size_t smem = static_cast<size_t>(kRouteWarps) * (mode == 3 ? 2 * E + groups : E) * sizeof(float);
-    if (smem > 48 * 1024) return CVB_E_SIZE;
-#define CALL(TY) launch_kernel(route_topk_kernel<TY>, dim3((T + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), smem, \
-                               stream, ids, weights, (const TY*)x, wr, bias, T, D, E, top, mode, scale, extra, extra_out, groups, keep)
+    const size_t row = static_cast<size_t>(mode == 3 ? 2 * E + groups : E) * sizeof(float);
+    if (row * kRouteWarps * kRouteTokens > 200 * 1024) return CVB_E_SIZE;
+    const bool few = T <= 512;
+    const bool four = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(wr)) & 15) == 0;
+    const size_t smem = few ? row : row * kRouteWarps * kRouteTokens;
+#define CALL_V(TY, V)                                                                                                         \
+    do {                                                                                                                      \
+        if (few) {                                                                                                            \
+            launch_kernel(route_topk_few_kernel<TY, V>, dim3(T), dim3(kRouteFewWarps * 32), smem, stream, ids, weights, (const TY*)x, wr, bias, \
+                          D, E, top, mode, scale, extra, extra_out, groups, keep);                                            \
+        } else {                                                                                                              \
+            if (smem > 48 * 1024) cudaFuncSetAttribute(route_topk_kernel<TY, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
+            launch_kernel(route_topk_kernel<TY, V>, dim3((T + kRouteWarps * kRouteTokens - 1) / (kRouteWarps * kRouteTokens)),                  \
+                          dim3(kRouteWarps * 32), smem, stream, ids, weights, (const TY*)x, wr, bias, T, D, E, top, mode, scale, extra,         \
+                          extra_out, groups, keep);                                                                           \
+        }                                                                                                                     \
+    } while (0)
+#define CALL(TY) if (four) { CALL_V(TY, 4); } else { CALL_V(TY, 1); }
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
+#undef CALL_V
     return launch_status();
 }
 

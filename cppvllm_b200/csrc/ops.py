@@ -614,8 +614,7 @@ def _recurrent_lib():
     global _recurrent
     if _recurrent is None:
         lib = load_library("recurrent")
-        for name in ("cvb_lightning_prep", "cvb_lightning_scan", "cvb_linear_prep", "cvb_linear_scan", "cvb_linear_step", "cvb_delta_prep",
-                     "cvb_conv_history", "cvb_delta_scan"):
+        for name in ("cvb_lightning_prep", "cvb_lightning_scan", "cvb_delta_prep", "cvb_conv_history", "cvb_delta_scan"):
             getattr(lib, name).restype = c_int
         _recurrent = lib
     return _recurrent
@@ -658,34 +657,117 @@ def lightning_scan(out: torch.Tensor, qf: torch.Tensor, kf: torch.Tensor, vf: to
     return out
 
 
-def linear_prep(qf: torch.Tensor, kf: torch.Tensor, vf: torch.Tensor, gg: torch.Tensor, packed: torch.Tensor, q_off: int, k_off: int,
-                v_off: int, z: torch.Tensor, bias: torch.Tensor, qk_scale: float, tau: float) -> None:
-    """qf = qk_scale * q, kf = k [T, H * dim] and vf = v [T, H * vdim] (float32) from the packed projection's column ranges, and the decays
-    gg = sigmoid(z + bias)^(1 / tau) [T, H * dim] from the float32 product z (gg may be z itself)."""
-    _cuda(qf, kf, vf, gg, packed, z, bias); _contig(qf, kf, vf, gg, z, bias)
-    T = packed.shape[0]
-    if (any(t.dtype != torch.float32 for t in (qf, kf, vf, gg, z, bias)) or kf.shape != qf.shape or gg.shape != qf.shape or z.shape != qf.shape
-            or qf.shape[0] != T or vf.shape[0] != T or bias.numel() != qf.shape[1] or packed.stride(1) != 1):
-        raise KernelError("linear_prep: q, k, decays and z float32 [T, H * dim], v float32 [T, H * vdim], bias float32 [H * dim]")
-    _check(_recurrent_lib().cvb_linear_prep(_ptr(qf), _ptr(kf), _ptr(vf), _ptr(gg), _ptr(packed), c_int(T), c_int(packed.stride(0)), c_int(q_off),
-                                            c_int(k_off), c_int(v_off), _ptr(z), _ptr(bias), c_float(qk_scale), c_float(1.0 / tau),
-                                            c_int(qf.shape[1]), c_int(vf.shape[1]), c_int(dtype_code(packed.dtype)), _stream()), "linear_prep")
-
-
-def linear_scan(out: torch.Tensor, qf: torch.Tensor, kf: torch.Tensor, vf: torch.Tensor, gg: torch.Tensor, state: torch.Tensor,
-                cu_seqlens: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, num_heads: int, dim: int, vdim: int) -> torch.Tensor:
-    """Per request and head, over the request's tokens of this step: S <- diag(g) S + k v^T, out = S^T q; q, k, g [T, H * dim] and v
-    [T, H * vdim] float32; S [dim, vdim] float32 at the front of the request's state row.  out float32 [T, H * vdim]."""
-    _cuda(out, qf, kf, vf, gg, state, cu_seqlens, state_slots); _contig(out, qf, kf, vf, gg, cu_seqlens, state_slots)
+def delta_prep(qn, kn, vv, gg, bb, packed: torch.Tensor, qkv_off: int, conv_w: torch.Tensor, a: torch.Tensor, dt_bias: torch.Tensor,
+               a_log: torch.Tensor, b: torch.Tensor, state: torch.Tensor, conv_off: int, seq_of_token, cu_seqlens, state_slots,
+               num_heads: int, num_kv_heads: int, dim: int, vdim: int, decay_dim: Optional[int] = None) -> None:
+    """Per token: convolutions with silu, unit q and k, sigmoid(b), the decay; all outputs float32 (see csrc/recurrent.cu).
+    `decay_dim`: decays per head, `dim` (one per key channel, the default) or 1 (one per head)."""
+    _cuda(qn, kn, vv, gg, bb, packed, conv_w, a, dt_bias, a_log, b, state, seq_of_token, cu_seqlens, state_slots)
+    _contig(qn, kn, vv, gg, bb, packed, conv_w, a, dt_bias, a_log, b, seq_of_token, cu_seqlens, state_slots)
     sp, sf, n_slots = _state_args(state)
-    T = qf.shape[0]
-    if (any(t.dtype != torch.float32 for t in (out, qf, kf, vf, gg)) or out.shape != (T, num_heads * vdim) or qf.shape != (T, num_heads * dim)
-            or kf.shape != qf.shape or gg.shape != qf.shape or vf.shape != out.shape or cu_seqlens.dtype != torch.int32
-            or state_slots.dtype != torch.int32):
-        raise KernelError("linear_scan: q, k, g float32 [T, H * dim]; v, out float32 [T, H * vdim]; cu_seqlens, state_slots int32")
-    _check(_recurrent_lib().cvb_linear_scan(
-        _ptr(out), _ptr(qf), _ptr(kf), _ptr(vf), _ptr(gg), sp, sf, _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs),
-        c_int(num_heads), c_int(dim), c_int(vdim), _ptr(error_flag(out.device)), _stream()), "linear_scan")
+    T = packed.shape[0]
+    H, G = num_heads, num_kv_heads
+    C = 2 * G * dim + H * vdim
+    gd = dim if decay_dim is None else int(decay_dim)
+    for t_, n_ in ((qn, T * G * dim), (kn, T * G * dim), (vv, T * H * vdim), (gg, T * H * gd), (bb, T * H), (a, T * H * gd), (b, T * H),
+                   (dt_bias, H * gd), (a_log, H)):
+        if t_.dtype != torch.float32 or t_.numel() != n_:
+            raise KernelError("delta_prep: float32 buffers of the sizes the head counts give")
+    if conv_w.dtype != torch.float32 or conv_w.dim() != 2 or conv_w.shape[0] != C:
+        raise KernelError("delta_prep: conv_w float32 [channels, taps]")
+    _check(_recurrent_lib().cvb_delta_prep(
+        _ptr(qn), _ptr(kn), _ptr(vv), _ptr(gg), _ptr(bb), _ptr(packed), c_int(T), c_int(packed.shape[1]), c_int(qkv_off), _ptr(conv_w),
+        c_int(conv_w.shape[1]), _ptr(a), _ptr(dt_bias), _ptr(a_log), _ptr(b), sp, sf, c_int64(conv_off), _ptr(seq_of_token),
+        _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(H), c_int(G), c_int(dim), c_int(vdim), c_int(gd), c_int(dtype_code(packed.dtype)),
+        _ptr(error_flag(packed.device)), _stream()), "delta_prep")
+
+
+def conv_history(state: torch.Tensor, conv_off: int, packed: torch.Tensor, qkv_off: int, channels: int, taps: int, cu_seqlens,
+                 state_slots, num_seqs: int) -> None:
+    """The last taps - 1 raw inputs of every request's portion (older ones from the old history) become its history."""
+    _cuda(state, packed, cu_seqlens, state_slots); _contig(packed, cu_seqlens, state_slots)
+    sp, sf, n_slots = _state_args(state)
+    _check(_recurrent_lib().cvb_conv_history(sp, sf, c_int64(conv_off), _ptr(packed), c_int(packed.shape[1]), c_int(qkv_off), c_int(channels),
+                                             c_int(taps), _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs),
+                                             c_int(dtype_code(packed.dtype)), _stream()), "conv_history", kernels=1 if taps > 1 else 0)
+
+
+def delta_scan(out, qn, kn, vv, gg, bb, state: torch.Tensor, cu_seqlens, state_slots, num_seqs: int, num_heads: int, num_kv_heads: int,
+               dim: int, vdim: int, decay_dim: Optional[int] = None) -> torch.Tensor:
+    """Per request and head: S <- diag(g) S; u = b (v - S^T k); S <- S + k u^T; out = S^T q.  out float32 [T, H * vdim].
+    gg is [T, H * dim], or [T, H] with `decay_dim` = 1 (one decay per head: S <- g S)."""
+    _cuda(out, qn, kn, vv, gg, bb, state, cu_seqlens, state_slots); _contig(out, qn, kn, vv, gg, bb, cu_seqlens, state_slots)
+    sp, sf, n_slots = _state_args(state)
+    if out.dtype != torch.float32:
+        raise KernelError("delta_scan: out is float32")
+    _check(_recurrent_lib().cvb_delta_scan(_ptr(out), _ptr(qn), _ptr(kn), _ptr(vv), _ptr(gg), _ptr(bb), sp, sf, _ptr(cu_seqlens),
+                                           _ptr(state_slots), c_int(n_slots), c_int(num_seqs), c_int(num_heads), c_int(num_kv_heads),
+                                           c_int(dim), c_int(vdim), c_int(dim if decay_dim is None else int(decay_dim)),
+                                           _ptr(error_flag(out.device)), _stream()), "delta_scan")
+    return out
+
+
+# ---- gated linear attention (csrc/linear.cu) ------------------------------------------------------------------------------------
+
+_linear = None
+LINEAR_BLOCKS = 1184        # blocks of a scan that keep every SM busy
+LINEAR_MIN_CHUNK = 64
+
+
+def _linear_lib():
+    global _linear
+    if _linear is None:
+        lib = load_library("linear")
+        for name in ("cvb_linear_decay", "cvb_linear_scan", "cvb_linear_step"):
+            getattr(lib, name).restype = c_int
+        _linear = lib
+    return _linear
+
+
+def linear_decay(z: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
+    """z (float32 [T, n], in place) <- sigmoid(z + bias)^(1 / tau)."""
+    _cuda(z, bias); _contig(z, bias)
+    if z.dtype != torch.float32 or bias.dtype != torch.float32 or bias.numel() != z.shape[1]:
+        raise KernelError("linear_decay: z float32 [T, n], bias float32 [n]")
+    _check(_linear_lib().cvb_linear_decay(_ptr(z), _ptr(bias), c_float(1.0 / tau), c_int(z.shape[0]), c_int(z.shape[1]), _stream()), "linear_decay")
+    return z
+
+
+def linear_chunk_tokens(num_tokens: int, num_heads: int, vdim: int) -> int:
+    """Tokens per chunk of a portion: as many chunks as it takes to keep every SM busy, none shorter than 64 tokens."""
+    per_chunk = num_heads * ((vdim + 31) // 32)
+    n = -(-num_tokens * per_chunk // LINEAR_BLOCKS)
+    return max(LINEAR_MIN_CHUNK, -(-n // 64) * 64)
+
+
+def linear_held_chunks(max_tokens: int, num_heads: int, vdim: int) -> int:
+    """The most chunks that requests with more than one chunk can have in a step of up to `max_tokens` tokens: a request of n tokens has
+    fewer than 2 n / len."""
+    per_chunk = num_heads * ((vdim + 31) // 32)
+    return min(2 * max_tokens // LINEAR_MIN_CHUNK, 2 * LINEAR_BLOCKS // per_chunk) + 2
+
+
+def linear_scan(out: torch.Tensor, packed: torch.Tensor, q_off: int, k_off: int, v_off: int, qk_scale: float, gg: torch.Tensor,
+                state: torch.Tensor, cu_seqlens: torch.Tensor, state_slots: torch.Tensor, q_lens, num_heads: int, dim: int, vdim: int,
+                chunk_tokens: int, ends: Optional[torch.Tensor] = None, decays: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per request and head, over the request's tokens of this step: S <- diag(g) S + k v^T, out = S^T (qk_scale q), with q, k, v column
+    ranges of `packed`, g float32 [T, H * dim], S [dim, vdim] float32 at the front of the request's state row.  out float32 [T, H * vdim].
+    `q_lens`: the requests' portion lengths; portions longer than `chunk_tokens` are worked on in chunks side by side through `ends`
+    (float32, H dim vdim per chunk of such a portion) and `decays` (float32, H dim per chunk)."""
+    _cuda(out, packed, gg, state, cu_seqlens, state_slots, ends, decays); _contig(out, gg, cu_seqlens, state_slots, ends, decays)
+    sp, sf, n_slots = _state_args(state)
+    T = packed.shape[0]
+    if (out.dtype != torch.float32 or gg.dtype != torch.float32 or out.shape != (T, num_heads * vdim) or gg.shape != (T, num_heads * dim)
+            or packed.stride(1) != 1 or cu_seqlens.dtype != torch.int32 or state_slots.dtype != torch.int32
+            or any(t is not None and t.dtype != torch.float32 for t in (ends, decays))):
+        raise KernelError("linear_scan: g float32 [T, H * dim], out float32 [T, H * vdim], cu_seqlens and state_slots int32")
+    per = [-(-n // chunk_tokens) for n in q_lens]
+    held = sum(c for c in per if c > 1)
+    _check(_linear_lib().cvb_linear_scan(
+        _ptr(out), _ptr(packed), c_int(packed.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), c_float(qk_scale), _ptr(gg), sp, sf, c_int(n_slots),
+        _ptr(ends), c_int64(ends.numel() if ends is not None else 0), _ptr(decays), c_int64(decays.numel() if decays is not None else 0),
+        _ptr(cu_seqlens), _ptr(state_slots), c_int(len(per)), c_int(chunk_tokens), c_int(sum(per)), c_int(held), c_int(num_heads), c_int(dim),
+        c_int(vdim), c_int(dtype_code(packed.dtype)), _ptr(error_flag(out.device)), _stream()), "linear_scan", kernels=3 if held else 1)
     return out
 
 
@@ -709,7 +791,7 @@ def linear_step(out: torch.Tensor, packed: torch.Tensor, q_off: int, k_off: int,
             or a2_bias.dtype != torch.float32 or a2_bias.numel() != num_heads * dim or norm_weight.dtype != torch.float32
             or norm_weight.numel() != vdim or cu_seqlens.dtype != torch.int32 or state_slots.dtype != torch.int32):
         raise KernelError("linear_step: out [S, H * vdim], w_a2 [H * dim, rank] of packed's element type; bias, norm weight float32")
-    _check(_recurrent_lib().cvb_linear_step(
+    _check(_linear_lib().cvb_linear_step(
         _ptr(out), c_int(out.stride(0)), _ptr(packed), c_int(packed.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), c_int(g_off),
         c_int(a_off), c_int(rank), _ptr(w_a2), _ptr(a2_bias), c_float(qk_scale), c_float(1.0 / tau), _ptr(norm_weight), c_float(eps),
         c_float(out_scale), sp, sf, _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs), c_int(num_heads), c_int(dim),
@@ -829,56 +911,6 @@ def lru_step(out: torch.Tensor, packed: torch.Tensor, y_off: int, x_off: int, bi
         _ptr(neg_softplus), sp, sf, c_int(n_slots), _ptr(cu_seqlens), _ptr(state_slots), _ptr(positions), c_int(num_seqs), c_int(W), c_int(parts),
         c_int(taps), c_int(packed.stride(0)), c_int(y_off), c_int(x_off), c_int(dtype_code(packed.dtype)), _ptr(error_flag(out.device)),
         _stream()), "lru_step")
-    return out
-
-
-def delta_prep(qn, kn, vv, gg, bb, packed: torch.Tensor, qkv_off: int, conv_w: torch.Tensor, a: torch.Tensor, dt_bias: torch.Tensor,
-               a_log: torch.Tensor, b: torch.Tensor, state: torch.Tensor, conv_off: int, seq_of_token, cu_seqlens, state_slots,
-               num_heads: int, num_kv_heads: int, dim: int, vdim: int, decay_dim: Optional[int] = None) -> None:
-    """Per token: convolutions with silu, unit q and k, sigmoid(b), the decay; all outputs float32 (see csrc/recurrent.cu).
-    `decay_dim`: decays per head, `dim` (one per key channel, the default) or 1 (one per head)."""
-    _cuda(qn, kn, vv, gg, bb, packed, conv_w, a, dt_bias, a_log, b, state, seq_of_token, cu_seqlens, state_slots)
-    _contig(qn, kn, vv, gg, bb, packed, conv_w, a, dt_bias, a_log, b, seq_of_token, cu_seqlens, state_slots)
-    sp, sf, n_slots = _state_args(state)
-    T = packed.shape[0]
-    H, G = num_heads, num_kv_heads
-    C = 2 * G * dim + H * vdim
-    gd = dim if decay_dim is None else int(decay_dim)
-    for t_, n_ in ((qn, T * G * dim), (kn, T * G * dim), (vv, T * H * vdim), (gg, T * H * gd), (bb, T * H), (a, T * H * gd), (b, T * H),
-                   (dt_bias, H * gd), (a_log, H)):
-        if t_.dtype != torch.float32 or t_.numel() != n_:
-            raise KernelError("delta_prep: float32 buffers of the sizes the head counts give")
-    if conv_w.dtype != torch.float32 or conv_w.dim() != 2 or conv_w.shape[0] != C:
-        raise KernelError("delta_prep: conv_w float32 [channels, taps]")
-    _check(_recurrent_lib().cvb_delta_prep(
-        _ptr(qn), _ptr(kn), _ptr(vv), _ptr(gg), _ptr(bb), _ptr(packed), c_int(T), c_int(packed.shape[1]), c_int(qkv_off), _ptr(conv_w),
-        c_int(conv_w.shape[1]), _ptr(a), _ptr(dt_bias), _ptr(a_log), _ptr(b), sp, sf, c_int64(conv_off), _ptr(seq_of_token),
-        _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(H), c_int(G), c_int(dim), c_int(vdim), c_int(gd), c_int(dtype_code(packed.dtype)),
-        _ptr(error_flag(packed.device)), _stream()), "delta_prep")
-
-
-def conv_history(state: torch.Tensor, conv_off: int, packed: torch.Tensor, qkv_off: int, channels: int, taps: int, cu_seqlens,
-                 state_slots, num_seqs: int) -> None:
-    """The last taps - 1 raw inputs of every request's portion (older ones from the old history) become its history."""
-    _cuda(state, packed, cu_seqlens, state_slots); _contig(packed, cu_seqlens, state_slots)
-    sp, sf, n_slots = _state_args(state)
-    _check(_recurrent_lib().cvb_conv_history(sp, sf, c_int64(conv_off), _ptr(packed), c_int(packed.shape[1]), c_int(qkv_off), c_int(channels),
-                                             c_int(taps), _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs),
-                                             c_int(dtype_code(packed.dtype)), _stream()), "conv_history", kernels=1 if taps > 1 else 0)
-
-
-def delta_scan(out, qn, kn, vv, gg, bb, state: torch.Tensor, cu_seqlens, state_slots, num_seqs: int, num_heads: int, num_kv_heads: int,
-               dim: int, vdim: int, decay_dim: Optional[int] = None) -> torch.Tensor:
-    """Per request and head: S <- diag(g) S; u = b (v - S^T k); S <- S + k u^T; out = S^T q.  out float32 [T, H * vdim].
-    gg is [T, H * dim], or [T, H] with `decay_dim` = 1 (one decay per head: S <- g S)."""
-    _cuda(out, qn, kn, vv, gg, bb, state, cu_seqlens, state_slots); _contig(out, qn, kn, vv, gg, bb, cu_seqlens, state_slots)
-    sp, sf, n_slots = _state_args(state)
-    if out.dtype != torch.float32:
-        raise KernelError("delta_scan: out is float32")
-    _check(_recurrent_lib().cvb_delta_scan(_ptr(out), _ptr(qn), _ptr(kn), _ptr(vv), _ptr(gg), _ptr(bb), sp, sf, _ptr(cu_seqlens),
-                                           _ptr(state_slots), c_int(n_slots), c_int(num_seqs), c_int(num_heads), c_int(num_kv_heads),
-                                           c_int(dim), c_int(vdim), c_int(dim if decay_dim is None else int(decay_dim)),
-                                           _ptr(error_flag(out.device)), _stream()), "delta_scan")
     return out
 
 

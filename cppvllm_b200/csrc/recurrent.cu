@@ -2,12 +2,6 @@
 //
 //   lightning_prep : q = silu(a_q), k = silu(a_k), v = silu(a_v) in float, from a packed projection
 //   lightning_scan : S <- d_h S + k v^T;  o = S^T q
-//   linear_prep    : q = qk_scale * a_q, k = a_k, v = a_v in float from a packed projection, and the decay of every head and key channel
-//                    g = sigmoid(z + b)^(1 / tau) from the float product z
-//   linear_scan    : S <- diag(g) S + k v^T;  o = S^T q      (lightning_scan with a decay per token, head and key channel)
-//   linear_step    : a step of decoded tokens (one per request) of that rule in one kernel, a block per (request, head): the low-rank
-//                    decay product, the decay, the rule on S, the RMS norm of the head's output, its weight, silu of the gate and
-//                    a constant, into a column range of wider rows
 //   delta_prep     : per token, everything the delta rule needs, in float: short causal convolutions over time (per channel,
 //                    the last tap on the current token, history from the request's state where the portion begins) with
 //                    silu behind them; q and k made unit vectors per head (x / sqrt(sum x^2 + 1e-6); q also times
@@ -32,9 +26,6 @@ constexpr int kScanChunk = 8;                            // tokens per stage
 
 __device__ __forceinline__ float silu_of(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
-
-// sigmoid(z)^(1 / tau), through its logarithm min(z, 0) - ln(1 + e^-|z|)
-__device__ __forceinline__ float root_of_sigmoid(float z, float inv_tau) { return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau); }
 
 __device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_u32(smem)), "l"(gmem));
@@ -62,7 +53,7 @@ __global__ void lightning_prep_kernel(float* __restrict__ qf, float* __restrict_
 // (rows r * kScanLanes + lane part) and add their parts up by shuffles.  The tokens' q, k (and g), v (and b) travel through
 // two stages of shared memory by cp.async, kScanChunk tokens a stage, so that the next tokens arrive while these are used.
 // MODE 1: S <- diag(g) S; u = b (v - S^T k); S <- S + k u^T; o = S^T q.  MODE 2: the same with one decay per head and token
-// (S <- g S).  MODE 0: S <- d S + k v^T; o = S^T q.  MODE 3: S <- diag(g) S + k v^T; o = S^T q.
+// (S <- g S).  MODE 0: S <- d S + k v^T; o = S^T q.
 template <int KPT, int MODE>
 __global__ void __launch_bounds__(kScanThreads)
 recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vv,
@@ -73,9 +64,8 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
     constexpr int dkp = KPT * kScanLanes;
-    constexpr bool DELTA = MODE == 1 || MODE == 2;
-    constexpr bool GROWS = MODE == 1 || MODE == 3;         // a decay per key channel travels with the tokens
-    constexpr int kArrays = GROWS ? 3 : 2;
+    constexpr bool DELTA = MODE != 0;
+    constexpr int kArrays = MODE == 1 ? 3 : 2;
     constexpr int kStage = kArrays * kScanChunk * dkp + kScanChunk * kScanCols + 2 * kScanChunk;
     const int s = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * kScanCols;
     const int kvh = h / (H / G);
@@ -95,14 +85,14 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
         const int i = r * kScanLanes + part;
         S[r] = (i < dk && j < dv) ? st[static_cast<int64_t>(i) * dv + j] : 0.f;
     }
-    const float d = MODE == 0 ? decay[h] : 1.f;
+    const float d = DELTA ? 1.f : decay[h];
     const bool vec = (dk & 3) == 0 && (dv & 3) == 0;
 
     auto load = [&](int t0, int stage) {
         const int n = min(kScanChunk, end - t0);
         float* qs = sm + stage * kStage;
         float* ks = qs + kScanChunk * dkp;
-        float* gs = ks + kScanChunk * dkp;                                  // MODE 1 and 3 only
+        float* gs = ks + kScanChunk * dkp;                                  // MODE 1 only
         float* vs = qs + kArrays * kScanChunk * dkp;
         float* bs = vs + kScanChunk * kScanCols;
         float* g1 = bs + kScanChunk;                                        // MODE 2 only: one decay per token
@@ -113,7 +103,7 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
                 const int64_t tok = t0 + tt;
                 cp_async16(qs + tt * dkp + i, qn + (tok * G + kvh) * dk + i, true);
                 cp_async16(ks + tt * dkp + i, kn + (tok * G + kvh) * dk + i, true);
-                if (GROWS) cp_async16(gs + tt * dkp + i, gg + (tok * H + h) * dk + i, true);
+                if (MODE == 1) cp_async16(gs + tt * dkp + i, gg + (tok * H + h) * dk + i, true);
             }
             for (int idx = tid; idx < n * (kScanCols / 4); idx += kScanThreads) {
                 const int tt = idx / (kScanCols / 4), c = (idx - tt * (kScanCols / 4)) * 4;
@@ -125,7 +115,7 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
                 const int64_t tok = t0 + tt;
                 cp_async4(qs + tt * dkp + i, qn + (tok * G + kvh) * dk + i);
                 cp_async4(ks + tt * dkp + i, kn + (tok * G + kvh) * dk + i);
-                if (GROWS) cp_async4(gs + tt * dkp + i, gg + (tok * H + h) * dk + i);
+                if (MODE == 1) cp_async4(gs + tt * dkp + i, gg + (tok * H + h) * dk + i);
             }
             for (int idx = tid; idx < n * kScanCols; idx += kScanThreads) {
                 const int tt = idx / kScanCols, c = idx - tt * kScanCols;
@@ -177,7 +167,7 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
             } else {
 #pragma unroll
                 for (int r = 0; r < KPT; ++r) {
-                    S[r] = fmaf(MODE == 3 ? gs[tt * dkp + part + r * kScanLanes] : d, S[r], kq[r * kScanLanes] * v);
+                    S[r] = fmaf(d, S[r], kq[r * kScanLanes] * v);
                     if (r & 1) o1 = fmaf(S[r], qq[r * kScanLanes], o1); else o0 = fmaf(S[r], qq[r * kScanLanes], o0);
                 }
             }
@@ -199,112 +189,6 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
     for (int r = 0; r < KPT; ++r) {
         const int i = r * kScanLanes + part;
         if (i < dk && j < dv) st[static_cast<int64_t>(i) * dv + j] = S[r];
-    }
-}
-
-template <typename T>
-__global__ void linear_prep_kernel(float* __restrict__ qf, float* __restrict__ kf, float* __restrict__ vf, float* __restrict__ gg,
-                                   const T* __restrict__ packed, int stride, int q_off, int k_off, int v_off, const float* __restrict__ z,
-                                   const float* __restrict__ bias, float qk_scale, float inv_tau, int nqk, int nv, int64_t total) {
-    pdl_trigger();
-    pdl_wait();
-    const int per = 3 * nqk + nv;
-    for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
-         i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
-        const int64_t t = i / per;
-        const int c = static_cast<int>(i - t * per);
-        const T* row = packed + t * stride;
-        if (c < nqk) qf[t * nqk + c] = to_float(row[q_off + c]) * qk_scale;
-        else if (c < 2 * nqk) kf[t * nqk + c - nqk] = to_float(row[k_off + c - nqk]);
-        else if (c < 3 * nqk) gg[t * nqk + c - 2 * nqk] = root_of_sigmoid(z[t * nqk + c - 2 * nqk] + bias[c - 2 * nqk], inv_tau);
-        else vf[t * nv + c - 3 * nqk] = to_float(row[v_off + c - 3 * nqk]);
-    }
-}
-
-// One token per request.  The block's threads are laid out as rows of S by groups of V neighbouring columns (V = 4 where the
-// value size allows 16-byte accesses): a thread updates its columns of every R-th row, adds its part of S^T q up in registers,
-// and the R partial sums of a column meet in shared memory in a fixed order.
-constexpr int kLinearThreads = 256;
-
-template <typename T, int V>
-__global__ void __launch_bounds__(kLinearThreads)
-linear_step_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ packed, int stride, int q_off, int k_off, int v_off, int g_off,
-                   int a_off, int rank, const T* __restrict__ wa2, const float* __restrict__ a2_bias, float qk_scale, float inv_tau,
-                   const float* __restrict__ norm_w, float eps, float out_scale, float* __restrict__ state, int64_t state_floats,
-                   const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, int num_slots, int dk, int dv,
-                   int* __restrict__ err) {
-    pdl_trigger();
-    pdl_wait();
-    extern __shared__ __align__(16) float sm[];
-    __shared__ float scratch[32];
-    const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
-    const int slot = state_slots[s];
-    if (slot < 0 || slot >= num_slots) {
-        if (tid == 0) atomicExch(err, 2);
-        return;
-    }
-    float* qs = sm;                                      // [dk] each
-    float* ks = qs + dk;
-    float* as = ks + dk;
-    float* lo = as + dk;                                 // [rank]
-    float* part = lo + rank;                             // [R, dv]
-    const int nvec = (dv + V - 1) / V;
-    const int R = nvec < kLinearThreads ? kLinearThreads / nvec : 1;      // rows worked on side by side
-    const int64_t t = cu_seqlens[s];
-    const T* row = packed + t * stride;
-    for (int i = tid; i < rank; i += kLinearThreads) lo[i] = to_float(row[a_off + i]);
-    for (int i = tid; i < dk; i += kLinearThreads) {
-        qs[i] = to_float(row[q_off + h * dk + i]) * qk_scale;
-        ks[i] = to_float(row[k_off + h * dk + i]);
-    }
-    __syncthreads();
-    for (int i = tid; i < dk; i += kLinearThreads) {
-        const T* w = wa2 + static_cast<int64_t>(h * dk + i) * rank;
-        float z = 0.f;
-        for (int r = 0; r < rank; ++r) z = fmaf(to_float(w[r]), lo[r], z);
-        as[i] = root_of_sigmoid(z + a2_bias[h * dk + i], inv_tau);
-    }
-    __syncthreads();
-    float* st = state + static_cast<int64_t>(slot) * state_floats + static_cast<int64_t>(h) * dk * dv;
-    const int rg = tid / nvec;
-    for (int cv = nvec < kLinearThreads ? tid - rg * nvec : tid; cv < nvec; cv += (nvec < kLinearThreads ? nvec : kLinearThreads)) {
-        if (nvec < kLinearThreads && rg >= R) break;
-        const int first = nvec < kLinearThreads ? rg : 0;
-        float v[V], o[V];
-#pragma unroll
-        for (int j = 0; j < V; ++j) { v[j] = cv * V + j < dv ? to_float(row[v_off + h * dv + cv * V + j]) : 0.f; o[j] = 0.f; }
-#pragma unroll 4
-        for (int i = first; i < dk; i += R) {
-            float* p = st + static_cast<int64_t>(i) * dv + cv * V;
-            const float a = as[i], k = ks[i], q = qs[i];
-            if constexpr (V == 4) {
-                float4 x = *reinterpret_cast<const float4*>(p);
-                x.x = fmaf(a, x.x, k * v[0]); x.y = fmaf(a, x.y, k * v[1]); x.z = fmaf(a, x.z, k * v[2]); x.w = fmaf(a, x.w, k * v[3]);
-                o[0] = fmaf(q, x.x, o[0]); o[1] = fmaf(q, x.y, o[1]); o[2] = fmaf(q, x.z, o[2]); o[3] = fmaf(q, x.w, o[3]);
-                *reinterpret_cast<float4*>(p) = x;
-            } else {
-                const float x = fmaf(a, p[0], k * v[0]);
-                o[0] = fmaf(q, x, o[0]);
-                p[0] = x;
-            }
-        }
-#pragma unroll
-        for (int j = 0; j < V; ++j)
-            if (cv * V + j < dv) part[first * dv + cv * V + j] = o[j];
-    }
-    __syncthreads();
-    float ss = 0.f;
-    for (int j = tid; j < dv; j += kLinearThreads) {
-        float o = 0.f;
-        for (int r = 0; r < R; ++r) o += part[r * dv + j];
-        part[j] = o;                                     // a column is added up and read back by one thread
-        ss = fmaf(o, o, ss);
-    }
-    ss = block_sum(ss, scratch);
-    const float inv = out_scale / sqrtf(ss / static_cast<float>(dv) + eps);
-    for (int j = tid; j < dv; j += kLinearThreads) {
-        const float g = to_float(row[g_off + h * dv + j]);
-        out[t * out_stride + h * dv + j] = from_float<T>(part[j] * inv * norm_w[j] * silu_of(g));
     }
 }
 
@@ -406,7 +290,7 @@ template <int KPT, int MODE>
 static int launch_scan(float* out, const float* qn, const float* kn, const float* vv, const float* gg, const float* bb, const float* decay,
                        float* state, int64_t state_floats, const int* cu_seqlens, const int* state_slots, int num_slots, int S, int H, int G,
                        int dk, int dv, int* err_flag, cudaStream_t stream) {
-    constexpr int arrays = MODE == 1 || MODE == 3 ? 3 : 2;
+    constexpr int arrays = MODE == 1 ? 3 : 2;
     const size_t smem = static_cast<size_t>(2) * (arrays * kScanChunk * KPT * kScanLanes + kScanChunk * kScanCols + 2 * kScanChunk) * sizeof(float);
     static bool raised = false;
     if (smem > 48 * 1024 && !raised) {
@@ -448,61 +332,6 @@ extern "C" int cvb_lightning_scan(float* out, const float* qf, const float* kf, 
                                                    num_slots, S, H, H, dk, dv, err_flag, stream)
     CVB_DISPATCH_KPT(dk, CALL_K);
 #undef CALL_K
-}
-
-extern "C" int cvb_linear_prep(float* qf, float* kf, float* vf, float* gg, const void* packed, int T, int stride, int q_off, int k_off,
-                               int v_off, const float* z, const float* bias, float qk_scale, float inv_tau, int nqk, int nv, int dtype,
-                               cudaStream_t stream) {
-    if (T == 0) return CVB_OK;
-    if (T < 0 || nqk <= 0 || nv <= 0) return CVB_E_SIZE;
-    if (q_off < 0 || k_off < 0 || v_off < 0 || stride < q_off + nqk || stride < k_off + nqk || stride < v_off + nv) return CVB_E_SHAPE;
-    const int64_t total = static_cast<int64_t>(T) * (3 * nqk + nv);
-    const int64_t want = (total + 255) / 256;
-    const unsigned blocks = static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16);
-#define CALL(TY) launch_kernel(linear_prep_kernel<TY>, dim3(blocks), dim3(256), 0, stream, qf, kf, vf, gg, (const TY*)packed, stride, q_off, \
-                               k_off, v_off, z, bias, qk_scale, inv_tau, nqk, nv, total)
-    CVB_DISPATCH_DTYPE(dtype, CALL);
-#undef CALL
-    return launch_status();
-}
-
-extern "C" int cvb_linear_scan(float* out, const float* qf, const float* kf, const float* vf, const float* gg, float* state,
-                               int64_t state_floats, const int* cu_seqlens, const int* state_slots, int num_slots, int S, int H, int dk,
-                               int dv, int* err_flag, cudaStream_t stream) {
-    if (S == 0) return CVB_OK;
-    if (S < 0 || H <= 0 || H > 65535 || dk <= 0 || dk > 512 || dv <= 0 || num_slots <= 0) return CVB_E_SIZE;
-    if (state_floats < static_cast<int64_t>(H) * dk * dv) return CVB_E_SHAPE;
-    if (!aligned16(qf) || !aligned16(kf) || !aligned16(vf) || !aligned16(gg)) return CVB_E_ALIGN;
-#define CALL_K(KPT) return launch_scan<KPT, 3>(out, qf, kf, vf, gg, nullptr, nullptr, state, state_floats, cu_seqlens, state_slots, \
-                                               num_slots, S, H, H, dk, dv, err_flag, stream)
-    if (dk > 256) { CALL_K(64); }
-    CVB_DISPATCH_KPT(dk, CALL_K);
-#undef CALL_K
-}
-
-extern "C" int cvb_linear_step(void* out, int out_stride, const void* packed, int stride, int q_off, int k_off, int v_off, int g_off, int a_off,
-                               int rank, const void* wa2, const float* a2_bias, float qk_scale, float inv_tau, const float* norm_w, float eps,
-                               float out_scale, float* state, int64_t state_floats, const int* cu_seqlens, const int* state_slots,
-                               int num_slots, int S, int H, int dk, int dv, int dtype, int* err_flag, cudaStream_t stream) {
-    if (S == 0) return CVB_OK;
-    if (S < 0 || H <= 0 || H > 65535 || dk <= 0 || dv <= 0 || rank <= 0 || num_slots <= 0) return CVB_E_SIZE;
-    if (state_floats < static_cast<int64_t>(H) * dk * dv || out_stride < H * dv) return CVB_E_SHAPE;
-    for (int off : {q_off, k_off}) if (off < 0 || stride < off + H * dk) return CVB_E_SHAPE;
-    for (int off : {v_off, g_off}) if (off < 0 || stride < off + H * dv) return CVB_E_SHAPE;
-    if (a_off < 0 || stride < a_off + rank) return CVB_E_SHAPE;
-    const bool four = dv % 4 == 0 && (state_floats & 3) == 0 && aligned16(state);
-    const int V = four ? 4 : 1, nvec = (dv + V - 1) / V, R = nvec < kLinearThreads ? kLinearThreads / nvec : 1;
-    const size_t smem = (static_cast<size_t>(3) * dk + rank + static_cast<size_t>(R) * dv) * sizeof(float);
-    if (smem > 48 * 1024) return CVB_E_SIZE;
-#define CALL_V(TY, VV)                                                                                                        \
-    launch_kernel(linear_step_kernel<TY, VV>, dim3(S, H), dim3(kLinearThreads), smem, stream, (TY*)out, out_stride, (const TY*)packed, stride, \
-                  q_off, k_off, v_off, g_off, a_off, rank, (const TY*)wa2, a2_bias, qk_scale, inv_tau, norm_w, eps, out_scale, state,          \
-                  state_floats, cu_seqlens, state_slots, num_slots, dk, dv, err_flag)
-#define CALL(TY) if (four) { CALL_V(TY, 4); } else { CALL_V(TY, 1); }
-    CVB_DISPATCH_DTYPE(dtype, CALL);
-#undef CALL
-#undef CALL_V
-    return launch_status();
 }
 
 extern "C" int cvb_delta_prep(float* qn, float* kn, float* vv, float* gg, float* bb, const void* packed, int T, int stride, int qkv_off,

@@ -328,6 +328,62 @@ gated_norm_kernel(T* __restrict__ out, const float* __restrict__ o, const T* __r
     }
 }
 
+// Groups of up to 512 floats in steps of four whose rows start on 16 bytes: a warp per (token, group), the group in registers.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_norm_vec_kernel(T* __restrict__ out, const float* __restrict__ o, const T* __restrict__ gate, int gate_stride,
+                      const float* __restrict__ w, int64_t n_groups, int groups, int G, float eps, int gate_act, int out_stride) {
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const int64_t id = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+    if (id >= n_groups) return;
+    const int64_t row = id / groups;
+    const int g = static_cast<int>(id - row * groups);
+    const float* og = o + id * G;
+    const T* gg = gate + row * gate_stride + g * G;
+    T* dst = out + row * out_stride + g * G;
+    float4 v[4];
+    float z[4][4];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const int j = (lane + 32 * k) * 4;
+        if (j < G) {
+            v[k] = *reinterpret_cast<const float4*>(og + j);
+            if constexpr (sizeof(T) == 2) {
+                const uint2 raw = *reinterpret_cast<const uint2*>(gg + j);
+                const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+                z[k][0] = a.x; z[k][1] = a.y; z[k][2] = b.x; z[k][3] = b.y;
+            } else {
+                const float4 a = *reinterpret_cast<const float4*>(gg + j);
+                z[k][0] = a.x; z[k][1] = a.y; z[k][2] = a.z; z[k][3] = a.w;
+            }
+            ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+        }
+    }
+    ss = warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / static_cast<float>(G) + eps);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const int j = (lane + 32 * k) * 4;
+        if (j >= G) break;
+        const float4 ww = *reinterpret_cast<const float4*>(w + j);
+        const float x[4] = {v[k].x * inv * ww.x, v[k].y * inv * ww.y, v[k].z * inv * ww.z, v[k].w * inv * ww.w};
+        float y[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] = x[e] * (gate_act ? z[k][e] : 1.f) * (1.f / (1.f + expf(-z[k][e])));
+        if constexpr (sizeof(T) == 2) {
+            uint2 raw;
+            *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(y[0], y[1]);
+            *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(y[2], y[3]);
+            *reinterpret_cast<uint2*>(dst + j) = raw;
+        } else {
+            *reinterpret_cast<float4*>(dst + j) = make_float4(y[0], y[1], y[2], y[3]);
+        }
+    }
+}
+
 // src row t holds, from column col0 on, `heads` vectors of `width` elements; they land at
 // pages[slot / page_size, head, slot % page_size, :].
 template <typename T>
@@ -454,6 +510,18 @@ extern "C" int cvb_gated_norm(void* out, const float* o, const void* gate, int g
     if (gate_stride < groups * G || out_stride < groups * G) return CVB_E_SHAPE;
     if (groups > 65535) return CVB_E_SIZE;
     const int per_block = kUpdateThreads / 32;
+    // whole groups of four elements that start on 16 bytes (8 bytes of a bf16 row)
+    const uintptr_t ab = dtype == CVB_DTYPE_BF16 ? 7 : 15;
+    const bool vec = G % 4 == 0 && G <= 512 && gate_stride % 4 == 0 && out_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0
+                     && (reinterpret_cast<uintptr_t>(w) & 15) == 0 && ((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & ab) == 0;
+    const int64_t n_groups = static_cast<int64_t>(T) * groups;
+    if (vec && (n_groups + 7) / 8 <= 2147483647LL) {
+#define CALL(TY) launch_kernel(gated_norm_vec_kernel<TY>, dim3(static_cast<unsigned>((n_groups + 7) / 8)), dim3(256), 0, stream, (TY*)out, o,   \
+                               (const TY*)gate, gate_stride, w, n_groups, groups, G, eps, gate_act, out_stride)
+        CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+        return launch_status();
+    }
 #define CALL(TY)                                                                                                                 \
     if (G > 256) launch_kernel(gated_norm_block_kernel<TY>, dim3(T, groups), dim3(kUpdateThreads), 0, stream, (TY*)out, o,       \
                                (const TY*)gate, gate_stride, w, groups, G, eps, gate_act, out_stride);                                                 \

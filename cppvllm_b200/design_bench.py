@@ -39,6 +39,17 @@ gated experts, 2 per token, of half the inner size, whose logistic scores multip
 size.  Whole models stand beside Givirax (the closest existing model: a float32 stream, attention over cache entries behind a
 window, routed gated experts) and Qwen3; its kernels beside the like kernels of Lorulix (attention over entries of a key and its
 value), Givirax (the stream update, the router, the experts), Qwen3 (the projection's epilogue) and Dugulorn (the gate).
+
+    python bench.py --design sumevik
+
+The Sumevik model of a size has the same width, heads and head size; its layers repeat the pattern [gated recurrence with a dense
+tanh-GELU gate, chunked attention beside gated linear attention with experts]: as many channels as the width in parts of 256, 4 taps;
+chunks of 1,024 positions, every element turned, a gate per element; linear attention of as many heads with 64 x 128 of state each
+(the query/key size half the value size); 8 clamped experts of half the inner size and 2 identity outputs in 2 groups, 2 per token
+from the best group.  Whole models stand beside Lorulix (the closest existing model: a float32 stream, attention over entries of a key
+and its value, a mixer with a matrix of state per head, dense and routed feed-forwards) and Qwen3; its kernels beside the like kernels
+of Rumurax (attention, the projection's epilogue, the router), Dugulorn and Lorulix (scans, convolution, preparation), Givirax
+(experts), Qwen3 (the gated product) and the weight-streaming product (the recurrence of decoded tokens, which reads gate matrices).
 """
 from __future__ import annotations
 
@@ -131,6 +142,21 @@ def rumurax_config(s, max_positions):
     pattern = [windowed, chunked, latent, chunked]
     return {"architecture": "Rumurax", "vocab": s["vocab"], "width": s["width"], "streams": 2, "norm": {"eps": 1e-5},
             "layers": [dict(pattern[i % 4], mlp=moe) for i in range(s["layers"])]}
+
+
+SV_CHUNK, SV_PART, SV_IDENTITY = 1024, 256, 2
+
+
+def sumevik_config(s, max_positions):
+    D, H, KV, hd, I = s["width"], s["heads"], s["kv_heads"], s["dim"], s["ff"]
+    recurrence = {"type": "rglru", "mixer": {"width": D, "conv": 4, "blocks": D // SV_PART}, "mlp": {"kind": "dense", "ff": I}}
+    pair = {"type": "parallel", "mixer": {
+        "left": {"dim": hd, "heads": H, "kv_heads": KV, "vdim": hd, "scale": 1.0 / math.sqrt(hd), "mask": {"size": SV_CHUNK}, "rot": {"dims": hd, "base": 1.0e6}},
+        "right": {"dim": hd // 2, "heads": H, "vdim": hd, "tau": 16.0, "a_rank": 16}, "left_scale": 0.7, "right_scale": 0.9},
+        "mlp": {"kind": "moe", "expert": {"ff": I // 2, "limit": 7.0},
+                "router": {"experts": EXPERTS, "top": TOP, "groups": {"count": 2, "keep": 1}, "identity": SV_IDENTITY}}}
+    return {"architecture": "Sumevik", "vocab": s["vocab"], "width": D, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+            "layers": [(recurrence, pair)[i % 2] for i in range(s["layers"])]}
 
 
 def qwen3_config(s, max_positions):
@@ -823,9 +849,200 @@ def rumurax_kernel_pairs(s, pk):
     return out
 
 
+def sumevik_kernel_pairs(s, pk):
+    """The kernels that the Sumevik parts brought, each beside the like kernel of an existing model at the same sizes (`like`
+    names it)."""
+    from .csrc import ops
+    from .parts.base import Workspace
+    d = torch.device("cuda:0")
+    g = torch.Generator(device="cuda").manual_seed(0)
+    bf, f32, i32 = torch.bfloat16, torch.float32, torch.int32
+    D, H, KV, hd, I = s["width"], s["heads"], s["kv_heads"], s["dim"], s["ff"]
+    F, dk = I // 2, s["dim"] // 2
+    page, out = 32, {}
+    hbm, flop = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+
+    def rnd(*shape, scale=1.0, dtype=bf):
+        return (torch.randn(*shape, generator=g, device=d, dtype=f32) * scale).to(dtype)
+
+    def pair(name, new_us, new_work, like_us, like_work, unit, like, note=None):
+        peak = hbm if unit == "bytes" else flop
+        fn, fl = new_work / (new_us * 1e-6) / peak, like_work / (like_us * 1e-6) / peak
+        out[name] = {"new_us": round(new_us, 2), "new_frac": round(fn, 4), "like_us": round(like_us, 2), "like_frac": round(fl, 4),
+                     "gap": round(fl / fn, 2), "roofline": "copy bandwidth" if unit == "bytes" else "bf16 peak", "like": like}
+        if note:
+            out[name]["note"] = note
+
+    # -- chunked attention: a prompt of 2,048 tokens, 8 decoded tokens ------------------------------------------------------
+    T, B = 2048, 8
+    n_pages = T // page
+    tables = torch.arange(n_pages, dtype=i32, device=d).view(1, n_pages)
+    cu, pos, slot0 = torch.tensor([0, T], dtype=i32, device=d), torch.arange(T, dtype=i32, device=d), torch.zeros(1, dtype=i32, device=d)
+    seq_of = torch.zeros(T, dtype=i32, device=d)
+    cu_b, pos_b = torch.arange(0, B + 1, dtype=i32, device=d), torch.full((B,), 4095, dtype=i32, device=d)
+    slots_b, seq_b = torch.arange(0, B, dtype=i32, device=d), torch.arange(0, B, dtype=i32, device=d)
+    scale = 1 / math.sqrt(hd)
+    q, att, gate_e, gate_h = rnd(T, H * hd), torch.empty(T, H * hd, dtype=bf, device=d), rnd(T, H * hd), rnd(T, H)
+    tiles = ops.attn_keys_tiles([T], H, KV)
+    ent = rnd(n_pages + 1, KV, page, 2 * hd)
+    kw = dict(chunk=SV_CHUNK)
+    new = _us(lambda i: ops.attn_masked_bf16(att, q, ent, tables, cu, pos, 1, tiles, H, KV, hd, hd, page, scale, gate=gate_e, out_scale=0.7, **kw))
+    like = _us(lambda i: ops.attn_masked_bf16(att, q, ent, tables, cu, pos, 1, tiles, H, KV, hd, hd, page, scale, gate=gate_h, **kw))
+    flops = 4.0 * H * hd * sum(p % SV_CHUNK + 1 for p in range(T))
+    pair("attention_chunked_prefill_2048", new, flops, like, flops, "flops", "Rumurax attn_masked_kernel, gate per head")
+    copies, ctx = 4, 4096
+    pps = ctx // page
+    tabs = [torch.randperm(B * pps, generator=g, device=d).to(i32).view(B, pps).contiguous() for _ in range(copies)]
+    ents = [rnd(B * pps + 1, KV, page, 2 * hd) for _ in range(copies)]
+    z = ops.attn_masked_decode_splits(B, KV, SV_CHUNK)
+    parts = torch.empty(max(1, ops.attn_keys_scratch_floats(B, KV, hd, z)), dtype=f32, device=d)
+    run = lambda gate: _us(lambda i: ops.attn_masked_bf16(att[:B], q[:B], ents[i % copies], tabs[i % copies], cu_b, pos_b, B, B, H, KV, hd, hd,   # noqa: E731
+                                                          page, scale, gate=gate, all_single=True, splits=z, scratch=parts, **kw))
+    new, like = run(gate_e[:B]), run(gate_h[:B])
+    seen = B * SV_CHUNK * KV * hd * 4.0
+    pair("attention_chunked_decode_b8", new, seen, like, seen, "bytes", "Rumurax attn_masked_decode_kernel, gate per head", note="the last token of a chunk")
+    del ents
+    n_left = (H + 2 * KV) * hd
+    packed, q_out, w1 = rnd(T, n_left), torch.empty(T, H * hd, dtype=bf, device=d), torch.ones(hd, device=d)
+    cos, sin = torch.rand(T, hd // 2, generator=g, device=d), torch.rand(T, hd // 2, generator=g, device=d)
+    bias = rnd(n_left, dtype=f32)
+    prep = lambda b: _us(lambda i: ops.masked_qkv_prep(q_out, packed, H, KV, hd, hd, 1e-5, q_weight=w1, k_weight=w1, cos=cos, sin=sin, rot=hd,   # noqa: E731
+                                                       positions=pos, pages=ent, slots=pos, page_size=page, bias=b))
+    new, like = prep(bias), prep(None)
+    pair("projection_epilogue_2048_tokens", new, T * n_left * 4.0, like, T * n_left * 4.0, "bytes", "Rumurax masked_qkv_prep, no biases")
+
+    # -- gated linear attention: dk = hd / 2 rows and hd columns of state per head -----------------------------------------
+    HK, HV = H * dk, H * hd
+    R = 16
+    lin = rnd(T, 2 * HK + 2 * HV + R)
+    wa2, ab, wn = rnd(HK, R, scale=0.1), rnd(HK, dtype=f32), torch.ones(hd, device=d)
+    qf, kf, zz = (torch.zeros(T, HK, dtype=f32, device=d) for _ in range(3))
+    vf, o32 = torch.zeros(T, HV, dtype=f32, device=d), torch.empty(T, HV, dtype=f32, device=d)
+    y_lin = torch.empty(T, HV, dtype=bf, device=d)
+    state = torch.zeros(2, H * dk * hd, dtype=f32, device=d)
+    chunk = ops.linear_chunk_tokens(T, H, hd)
+    held = ops.linear_held_chunks(T, H, hd)
+    ends, decays = torch.empty(held * H * dk * hd, dtype=f32, device=d), torch.empty(held * H * dk, dtype=f32, device=d)
+
+    def core(i):                                 # as parts/recurrent.py does for portions of prompts
+        ops.linear(lin[:, 2 * HK + 2 * HV:], wa2, out=zz, out_dtype=f32)
+        ops.linear_decay(zz, ab, 16.0)
+        ops.linear_scan(o32, lin, 0, HK, 2 * HK, dk ** -0.5, zz, state, cu, slot0, [T], H, dk, hd, chunk, ends, decays)
+        ops.gated_norm(y_lin, o32, lin[:, 2 * HK + HV:2 * HK + 2 * HV], wn, H, 1e-5, gate_act="silu")
+    new = _us(core)
+    # Dugulorn's channel-delta mixer over the same heads and sizes, from its packed projection to its normed output
+    C = 2 * HK + HV
+    raw, conv_w = rnd(T, C), rnd(C, 4, dtype=f32)
+    st_delta = torch.zeros(2, H * dk * hd + 3 * C, dtype=f32, device=d)
+    a32, b32, bb = rnd(T, HK, dtype=f32), rnd(T, H, dtype=f32), torch.empty(T, H, dtype=f32, device=d)
+    dt, alog, gate16 = rnd(HK, dtype=f32), rnd(H, dtype=f32), rnd(T, HV)
+
+    def delta(i):
+        ops.delta_prep(qf, kf, vf, zz, bb, raw, 0, conv_w, a32, dt, alog, b32, st_delta, H * dk * hd, seq_of, cu, slot0, H, H, dk, hd)
+        ops.conv_history(st_delta, H * dk * hd, raw, 0, C, 4, cu, slot0, 1)
+        ops.delta_scan(o32, qf, kf, vf, zz, bb, st_delta, cu, slot0, 1, H, H, dk, hd)
+        ops.gated_norm(y_lin, o32, gate16, wn, H, 1e-5)
+    like = _us(delta)
+    pair("linear_attention_core_2048_tokens", new, 4.0 * H * dk * hd * T, like, 6.0 * H * dk * hd * T, "flops",
+         "Dugulorn channel delta, the same span", note="from the packed projection to the gated, normed output; four flops an element of state and token (six)")
+    Bs = B
+    n_copy = max(2, int(300e6 // (Bs * H * dk * hd * 4)) + 1)
+    states = [torch.zeros(Bs + 1, H * dk * hd, dtype=f32, device=d) for _ in range(n_copy)]
+    new = _us(lambda i: ops.linear_step(y_lin[:Bs], lin[:Bs], 0, HK, 2 * HK, 2 * HK + HV, 2 * HK + 2 * HV, wa2, ab, dk ** -0.5, 16.0, wn, 1e-5, 0.9,
+                                        states[i % n_copy], cu_b, slots_b, Bs, H, dk, hd))
+    sdel = [torch.zeros(Bs + 1, H * dk * hd + 3 * C, dtype=f32, device=d) for _ in range(n_copy)]
+
+    def delta_b(i):
+        st = sdel[i % n_copy]
+        ops.delta_prep(qf[:Bs], kf[:Bs], vf[:Bs], zz[:Bs], bb[:Bs], raw[:Bs], 0, conv_w, a32[:Bs], dt, alog, b32[:Bs], st, H * dk * hd, seq_b, cu_b, slots_b, H, H, dk, hd)
+        ops.conv_history(st, H * dk * hd, raw[:Bs], 0, C, 4, cu_b, slots_b, Bs)
+        ops.delta_scan(o32[:Bs], qf[:Bs], kf[:Bs], vf[:Bs], zz[:Bs], bb[:Bs], st, cu_b, slots_b, Bs, H, H, dk, hd)
+        ops.gated_norm(y_lin[:Bs], o32[:Bs], gate16[:Bs], wn, H, 1e-5)
+    like = _us(delta_b)
+    pair("linear_attention_decode_b8", new, Bs * H * dk * hd * 8.0, like, Bs * H * dk * hd * 8.0, "bytes", "Dugulorn channel delta, the same span")
+    del states, sdel
+
+    # -- gated recurrence over channels --------------------------------------------------------------------------------------
+    W, P = D, D // SV_PART
+    lru_in = rnd(T, 2 * W)
+    u, o_lru = torch.empty(T, W, dtype=bf, device=d), torch.empty(T, W, dtype=bf, device=d)
+    zg = torch.empty(P, T, 2 * SV_PART, dtype=f32, device=d)
+    gates = rnd(P, 2 * SV_PART, SV_PART, scale=0.05)
+    by, bx, cb, br, bi = (rnd(W, dtype=f32) for _ in range(5))
+    cw, nsp = rnd(4, W, dtype=f32), -torch.rand(W, generator=g, device=d) * 0.1
+    st_l = torch.zeros(2, 5 * W, dtype=f32, device=d)
+    summary = torch.empty(2 * W * (T // 16 + 2), dtype=f32, device=d)
+    L = ops.lru_chunk_tokens(T)
+    new = _us(lambda i: ops.lru_conv(u, lru_in, 0, W, P, bx, cw, cb, st_l, seq_of, cu, slot0, pos))
+    a_in, hist = rnd(T, W), torch.zeros(2, 3 * W, dtype=f32, device=d)
+    like = _us(lambda i: ops.input_conv(o_lru, a_in, cw, hist, 0, seq_of, cu, slot0))
+    pair("convolution_2048_tokens", new, T * W * 4.0, like, T * W * 4.0, "bytes", "Lorulix input_conv")
+    new = _us(lambda i: ops.lru_scan(o_lru, zg, u, lru_in, 0, W, P, 4, by, bx, br, bi, nsp, st_l, cu, slot0, pos, [T], L, summary))
+    v_d = torch.full((H,), 0.9, device=d)
+    l_us = _us(lambda i: ops.lightning_scan(o32, qf, kf, vf, state, v_d, cu, slot0, 1, H, dk, hd))
+    pair("recurrence_2048_tokens", new, T * W * 14.0, l_us, T * (2 * HK + 2 * HV) * 4.0, "bytes", "Dugulorn lightning_scan, the bytes of its rows",
+         note="gate products in float32 (8), u, y and the output in bf16 (6)")
+
+    def lru_all(i):
+        ops.lru_conv(u, lru_in, 0, W, P, bx, cw, cb, st_l, seq_of, cu, slot0, pos)
+        ops.lru_gates(zg, u, gates)
+        ops.lru_scan(o_lru, zg, u, lru_in, 0, W, P, 4, by, bx, br, bi, nsp, st_l, cu, slot0, pos, [T], L, summary)
+    new = _us(lru_all)
+    pair("recurrence_core_2048_tokens", new, T * W * 6.0, like=
+         "Dugulorn channel delta, the bytes of its rows", like_us=_us(delta), like_work=T * (C + 2 * HV) * 2.0 + T * HK * 4.0, unit="bytes",
+         note="convolution, gate products, scan: both projections read, one output written")
+    n_copy = max(2, int(300e6 // (gates.numel() * 2)) + 1)
+    gs = [gates.clone() for _ in range(n_copy)]
+    st8 = torch.zeros(Bs + 1, 5 * W, dtype=f32, device=d)
+    new = _us(lambda i: ops.lru_step(o_lru[:Bs], lru_in[:Bs], 0, W, by, bx, cw, cb, gs[i % n_copy], br, bi, nsp, st8, cu_b, slots_b, pos_b, Bs))
+    w_like = [rnd(2 * W, SV_PART, scale=0.05) for _ in range(n_copy)]
+    x_like, y_like = rnd(Bs, SV_PART), torch.empty(Bs, 2 * W, dtype=bf, device=d)
+    like = _us(lambda i: ops.gemv_bf16(y_like, x_like, w_like[i % n_copy], Bs))
+    gb = gates.numel() * 2.0
+    pair("recurrence_decode_b8", new, gb + Bs * W * (8 + 4 * 5 + 6.0), like, gb, "bytes", "gemv_bf16 over a weight of the gates' size",
+         note="gate matrices, S, ring, both projections and the output")
+    del gs, w_like
+
+    # -- feed-forwards ---------------------------------------------------------------------------------------------------------
+    x = rnd(T, D)
+    gu, act = rnd(T, 2 * I), torch.empty(T, I, dtype=bf, device=d)
+    new, like = _us(lambda i: ops.geglu(act, gu)), _us(lambda i: ops.swiglu(act, gu))
+    pair("activation_2048_tokens", new, T * I * 6.0, like, T * I * 6.0, "bytes", "Qwen3 swiglu")
+    w_gu1 = rnd(2 * I, D, scale=0.02)
+    new, like = _us(lambda i: ops.gemm_bf16_tcgen05(act, x, w_gu1, geglu=True)), _us(lambda i: ops.gemm_bf16_tcgen05(act, x, w_gu1, swiglu=True))
+    pair("gated_product_2048_tokens", new, 4.0 * T * D * I, like, 4.0 * T * D * I, "flops", "Qwen3 swiglu product (tcgen05)")
+    n_out = EXPERTS + SV_IDENTITY
+    w_router, corr = torch.randn(n_out, D, generator=g, device=d), torch.randn(n_out, generator=g, device=d) * 0.1
+    ids, wts = torch.empty(T, TOP, dtype=i32, device=d), torch.empty(T, TOP, dtype=f32, device=d)
+    ids2, wts2 = torch.empty(T, TOP, dtype=i32, device=d), torch.empty(T, TOP, dtype=f32, device=d)
+    new = _us(lambda i: ops.route_topk(ids, wts, x, w_router, corr, groups=2, keep=1))
+    like = _us(lambda i: ops.route_topk(ids2, wts2, x, w_router[:EXPERTS].contiguous(), None, logistic=True))
+    pair("router_2048_tokens", new, T * D * 2.0, like, T * D * 2.0, "bytes", "Rumurax route_topk", note="ten outputs against eight")
+    ws = Workspace(d, T)
+    w_gu, w_dn = rnd(EXPERTS, 2 * F, D, scale=0.02), rnd(EXPERTS, D, F, scale=0.02)
+    y = torch.empty(T, D, dtype=bf, device=d)
+    kw = dict(activation="clamped", identity=SV_IDENTITY, limit=7.0)
+    new = _us(lambda i: ops.routed_experts(y, x, ids, wts, w_gu, w_dn, workspace=ws, **kw))
+    like = _us(lambda i: ops.routed_experts(y, x, ids2, wts2, w_gu, w_dn, workspace=ws))
+    real = int((ids < EXPERTS).sum())
+    pair("experts_2048_tokens", new, 2.0 * real * 3 * D * F, like, 2.0 * T * TOP * 3 * D * F, "flops", "Givirax gated experts",
+         note=f"{real} of {T * TOP} pairs are experts, the others the input itself")
+    ws8 = Workspace(d, 8)
+    copies = max(2, int(300e6 // (w_gu.numel() * 2 + w_dn.numel() * 2)) + 1)
+    gus = [w_gu] + [rnd(EXPERTS, 2 * F, D, scale=0.02) for _ in range(copies - 1)]
+    dns = [w_dn] + [rnd(EXPERTS, D, F, scale=0.02) for _ in range(copies - 1)]
+    x8, y8 = x[:8].contiguous(), torch.empty(8, D, dtype=bf, device=d)
+    ids8, wts8, ids28, wts28 = ids[:8].contiguous(), wts[:8].contiguous(), ids2[:8].contiguous(), wts2[:8].contiguous()
+    new = _us(lambda i: ops.routed_experts(y8, x8, ids8, wts8, gus[i % copies], dns[i % copies], workspace=ws8, **kw))
+    like = _us(lambda i: ops.routed_experts(y8, x8, ids28, wts28, gus[i % copies], dns[i % copies], workspace=ws8))
+    used, used2 = len({e for e in ids8.flatten().tolist() if e < EXPERTS}), len(set(ids28.flatten().tolist()))
+    pair("experts_8_decoded_tokens", new, used * 3.0 * D * F * 2, like, used2 * 3.0 * D * F * 2, "bytes", "Givirax gated experts")
+    return out
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="design_bench", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--design", default="givirax", choices=["givirax", "dugulorn", "lorulix", "rumurax"])
+    ap.add_argument("--design", default="givirax", choices=["givirax", "dugulorn", "lorulix", "rumurax", "sumevik"])
     ap.add_argument("--sizes", default="small,large")
     ap.add_argument("--steps", type=int, default=48)
     ap.add_argument("--no-kernels", action="store_true", help="whole models only")
@@ -844,20 +1061,25 @@ def main(argv=None) -> int:
         result.update(closest="Givirax", bias_rows=BIAS_ROWS, bias_far=BIAS_FAR, experts=EXPERTS, top=TOP)
     if a.design == "rumurax":
         result.update(closest="Givirax", window=RX_WINDOW, pool=RX_POOL, chunk=RX_CHUNK, streams=2, experts=EXPERTS, top=TOP)
+    if a.design == "sumevik":
+        result.update(closest="Lorulix", chunk=SV_CHUNK, part=SV_PART, experts=EXPERTS, identity=SV_IDENTITY, top=TOP)
     for name in a.sizes.split(","):
         s = SIZES[name]
         entry = {"shape": s}
         if not a.no_models:
             t0 = time.time()
-            design_config = {"givirax": givirax_config, "dugulorn": dugulorn_config, "lorulix": lorulix_config, "rumurax": rumurax_config}[a.design]
+            design_config = {"givirax": givirax_config, "dugulorn": dugulorn_config, "lorulix": lorulix_config, "rumurax": rumurax_config,
+                             "sumevik": sumevik_config}[a.design]
             entry[a.design] = model_points(design_config(s, 4160), 2048, 8, 4096, a.steps)
             if a.design in ("lorulix", "rumurax"):
                 entry["givirax"] = model_points(givirax_config(s, 4160), 2048, 8, 4096, a.steps)
+            if a.design == "sumevik":
+                entry["lorulix"] = model_points(lorulix_config(s, 4160), 2048, 8, 4096, a.steps)
             entry["qwen3"] = model_points(qwen3_config(s, 4160), 2048, 8, 4096, a.steps)
             entry["seconds"] = round(time.time() - t0, 1)
         if not a.no_kernels:
             entry["kernels"] = {"givirax": kernel_pairs, "dugulorn": dugulorn_kernel_pairs, "lorulix": lorulix_kernel_pairs,
-                                "rumurax": rumurax_kernel_pairs}[a.design](s, pk)
+                                "rumurax": rumurax_kernel_pairs, "sumevik": sumevik_kernel_pairs}[a.design](s, pk)
         result["sizes"][name] = entry
     print(json.dumps(result))
     return 0

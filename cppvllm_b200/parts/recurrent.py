@@ -273,10 +273,16 @@ class GatedLinearMixer(Mixer):
         ws, f32 = self.rt.workspace, torch.float32
         # the decay's logits leave their product unrounded and become the decays in place
         z = ops.linear(packed[:, a_off:a_off + R], self.w_a2, out=ws.rows("linear_g", T, H * dk, f32), out_dtype=f32)
-        qf, kf, vf = ws.rows("delta_q", T, H * dk, f32), ws.rows("delta_k", T, H * dk, f32), ws.rows("delta_v", T, H * dv, f32)
-        ops.linear_prep(qf, kf, vf, z, packed, q_off, k_off, v_off, z, self.b_a2, qk_scale, self.tau)
+        ops.linear_decay(z, self.b_a2, self.tau)
         o = ws.rows("rec_o", T, H * dv, f32)
-        ops.linear_scan(o, qf, kf, vf, z, state, ctx.cu_seqlens, ctx.state_slots, S, H, dk, dv)
+        q_lens = ctx.q_lens if ctx.q_lens is not None else [1] * S
+        chunk = ops.linear_chunk_tokens(T, H, dv)
+        ends = decays = None
+        if max(q_lens) > chunk:
+            held = ops.linear_held_chunks(ws.max_tokens, H, dv)
+            ends = ws.flat(f"linear_ends_{H}_{dk}_{dv}", held * H * dk * dv, f32)
+            decays = ws.flat(f"linear_decays_{H}_{dk}_{dv}", held * H * dk, f32)
+        ops.linear_scan(o, packed, q_off, k_off, v_off, qk_scale, z, state, ctx.cu_seqlens, ctx.state_slots, q_lens, H, dk, dv, chunk, ends, decays)
         if self._scaled[0] != scale:                      # the constant rides on the norm's weight
             self._scaled = (scale, (self.w_norm * scale).contiguous())
         return ops.gated_norm(out, o, packed[:, g_off:g_off + H * dv], self._scaled[1], H, self.eps, gate_act="silu")
