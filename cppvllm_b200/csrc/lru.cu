@@ -74,6 +74,90 @@ lru_conv_kernel(T* __restrict__ u, const T* __restrict__ packed, const float* __
         u[t * sh.W + c] = from_float<T>(lru_conv_of(packed, bias_x, conv_w, conv_b, ring, sh, t, local, pos, c));
 }
 
+// The same by vectors: a thread owns the channels of 16 bytes over `run` neighbouring tokens of the flattened batch and slides a
+// window of K rows along; a token whose window reaches back before its portion takes the general form.
+template <typename T> struct LruVec;
+template <> struct LruVec<float> {
+    static constexpr int N = 4;
+    static __device__ __forceinline__ void load(float (&f)[4], const float* p) { const float4 v = *reinterpret_cast<const float4*>(p); f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
+    static __device__ __forceinline__ void store(float* p, const float (&f)[4]) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+};
+template <> struct LruVec<__nv_bfloat16> {
+    static constexpr int N = 8;
+    static __device__ __forceinline__ void load(float (&f)[8], const __nv_bfloat16* p) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(p);
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { const float2 v = __bfloat1622float2(h[i]); f[2 * i] = v.x; f[2 * i + 1] = v.y; }
+    }
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&f)[8]) {
+        uint4 raw;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+        *reinterpret_cast<uint4*>(p) = raw;
+    }
+};
+
+template <typename T, int K>
+__global__ void __launch_bounds__(kLruThreads)
+lru_conv_vec_kernel(T* __restrict__ u, const T* __restrict__ packed, const float* __restrict__ bias_x, const float* __restrict__ conv_w,
+                    const float* __restrict__ conv_b, const float* __restrict__ state, const int* __restrict__ seq_of_token,
+                    const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, const int* __restrict__ positions, int n_tokens,
+                    int run, LruShape sh, int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    constexpr int N = LruVec<T>::N;
+    const int c = (blockIdx.y * kLruThreads + threadIdx.x) * N;
+    if (c >= sh.W) return;
+    const int t0 = blockIdx.x * run, t1 = min(t0 + run, n_tokens);
+    float w[K][N], b[N], cb[N], x[K][N];
+#pragma unroll
+    for (int e = 0; e < N; ++e) { b[e] = bias_x[c + e]; cb[e] = conv_b[c + e]; }
+#pragma unroll
+    for (int m = 0; m < K; ++m)
+#pragma unroll
+        for (int e = 0; e < N; ++e) w[m][e] = conv_w[static_cast<int64_t>(m) * sh.W + c + e];
+    const T* base = packed + sh.x_off + c;
+#pragma unroll
+    for (int m = 1; m < K; ++m) {                       // rows t0 - K + 1 .. t0 - 1; the loop shifts them into place
+        const int t = t0 - K + m;
+        LruVec<T>::load(x[m], base + static_cast<int64_t>(max(t, 0)) * sh.stride);
+#pragma unroll
+        for (int e = 0; e < N; ++e) x[m][e] += b[e];
+    }
+    for (int t = t0; t < t1; ++t) {
+#pragma unroll
+        for (int m = 0; m + 1 < K; ++m)
+#pragma unroll
+            for (int e = 0; e < N; ++e) x[m][e] = x[m + 1][e];
+        LruVec<T>::load(x[K - 1], base + static_cast<int64_t>(t) * sh.stride);
+#pragma unroll
+        for (int e = 0; e < N; ++e) x[K - 1][e] += b[e];
+        const int s = seq_of_token[t], local = t - cu_seqlens[s];
+        float y[N];
+        if (local >= K - 1) {
+#pragma unroll
+            for (int e = 0; e < N; ++e) {
+                float acc = 0.f;
+#pragma unroll
+                for (int m = 0; m < K; ++m) acc = fmaf(w[m][e], x[m][e], acc);
+                y[e] = acc + cb[e];
+            }
+        } else {
+            const int slot = state_slots[s];
+            if (slot < 0 || slot >= sh.num_slots) {
+                atomicExch(err, 2);
+                continue;
+            }
+            const float* ring = state + static_cast<int64_t>(slot) * sh.state_floats + sh.W;
+#pragma unroll
+            for (int e = 0; e < N; ++e) y[e] = lru_conv_of(packed, bias_x, conv_w, conv_b, ring, sh, t, local, positions[t], c + e);
+        }
+        LruVec<T>::store(u + static_cast<int64_t>(t) * sh.W + c, y);
+    }
+}
+
 // Which chunk of which request block x works on: chunk k of request s holds its tokens k * len .. (at most len of them).
 __device__ __forceinline__ bool lru_locate(const int* __restrict__ cu_seqlens, int S, int len, int x, int& s_out, int& k, int& first_chunk) {
     int base = 0;
@@ -86,10 +170,32 @@ __device__ __forceinline__ bool lru_locate(const int* __restrict__ cu_seqlens, i
     return false;
 }
 
+// 1 - e^y for y <= 0: by its series where the difference would cancel
+__device__ __forceinline__ float one_minus_exp(float y) {
+    const float series = y * (1.f + y * (1.f / 2.f) * (1.f + y * (1.f / 3.f) * (1.f + y * (1.f / 4.f) * (1.f + y * (1.f / 5.f) * (1.f + y * (1.f / 6.f) * (1.f + y * (1.f / 7.f)))))));
+    return y > -0.5f ? -series : 1.f - __expf(y);
+}
+
+// The decay and the weighted input from the two gate products.  With bf16 activations through the hardware's exponential and
+// division; in the 32-bit path through the library's functions.
+template <typename T>
 __device__ __forceinline__ void lru_gate(float zr, float zi, float br, float bi, float nsp, float u, float& a, float& in) {
-    const float l = lru_sigmoid(zr + br) * nsp;
-    a = expf(l);
-    in = sqrtf(fmaxf(-expm1f(2.f * l), 0.f)) * lru_sigmoid(zi + bi) * u;
+    if constexpr (sizeof(T) == 2) {
+        const float l = __fdividef(nsp, 1.f + __expf(-(zr + br)));
+        a = __expf(l);
+        in = __fsqrt_rn(fmaxf(one_minus_exp(2.f * l), 0.f)) * __fdividef(u, 1.f + __expf(-(zi + bi)));
+    } else {
+        const float l = lru_sigmoid(zr + br) * nsp;
+        a = expf(l);
+        in = sqrtf(fmaxf(-expm1f(2.f * l), 0.f)) * lru_sigmoid(zi + bi) * u;
+    }
+}
+
+// gelu_tanh: z / 2 (1 + tanh(s)) = z sigmoid(2 s)
+template <typename T>
+__device__ __forceinline__ float lru_gelu_of(float z) {
+    if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-2.f * 0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    else return lru_gelu(z);
 }
 
 template <typename T>
@@ -117,10 +223,10 @@ lru_chunk_kernel(float* __restrict__ z, const T* __restrict__ u, const float* __
     float A = 1.f, B = 0.f;
     if (k == 0) { B = state[static_cast<int64_t>(slot) * sh.state_floats + c]; }
     const float start = B;
-#pragma unroll 4
+#pragma unroll 8
     for (int i = 0; i < n; ++i) {
         float a, in;
-        lru_gate(zp[static_cast<int64_t>(i) * 2 * sh.part], zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part], rb, ib, ns,
+        lru_gate<T>(zp[static_cast<int64_t>(i) * 2 * sh.part], zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part], rb, ib, ns,
                  to_float(up[static_cast<int64_t>(i) * sh.W]), a, in);
         zp[static_cast<int64_t>(i) * 2 * sh.part] = a;
         zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part] = in;
@@ -172,12 +278,12 @@ lru_finish_kernel(T* __restrict__ out, const float* __restrict__ z, const T* __r
         }
     }
     const float rb = GATED ? br[c] : 0.f, ib = GATED ? bi[c] : 0.f, ns = GATED ? nsp[c] : 0.f, yb = bias_y[c];
-#pragma unroll 4
+#pragma unroll 8
     for (int i = 0; i < n; ++i) {
         float a = zp[static_cast<int64_t>(i) * 2 * sh.part], in = zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part];
-        if (GATED) lru_gate(a, in, rb, ib, ns, to_float(up[static_cast<int64_t>(i) * sh.W]), a, in);
+        if (GATED) lru_gate<T>(a, in, rb, ib, ns, to_float(up[static_cast<int64_t>(i) * sh.W]), a, in);
         st = fmaf(a, st, in);
-        op[static_cast<int64_t>(i) * sh.W] = from_float<T>(st * lru_gelu(to_float(yp[static_cast<int64_t>(i) * sh.stride]) + yb));
+        op[static_cast<int64_t>(i) * sh.W] = from_float<T>(st * lru_gelu_of<T>(to_float(yp[static_cast<int64_t>(i) * sh.stride]) + yb));
     }
     if (t0 + n == end) {
         row[c] = st;
@@ -191,7 +297,7 @@ lru_finish_kernel(T* __restrict__ out, const float* __restrict__ z, const T* __r
 
 constexpr int kStepThreads = 256;
 constexpr int kStepTokens = 8;          // requests per block
-constexpr int kStepChannels = 16;       // channels per block: two per warp
+constexpr int kStepWarps = kStepThreads / 32;
 
 __device__ __forceinline__ void fma8(const __nv_bfloat16* w, float (&f)[8]) {
     const uint4 raw = *reinterpret_cast<const uint4*>(w);
@@ -205,44 +311,95 @@ __device__ __forceinline__ void fma8(const float* w, float (&f)[8]) {
 }
 
 // gates [parts, 2 * part, part]: the rows of Ra over the rows of Ri
-template <typename T, int NT>
+// NT requests a block; K > 0: that many taps, known to the compiler
+template <typename T, int NT, int K>
 __global__ void __launch_bounds__(kStepThreads)
 lru_step_kernel(T* __restrict__ out, const T* __restrict__ packed, const float* __restrict__ bias_y, const float* __restrict__ bias_x,
                 const float* __restrict__ conv_w, const float* __restrict__ conv_b, const T* __restrict__ gates, const float* __restrict__ br,
                 const float* __restrict__ bi, const float* __restrict__ nsp, float* __restrict__ state, const int* __restrict__ cu_seqlens,
-                const int* __restrict__ state_slots, const int* __restrict__ positions, int S, LruShape sh, int vec, int* __restrict__ err) {
+                const int* __restrict__ state_slots, const int* __restrict__ positions, int S, LruShape sh, int vec, int per_warp, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float us[];         // [NT][ld]
-    const int per_part = (sh.part + kStepChannels - 1) / kStepChannels;
-    const int b = blockIdx.x / per_part, o0 = (blockIdx.x - b * per_part) * kStepChannels;
+    const int chans = kStepWarps * per_warp;            // channels of the block: a warp takes every eighth of them
+    const int per_part = (sh.part + chans - 1) / chans;
+    const int b = blockIdx.x / per_part, o0 = (blockIdx.x - b * per_part) * chans, o1 = min(o0 + chans, sh.part);
     const int s0 = blockIdx.y * NT, nt = min(NT, S - s0);
     const int ld = (sh.part + 7) / 8 * 8;
-    for (int i = threadIdx.x; i < NT * sh.part; i += kStepThreads) {
-        const int k = i / sh.part, ch = i - k * sh.part;
-        float v = 0.f;
-        if (k < nt) {
-            const int t = cu_seqlens[s0 + k], slot = state_slots[s0 + k];
-            if (slot >= 0 && slot < sh.num_slots)
-                v = rnd<T>(lru_conv_of(packed, bias_x, conv_w, conv_b, state + static_cast<int64_t>(slot) * sh.state_floats + sh.W, sh, t, 0,
-                                       positions[t], b * sh.part + ch));
-            else atomicExch(err, 2);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const T* rows_r = gates + static_cast<int64_t>(b) * 2 * sh.part * sh.part;
+    const T* rows_i = rows_r + static_cast<int64_t>(sh.part) * sh.part;
+    float fr[8], fi[8];                                 // a channel's first 256 gate weights are on their way before they are needed
+    auto ahead = [&](int o) {
+        if (vec && lane * 8 < sh.part && o < o1) {
+            fma8(rows_r + static_cast<int64_t>(o) * sh.part + lane * 8, fr);
+            fma8(rows_i + static_cast<int64_t>(o) * sh.part + lane * 8, fi);
         }
-        us[k * ld + ch] = v;
+    };
+    ahead(o0 + warp);
+    __shared__ int s_slot[NT], s_tok[NT], s_pos[NT];
+    if (threadIdx.x < NT) {
+        const int k = threadIdx.x;
+        const int t = k < nt ? cu_seqlens[s0 + k] : 0;
+        int slot = k < nt ? state_slots[s0 + k] : -1;
+        if (slot >= sh.num_slots || (slot < 0 && k < nt)) { atomicExch(err, 2); slot = -1; }
+        s_slot[k] = slot; s_tok[k] = t; s_pos[k] = positions[t];
     }
     __syncthreads();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int o = o0 + warp; o < min(o0 + kStepChannels, sh.part); o += kStepThreads / 32) {
-        const T* wr = gates + (static_cast<int64_t>(b) * 2 * sh.part + o) * sh.part;
-        const T* wi = wr + static_cast<int64_t>(sh.part) * sh.part;
+    for (int ch = threadIdx.x; ch < sh.part; ch += kStepThreads) {
+        const int c = b * sh.part + ch;
+        if constexpr (K > 0) {
+            float cw[K];
+#pragma unroll
+            for (int m = 0; m < K; ++m) cw[m] = conv_w[static_cast<int64_t>(m) * sh.W + c];
+            const float xb = bias_x[c], cb = conv_b[c];
+            float x[NT][K];
+#pragma unroll
+            for (int k = 0; k < NT; ++k) {
+                const bool live = s_slot[k] >= 0;
+                const float* ring = state + static_cast<int64_t>(live ? s_slot[k] : 0) * sh.state_floats + sh.W + c;
+#pragma unroll
+                for (int m = 0; m < K; ++m) {
+                    const int back = K - 1 - m, pos = s_pos[k];
+                    if (back == 0) x[k][m] = live ? to_float(packed[static_cast<int64_t>(s_tok[k]) * sh.stride + sh.x_off + c]) + xb : 0.f;
+                    else x[k][m] = (live && pos >= back) ? ring[static_cast<int64_t>((pos - back) % K) * sh.W] : 0.f;
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < NT; ++k) {
+                float acc = 0.f;
+#pragma unroll
+                for (int m = 0; m < K; ++m) acc = fmaf(cw[m], x[k][m], acc);
+                us[k * ld + ch] = rnd<T>(acc + cb);
+            }
+        } else {
+            for (int k = 0; k < NT; ++k)
+                us[k * ld + ch] = s_slot[k] < 0 ? 0.f
+                    : rnd<T>(lru_conv_of(packed, bias_x, conv_w, conv_b, state + static_cast<int64_t>(s_slot[k]) * sh.state_floats + sh.W, sh,
+                                         s_tok[k], 0, s_pos[k], c));
+        }
+    }
+    __syncthreads();
+    for (int o = o0 + warp; o < o1; o += kStepWarps) {
+        const T* wr = rows_r + static_cast<int64_t>(o) * sh.part;
+        const T* wi = rows_i + static_cast<int64_t>(o) * sh.part;
+        // what lane k needs of request k at the end, asked for before the products
+        const int c = b * sh.part + o;
+        const bool mine = lane < nt && s_slot[lane < NT ? lane : 0] >= 0;
+        const int t = mine ? s_tok[lane] : 0;
+        float* row = state + static_cast<int64_t>(mine ? s_slot[lane] : 0) * sh.state_floats;
+        float s_old = 0.f, rb = 0.f, ib = 0.f, ns = 0.f, yv = 0.f, xv = 0.f;
+        if (mine) {
+            s_old = row[c]; rb = br[c]; ib = bi[c]; ns = nsp[c];
+            yv = to_float(packed[static_cast<int64_t>(t) * sh.stride + sh.y_off + c]) + bias_y[c];
+            xv = to_float(packed[static_cast<int64_t>(t) * sh.stride + sh.x_off + c]) + bias_x[c];
+        }
         float zr[NT], zi[NT];
 #pragma unroll
         for (int k = 0; k < NT; ++k) zr[k] = zi[k] = 0.f;
         if (vec) {
             for (int e = lane * 8; e < sh.part; e += 256) {
-                float fr[8], fi[8];
-                fma8(wr + e, fr);
-                fma8(wi + e, fi);
+                if (e >= 256) { fma8(wr + e, fr); fma8(wi + e, fi); }
 #pragma unroll
                 for (int k = 0; k < NT; ++k) {
                     const float4 x0 = *reinterpret_cast<const float4*>(us + k * ld + e), x1 = *reinterpret_cast<const float4*>(us + k * ld + e + 4);
@@ -258,25 +415,20 @@ lru_step_kernel(T* __restrict__ out, const T* __restrict__ packed, const float* 
                 for (int k = 0; k < NT; ++k) { const float x = us[k * ld + e]; zr[k] = fmaf(x, fr, zr[k]); zi[k] = fmaf(x, fi, zi[k]); }
             }
         }
+        ahead(o + kStepWarps);
         float mr = 0.f, mi = 0.f;                       // lane k keeps request k's pair
 #pragma unroll
         for (int k = 0; k < NT; ++k) {
             const float a = warp_sum(zr[k]), d = warp_sum(zi[k]);
             if (lane == k) { mr = a; mi = d; }
         }
-        if (lane < nt) {
-            const int t = cu_seqlens[s0 + lane], slot = state_slots[s0 + lane], c = b * sh.part + o;
-            if (slot >= 0 && slot < sh.num_slots) {
-                float* row = state + static_cast<int64_t>(slot) * sh.state_floats;
-                float a, in;
-                lru_gate(mr, mi, br[c], bi[c], nsp[c], us[lane * ld + o], a, in);
-                const float st = fmaf(a, row[c], in);
-                row[c] = st;
-                out[static_cast<int64_t>(t) * sh.W + c] =
-                    from_float<T>(st * lru_gelu(to_float(packed[static_cast<int64_t>(t) * sh.stride + sh.y_off + c]) + bias_y[c]));
-                if (sh.taps > 1)
-                    row[sh.W + static_cast<int64_t>(positions[t] % sh.taps) * sh.W + c] = to_float(packed[static_cast<int64_t>(t) * sh.stride + sh.x_off + c]) + bias_x[c];
-            }
+        if (mine) {
+            float a, in;
+            lru_gate<T>(mr, mi, rb, ib, ns, us[lane * ld + o], a, in);
+            const float st = fmaf(a, s_old, in);
+            row[c] = st;
+            out[static_cast<int64_t>(t) * sh.W + c] = from_float<T>(st * lru_gelu_of<T>(yv));
+            if (sh.taps > 1) row[sh.W + static_cast<int64_t>(s_pos[lane] % sh.taps) * sh.W + c] = xv;
         }
     }
 }
@@ -301,6 +453,22 @@ extern "C" int cvb_lru_conv(void* u, const void* packed, const float* bias_x, co
     LruShape sh;
     const int rc = lru_shape(sh, W, parts, taps, stride, y_off, x_off, state_floats, num_slots);
     if (rc != CVB_OK || T < 0) return rc != CVB_OK ? rc : CVB_E_SIZE;
+    const int n = dtype == CVB_DTYPE_BF16 ? 8 : 4;
+    const bool vec = W % n == 0 && stride % n == 0 && x_off % n == 0 && ((reinterpret_cast<uintptr_t>(packed) | reinterpret_cast<uintptr_t>(u)) & 15) == 0;
+    const int vcols = (W / n + kLruThreads - 1) / kLruThreads;
+    int run = 8;                                        // shorter runs where long ones would leave SMs idle
+    while (run > 2 && static_cast<int64_t>((T + run - 1) / run) * vcols < 592) run /= 2;
+    const dim3 vgrid((T + run - 1) / run, vcols);
+    if (vec && taps >= 2 && taps <= 4 && vgrid.y <= 65535) {
+#define CALL_K(TY, K)                                                                                                         \
+    launch_kernel(lru_conv_vec_kernel<TY, K>, vgrid, dim3(kLruThreads), 0, stream, (TY*)u, (const TY*)packed, bias_x, conv_w, conv_b, state, \
+                  seq_of_token, cu_seqlens, state_slots, positions, T, run, sh, err_flag)
+#define CALL(TY) if (taps == 4) { CALL_K(TY, 4); } else if (taps == 3) { CALL_K(TY, 3); } else { CALL_K(TY, 2); }
+        CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+#undef CALL_K
+        return launch_status();
+    }
     const dim3 grid(T, min((W + kLruThreads - 1) / kLruThreads, 8));
 #define CALL(TY)                                                                                                              \
     launch_kernel(lru_conv_kernel<TY>, grid, dim3(kLruThreads), 0, stream, (TY*)u, (const TY*)packed, bias_x, conv_w, conv_b, state, \
@@ -349,22 +517,27 @@ extern "C" int cvb_lru_step(void* out, const void* packed, const float* bias_y, 
     const int rc = lru_shape(sh, W, parts, taps, stride, y_off, x_off, state_floats, num_slots);
     if (rc != CVB_OK) return rc;
     if (S < 0) return CVB_E_SIZE;
-    const int per_part = (sh.part + kStepChannels - 1) / kStepChannels;
+    // one channel a warp where that fills no more than two blocks per SM, else two or four
+    int per_warp = 1;
+    while (per_warp < 4 && static_cast<int64_t>(parts) * ((sh.part + kStepWarps * per_warp - 1) / (kStepWarps * per_warp)) > 296) per_warp *= 2;
+    const int per_part = (sh.part + kStepWarps * per_warp - 1) / (kStepWarps * per_warp);
     const int nt = S <= 1 ? 1 : (S <= 2 ? 2 : (S <= 4 ? 4 : kStepTokens));
     const dim3 grid(parts * per_part, (S + nt - 1) / nt);
     const size_t smem = static_cast<size_t>(nt) * ((sh.part + 7) / 8 * 8) * sizeof(float);
     if (smem > 200 * 1024 || grid.y > 65535) return CVB_E_SIZE;
     const int vec = sh.part % 8 == 0 && (reinterpret_cast<uintptr_t>(gates) & 15) == 0;
-#define CALL_N(TY, NT)                                                                                                        \
+#define CALL_NK(TY, NT, K)                                                                                                      \
     do {                                                                                                                      \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(lru_step_kernel<TY, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
-        launch_kernel(lru_step_kernel<TY, NT>, grid, dim3(kStepThreads), smem, stream, (TY*)out, (const TY*)packed, bias_y, bias_x,     \
-                      conv_w, conv_b, (const TY*)gates, br, bi, nsp, state, cu_seqlens, state_slots, positions, S, sh, vec, err_flag);  \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(lru_step_kernel<TY, NT, K>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
+        launch_kernel(lru_step_kernel<TY, NT, K>, grid, dim3(kStepThreads), smem, stream, (TY*)out, (const TY*)packed, bias_y, bias_x,     \
+                      conv_w, conv_b, (const TY*)gates, br, bi, nsp, state, cu_seqlens, state_slots, positions, S, sh, vec, per_warp, err_flag);  \
     } while (0)
+#define CALL_N(TY, NT) if (taps == 4) CALL_NK(TY, NT, 4); else CALL_NK(TY, NT, 0)
 #define CALL(TY)                                                                                                              \
     if (nt == 1) { CALL_N(TY, 1); } else if (nt == 2) { CALL_N(TY, 2); } else if (nt == 4) { CALL_N(TY, 4); } else { CALL_N(TY, 8); }
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
 #undef CALL_N
+#undef CALL_NK
     return launch_status();
 }

@@ -825,10 +825,16 @@ def _lru_check(packed, width, parts, y_off, x_off, vectors, ints):
             raise KernelError("lru: index tensors are int32")
 
 
-def lru_chunk_tokens(num_tokens: int) -> int:
+def lru_chunk_tokens(num_tokens: int, width: int) -> int:
     """Tokens per chunk of a request's portion: short enough that a long prompt's chunks fill the SMs, long enough that the chunks
     before a chunk are few."""
-    return 32 if num_tokens <= 1024 else (64 if num_tokens <= 4096 else 128)
+    n = -(-num_tokens * (-(-width // 128)) // LINEAR_BLOCKS)
+    return max(32, min(256, -(-n // 32) * 32))
+
+
+def lru_most_chunks(max_tokens: int, max_seqs: int, width: int) -> int:
+    """The most chunks a step of up to `max_tokens` tokens of `max_seqs` requests can have."""
+    return max(LINEAR_BLOCKS // (-(-width // 128)), max_tokens // 256) + 2 + max_seqs
 
 
 def lru_conv(u: torch.Tensor, packed: torch.Tensor, y_off: int, x_off: int, parts: int, bias_x, conv_w, conv_b, state, seq_of_token, cu_seqlens,

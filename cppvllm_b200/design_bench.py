@@ -972,7 +972,7 @@ def sumevik_kernel_pairs(s, pk):
     cw, nsp = rnd(4, W, dtype=f32), -torch.rand(W, generator=g, device=d) * 0.1
     st_l = torch.zeros(2, 5 * W, dtype=f32, device=d)
     summary = torch.empty(2 * W * (T // 16 + 2), dtype=f32, device=d)
-    L = ops.lru_chunk_tokens(T)
+    L = ops.lru_chunk_tokens(T, W)
     new = _us(lambda i: ops.lru_conv(u, lru_in, 0, W, P, bx, cw, cb, st_l, seq_of, cu, slot0, pos))
     a_in, hist = rnd(T, W), torch.zeros(2, 3 * W, dtype=f32, device=d)
     like = _us(lambda i: ops.input_conv(o_lru, a_in, cw, hist, 0, seq_of, cu, slot0))

@@ -71,8 +71,7 @@ class GatedLRUMixer(Mixer):
             u = ops.lru_conv(ws.rows("lru_u", T, W, x.dtype), packed, 0, W, self.blocks, self.b_x, self.conv_w, self.conv_b, state,
                              ctx.seq_of_token, ctx.cu_seqlens, ctx.state_slots, ctx.positions)
             z = ops.lru_gates(ws.rows("lru_z", T, 2 * W, torch.float32), u, self.gates)
-            most = max(64, ws.max_tokens // 128 + 1) + ws.max_seqs + 1            # chunks of the largest step
-            summary = ws.flat(f"lru_summary_{W}", most * 2 * W, torch.float32)
+            summary = ws.flat(f"lru_summary_{W}", ops.lru_most_chunks(ws.max_tokens, ws.max_seqs, W) * 2 * W, torch.float32)
             ops.lru_scan(out, z, u, packed, 0, W, self.blocks, self.taps, self.b_y, self.b_x, self.b_r, self.b_i, self.neg_softplus, state,
-                         ctx.cu_seqlens, ctx.state_slots, ctx.positions, q_lens, ops.lru_chunk_tokens(T), summary)
+                         ctx.cu_seqlens, ctx.state_slots, ctx.positions, q_lens, ops.lru_chunk_tokens(T, W), summary)
         return _project(self.rt, out, self.w_o, ws.rows("attn_proj", T, self.hidden_size, x.dtype), T)

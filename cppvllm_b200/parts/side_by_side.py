@@ -7,7 +7,9 @@ state)``: from the columns of its input projection (``w_in``) to ``core_width`` 
 (``w_o``), times `scale`.  The members' input projections are one product (their rows one below the other), the scaled cores lie
 side by side in one buffer, and their output projections are one product too (their columns side by side), whose sum over
 the inner dimension is the sum over the members: two products for the layer, and no kernel adds anything up.
-At most one member may keep cache entries and at most one per-request state.
+The cores share nothing, so every one but the first runs on a stream of its own beside it (inside a captured graph: a fork and
+a join), and attention and a recurrence fill the SMs together.  At most one member may keep cache entries and at most one
+per-request state.
 """
 from __future__ import annotations
 
@@ -15,6 +17,7 @@ from typing import Dict, Sequence
 
 import torch
 
+from ..csrc import ops
 from .base import Mixer, WeightSpec, register_part
 from .recurrent import _cat_rows, _project
 
@@ -35,6 +38,7 @@ class SideBySideMixer(Mixer):
             raise ValueError("at most one of the mixers keeps cache entries, and at most one per-request state")
         self.core_width = sum(m.core_width for m in self.members)
         self.w_in = self.w_o = None
+        self._streams = None
 
     @property
     def capturable(self) -> bool:
@@ -82,8 +86,28 @@ class SideBySideMixer(Mixer):
         ws = self.rt.workspace
         packed = _project(self.rt, x, self.w_in, ws.rows("pair_in", T, self.w_in.shape[0], x.dtype), T)
         joined = ws.rows("pair_out", T, self.core_width, x.dtype)
+        main = torch.cuda.current_stream(x.device)
+        if self._streams is None:
+            self._streams = [torch.cuda.Stream(x.device) for _ in self.members[1:]]
+        beside = not self.rt.plain_kernels
         o0 = 0
-        for m, scale, (c0, c1) in zip(self.members, self.scales, self.in_cols):
-            m.core(packed[:, c0:c1], joined[:, o0:o0 + m.core_width], scale, ctx, cache, state)
+        for i, (m, scale, (c0, c1)) in enumerate(zip(self.members, self.scales, self.in_cols)):
+            args = (packed[:, c0:c1], joined[:, o0:o0 + m.core_width], scale, ctx, cache, state)
             o0 += m.core_width
-        return _project(self.rt, joined, self.w_o, ws.rows("attn_proj", T, self.hidden_size, x.dtype), T)
+            if i == 0 or not beside:
+                first = (m, args) if beside else None
+                if not beside:
+                    m.core(*args)
+                continue
+            side = self._streams[i - 1]
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                m.core(*args)
+        if beside:
+            first[0].core(*first[1])                      # launched last, on the caller's stream
+            for side in self._streams:
+                main.wait_stream(side)
+        y = ws.rows("attn_proj", T, self.hidden_size, x.dtype)
+        if self.rt.plain_kernels:
+            return ops.linear(joined, self.w_o, out=y)
+        return ops.project_rows(joined, self.w_o, y, T, dependent=False)      # behind the join, not beside it
