@@ -5,11 +5,12 @@
 // float throughout; q, k, v (and the low-rank a, the output gate) are column ranges of a packed projection in the activations' type T.
 //
 //   linear_decay : g in place of the float product z = Wa2 a
-//   linear_scan  : portions of prompts.  A block owns 32 columns of S of one (chunk of a request's tokens, head); eight lanes share
-//                  two columns, a lane four neighbouring rows of every 32.  Eight tokens a stage travel through registers into
-//                  shared memory (converted on the way), so a token costs a lane three 16-byte reads of shared memory per four rows
-//                  and two columns; the eight partial outputs of a stage are added up and handed out over the eight lanes by one
-//                  transposing butterfly (seven shuffles a column).  Long portions are cut into chunks that run side by side:
+//   linear_scan  : portions of prompts.  A block owns 64 (32 for more than 128 rows) columns of S of one (chunk of a request's tokens,
+//                  head); eight lanes share four (two) columns, a lane four neighbouring rows of every 32.  Eight tokens a stage
+//                  travel through registers into shared memory (converted on the way), so a token costs a lane three 16-byte reads
+//                  of shared memory per four rows and four columns (the reads of shared memory are what bounds the kernel); the
+//                  eight partial outputs of a stage are added up and handed out over the eight lanes by one transposing butterfly
+//                  (seven shuffles a column).  Long portions are cut into chunks that run side by side:
 //                    pass 1: every chunk but a request's last: the state it leaves and the product of its decays, from zero (a
 //                            request's first chunk from the request's state); the last chunk's place receives the state in front
 //                    pass 2: the states behind the chunks in turn, element by element: E_k <- diag(P_k) E_(k-1) + E_k
@@ -50,7 +51,7 @@ linear_decay_vec_kernel(float* __restrict__ z, const float* __restrict__ bias, f
 
 constexpr int kLinThreads = 128;
 constexpr int kLinTokens = 8;                            // tokens per stage: as many as lanes share a column
-constexpr int kLinCols = 32;                             // columns of S per block, two per eight lanes
+constexpr int lin_cols(int kpt) { return kpt <= 16 ? 4 : 2; }         // columns of S per eight lanes; 16 times that per block
 
 struct LinearShape {
     int H, dk, dv, stride, q_off, k_off, v_off;
@@ -99,11 +100,12 @@ linear_scan_kernel(float* __restrict__ out, const T* __restrict__ packed, const 
     pdl_trigger();
     pdl_wait();
     constexpr int dkp = KPT * 8;                          // rows, padded
+    constexpr int NC = lin_cols(KPT), kLinCols = 16 * NC;
     constexpr int kArr = OUT ? 3 : 2;                     // k, g and, with outputs, q
     constexpr int kStage = kLinTokens * (kArr * dkp + kLinCols);
     extern __shared__ __align__(16) float sm[];           // two stages
     const int h = blockIdx.y, j0 = blockIdx.z * kLinCols, tid = threadIdx.x;
-    const int part = tid & 7, col = (tid >> 3) * 2, j = j0 + col;
+    const int part = tid & 7, col = (tid >> 3) * NC, j = j0 + col;
     const int dk = sh.dk, dv = sh.dv;
     int s, kc, nc, buf;
     if (!linear_locate(cu_seqlens, n_seqs, len, blockIdx.x, s, kc, nc, buf)) return;
@@ -116,34 +118,31 @@ linear_scan_kernel(float* __restrict__ out, const T* __restrict__ packed, const 
     float* st = state + static_cast<int64_t>(slot) * sh.state_floats + static_cast<int64_t>(h) * dk * dv;
     const int64_t mat = static_cast<int64_t>(sh.H) * dk * dv;
     auto end_of = [&](int k) { return ends + (static_cast<int64_t>(buf) + k) * mat + static_cast<int64_t>(h) * dk * dv; };
-    const bool c0 = j < dv, c1 = j + 1 < dv;
     // row r of this lane's KPT rows
     auto row = [&](int r) { return (r >> 2) * 32 + part * 4 + (r & 3); };
     const float* from = OUT ? (nc == 1 ? st : (kc == 0 ? end_of(nc - 1) : end_of(kc - 1))) : st;
     const bool zero = !OUT && kc > 0;
-    float S[KPT][2];
+    float S[KPT][NC];
 #pragma unroll
-    for (int r = 0; r < KPT; ++r) {
-        const int i = row(r);
-        S[r][0] = (i < dk && c0 && !(zero && kc < nc - 1)) ? from[static_cast<int64_t>(i) * dv + j] : 0.f;
-        S[r][1] = (i < dk && c1 && !(zero && kc < nc - 1)) ? from[static_cast<int64_t>(i) * dv + j + 1] : 0.f;
-    }
+    for (int r = 0; r < KPT; ++r)
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+            S[r][c] = (row(r) < dk && j + c < dv && !(zero && kc < nc - 1)) ? from[static_cast<int64_t>(row(r)) * dv + j + c] : 0.f;
+    auto put = [&](float* dst) {
+#pragma unroll
+        for (int r = 0; r < KPT; ++r)
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+                if (row(r) < dk && j + c < dv) dst[static_cast<int64_t>(row(r)) * dv + j + c] = S[r][c];
+    };
     if (!OUT && kc == nc - 1) {                           // the state in front of the portion, where the first chunk of pass 3 finds it
-        if (nc > 1) {
-            float* dst = end_of(kc);
-#pragma unroll
-            for (int r = 0; r < KPT; ++r) {
-                const int i = row(r);
-                if (i < dk && c0) dst[static_cast<int64_t>(i) * dv + j] = S[r][0];
-                if (i < dk && c1) dst[static_cast<int64_t>(i) * dv + j + 1] = S[r][1];
-            }
-        }
+        if (nc > 1) put(end_of(kc));
         return;
     }
     for (int i = tid; i < 2 * kStage; i += kLinThreads) sm[i] = 0.f;         // rows past dk and columns past dv stay zero
     __syncthreads();
 
-    // a stage: [tokens][dkp] of k, of g, (of q), [tokens][32] of v
+    // a stage: [tokens][dkp] of k, of g, (of q), [tokens][columns] of v
     constexpr int N = Raw16<T>::N;
     constexpr int kQK = (OUT ? 2 : 1) * kLinTokens * dkp / N;                // 16-byte pieces of k (and q) in a stage
     constexpr int kQKPer = (kQK + kLinThreads - 1) / kLinThreads;
@@ -226,11 +225,15 @@ linear_scan_kernel(float* __restrict__ out, const T* __restrict__ packed, const 
         __syncthreads();                                  // one barrier a stage: the other stage's readers passed the barrier before
         if (vec && t0 + kLinTokens < end) fetch(t0 + kLinTokens);
         const float* base = sm + stage * kStage;
-        float o0[kLinTokens], o1[kLinTokens];
+        float o[kLinTokens][NC];
 #pragma unroll
         for (int tt = 0; tt < kLinTokens; ++tt) {         // tokens past the end: k = 0 and g = 1 change nothing
-            const float2 v = *reinterpret_cast<const float2*>(base + kArr * kLinTokens * dkp + tt * kLinCols + col);
-            float a0 = 0.f, a1 = 0.f;
+            float v[NC];
+            const float* vp = base + kArr * kLinTokens * dkp + tt * kLinCols + col;
+            if constexpr (NC == 4) { const float4 x = *reinterpret_cast<const float4*>(vp); v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; }
+            else { const float2 x = *reinterpret_cast<const float2*>(vp); v[0] = x.x; v[1] = x.y; }
+#pragma unroll
+            for (int c = 0; c < NC; ++c) o[tt][c] = 0.f;
 #pragma unroll
             for (int m = 0; m < KPT / 4; ++m) {
                 const int at = tt * dkp + m * 32 + part * 4;
@@ -244,16 +247,15 @@ linear_scan_kernel(float* __restrict__ out, const T* __restrict__ packed, const 
                 }
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    float& x0 = S[m * 4 + e][0];
-                    float& x1 = S[m * 4 + e][1];
-                    x0 = fmaf(g[e], x0, kk[e] * v.x);
-                    x1 = fmaf(g[e], x1, kk[e] * v.y);
-                    if (OUT) { a0 = fmaf(x0, qq[e], a0); a1 = fmaf(x1, qq[e], a1); }
-                    else P[m * 4 + e] *= g[e];
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) {
+                        float& x = S[m * 4 + e][c];
+                        x = fmaf(g[e], x, kk[e] * v[c]);
+                        if (OUT) o[tt][c] = fmaf(x, qq[e], o[tt][c]);
+                    }
+                    if (!OUT) P[m * 4 + e] *= g[e];
                 }
             }
-            o0[tt] = a0;
-            o1[tt] = a1;
         }
         if (OUT) {
             // lane `part` of the eight receives the sums of token `part`
@@ -261,30 +263,27 @@ linear_scan_kernel(float* __restrict__ out, const T* __restrict__ packed, const 
             for (int half = kLinTokens / 2; half > 0; half >>= 1) {
                 const bool up = (part & half) != 0;
 #pragma unroll
-                for (int i = 0; i < half; ++i) {
-                    const float s0 = up ? o0[i] : o0[i + half], k0 = up ? o0[i + half] : o0[i];
-                    const float s1 = up ? o1[i] : o1[i + half], k1 = up ? o1[i + half] : o1[i];
-                    o0[i] = k0 + __shfl_xor_sync(0xffffffffu, s0, half);
-                    o1[i] = k1 + __shfl_xor_sync(0xffffffffu, s1, half);
-                }
+                for (int i = 0; i < half; ++i)
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) {
+                        const float away = up ? o[i][c] : o[i + half][c], own = up ? o[i + half][c] : o[i][c];
+                        o[i][c] = own + __shfl_xor_sync(0xffffffffu, away, half);
+                    }
             }
             const int t = t0 + part;
             if (t < end) {
                 float* dst = out + (static_cast<int64_t>(t) * sh.H + h) * dv + j;
-                if (c0) dst[0] = o0[0];
-                if (c1) dst[1] = o1[0];
+                if (NC == 4 && j + 3 < dv && (dv & 3) == 0) {
+                    *reinterpret_cast<float4*>(dst) = make_float4(o[0][0], o[0][1], o[0][NC - 2], o[0][NC - 1]);
+                } else {
+#pragma unroll
+                    for (int c = 0; c < NC; ++c)
+                        if (j + c < dv) dst[c] = o[0][c];
+                }
             }
         }
     }
-    float* dst = OUT ? st : end_of(kc);
-    if (!OUT || kc == nc - 1) {
-#pragma unroll
-        for (int r = 0; r < KPT; ++r) {
-            const int i = row(r);
-            if (i < dk && c0) dst[static_cast<int64_t>(i) * dv + j] = S[r][0];
-            if (i < dk && c1) dst[static_cast<int64_t>(i) * dv + j + 1] = S[r][1];
-        }
-    }
+    if (!OUT || kc == nc - 1) put(OUT ? st : end_of(kc));
     if (!OUT && j0 == 0 && col == 0) {
         float* pd = decays + ((static_cast<int64_t>(buf) + kc) * sh.H + h) * dk;
 #pragma unroll
@@ -421,13 +420,14 @@ static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) =
 template <typename T, int KPT, bool OUT>
 static void launch_linear(float* out, const T* packed, const float* gg, float* state, float* ends, float* decays, const int* cu_seqlens,
                           const int* state_slots, int S, int len, int chunks, const LinearShape& sh, int vec, int* err, cudaStream_t stream) {
-    const size_t smem = static_cast<size_t>(2) * kLinTokens * ((OUT ? 3 : 2) * KPT * 8 + kLinCols) * sizeof(float);
+    constexpr int cols = 16 * lin_cols(KPT);
+    const size_t smem = static_cast<size_t>(2) * kLinTokens * ((OUT ? 3 : 2) * KPT * 8 + cols) * sizeof(float);
     static bool raised = false;
     if (smem > 48 * 1024 && !raised) {
         if (cudaFuncSetAttribute(linear_scan_kernel<T, KPT, OUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess) return;
         raised = true;
     }
-    launch_kernel(linear_scan_kernel<T, KPT, OUT>, dim3(chunks, sh.H, (sh.dv + kLinCols - 1) / kLinCols), dim3(kLinThreads), smem, stream, out, packed,
+    launch_kernel(linear_scan_kernel<T, KPT, OUT>, dim3(chunks, sh.H, (sh.dv + cols - 1) / cols), dim3(kLinThreads), smem, stream, out, packed,
                   gg, state, ends, decays, cu_seqlens, state_slots, S, len, sh, vec, err);
 }
 
@@ -436,7 +436,7 @@ static int run_linear(float* out, const T* packed, const float* gg, float* state
                       const int* state_slots, int S, int len, int chunks, int single, const LinearShape& sh, int vec, int* err, cudaStream_t stream) {
     if (!single) {
         launch_linear<T, KPT, false>(out, packed, gg, state, ends, decays, cu_seqlens, state_slots, S, len, chunks, sh, vec, err, stream);
-        const int zs = (sh.dk * sh.dv + 1023) / 1024;
+        const int zs = (sh.dk * sh.dv + 255) / 256;
         launch_kernel(linear_carry_kernel, dim3(S, sh.H, zs < 64 ? zs : 64), dim3(256), 0, stream, ends, decays, cu_seqlens, S, len, sh.H, sh.dk, sh.dv);
     }
     launch_linear<T, KPT, true>(out, packed, gg, state, ends, decays, cu_seqlens, state_slots, S, len, chunks, sh, vec, err, stream);
@@ -469,10 +469,11 @@ extern "C" int cvb_linear_scan(float* out, const void* packed, int stride, int q
     LinearShape sh;
     const int rc = linear_shape(sh, H, dk, dv, stride, q_off, k_off, v_off, qk_scale, state_floats, num_slots);
     if (rc != CVB_OK) return rc;
-    if (S < 0 || dk > 512 || len <= 0 || len % kLinTokens || chunks <= 0 || (dv + kLinCols - 1) / kLinCols > 65535) return CVB_E_SIZE;
+    if (S < 0 || dk > 512 || len <= 0 || len % kLinTokens || chunks <= 0 || (dv + 31) / 32 > 65535) return CVB_E_SIZE;
     if (held > 0 && (ends == nullptr || decays == nullptr || ends_floats < static_cast<int64_t>(held) * H * dk * dv
                      || decays_floats < static_cast<int64_t>(held) * H * dk)) return CVB_E_SCRATCH;
     const int n = dtype == CVB_DTYPE_BF16 ? 8 : 4;
+    if (!al16(out)) return CVB_E_ALIGN;
     const int vec = dk % n == 0 && dv % n == 0 && stride % n == 0 && q_off % n == 0 && k_off % n == 0 && v_off % n == 0 && al16(packed) && al16(gg);
 #define CALL_K(TY, KPT) return run_linear<TY, KPT>(out, (const TY*)packed, gg, state, ends, decays, cu_seqlens, state_slots, S, len, chunks,    \
                                                    held == 0, sh, vec, err_flag, stream)

@@ -278,12 +278,24 @@ lru_finish_kernel(T* __restrict__ out, const float* __restrict__ z, const T* __r
         }
     }
     const float rb = GATED ? br[c] : 0.f, ib = GATED ? bi[c] : 0.f, ns = GATED ? nsp[c] : 0.f, yb = bias_y[c];
-#pragma unroll 8
-    for (int i = 0; i < n; ++i) {
-        float a = zp[static_cast<int64_t>(i) * 2 * sh.part], in = zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part];
-        if (GATED) lru_gate<T>(a, in, rb, ib, ns, to_float(up[static_cast<int64_t>(i) * sh.W]), a, in);
-        st = fmaf(a, st, in);
-        op[static_cast<int64_t>(i) * sh.W] = from_float<T>(st * lru_gelu_of<T>(to_float(yp[static_cast<int64_t>(i) * sh.stride]) + yb));
+    constexpr int kAhead = 8;                           // tokens whose rows are asked for together
+    for (int i0 = 0; i0 < n; i0 += kAhead) {
+        float a[kAhead], in[kAhead], y[kAhead], uu[kAhead];
+#pragma unroll
+        for (int e = 0; e < kAhead; ++e) {
+            const int i = min(i0 + e, n - 1);
+            a[e] = zp[static_cast<int64_t>(i) * 2 * sh.part];
+            in[e] = zp[static_cast<int64_t>(i) * 2 * sh.part + sh.part];
+            y[e] = to_float(yp[static_cast<int64_t>(i) * sh.stride]);
+            if (GATED) uu[e] = to_float(up[static_cast<int64_t>(i) * sh.W]);
+        }
+#pragma unroll
+        for (int e = 0; e < kAhead; ++e) {
+            if (i0 + e >= n) break;
+            if (GATED) lru_gate<T>(a[e], in[e], rb, ib, ns, uu[e], a[e], in[e]);
+            st = fmaf(a[e], st, in[e]);
+            op[static_cast<int64_t>(i0 + e) * sh.W] = from_float<T>(st * lru_gelu_of<T>(y[e] + yb));
+        }
     }
     if (t0 + n == end) {
         row[c] = st;
@@ -416,12 +428,25 @@ lru_step_kernel(T* __restrict__ out, const T* __restrict__ packed, const float* 
             }
         }
         ahead(o + kStepWarps);
-        float mr = 0.f, mi = 0.f;                       // lane k keeps request k's pair
+        // the 2 NT sums over the warp by a transposing butterfly: lane l ends with the sum of value l / (32 / (2 NT)), of which lane k
+        // fetches request k's two
+        float r[2 * NT];
 #pragma unroll
-        for (int k = 0; k < NT; ++k) {
-            const float a = warp_sum(zr[k]), d = warp_sum(zi[k]);
-            if (lane == k) { mr = a; mi = d; }
+        for (int k = 0; k < NT; ++k) { r[k] = zr[k]; r[NT + k] = zi[k]; }
+        int mask = 16;
+#pragma unroll
+        for (int half = NT; half > 0; half >>= 1, mask >>= 1) {
+            const bool up = (lane & mask) != 0;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+                const float away = up ? r[i] : r[i + half], own = up ? r[i + half] : r[i];
+                r[i] = own + __shfl_xor_sync(0xffffffffu, away, mask);
+            }
         }
+#pragma unroll
+        for (; mask > 0; mask >>= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], mask);
+        constexpr int kSpan = 32 / (2 * NT);
+        const float mr = __shfl_sync(0xffffffffu, r[0], (lane % NT) * kSpan), mi = __shfl_sync(0xffffffffu, r[0], (NT + lane % NT) * kSpan);
         if (mine) {
             float a, in;
             lru_gate<T>(mr, mi, rb, ib, ns, us[lane * ld + o], a, in);

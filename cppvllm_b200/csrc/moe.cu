@@ -33,8 +33,8 @@
 
 namespace cvb {
 
-constexpr int kRouteWarps = 4;          // many tokens: warps per block, kRouteTokens tokens each
-constexpr int kRouteTokens = 4;
+constexpr int kRouteWarps = 8;          // many tokens: warps per block, which share kRouteTokens tokens
+constexpr int kRouteTokens = 8;
 constexpr int kRouteFewWarps = 8;       // few tokens: the warps of a block share one token's router outputs out
 
 // The choice from the logits z [E] (shared memory of the calling warp; in mode 3 with 2 E + groups floats): see the top of this file.
@@ -120,8 +120,9 @@ template <int V> __device__ __forceinline__ void route_load(const __nv_bfloat16*
     } else f[0] = __bfloat162float(p[0]);
 }
 
-// Many tokens: a warp holds kRouteTokens tokens by four router outputs in registers, so a weight it loads serves four tokens and
-// an activation four outputs.
+// Many tokens: a block takes kRouteTokens tokens, its warps a slice of D each.  A warp holds all the block's tokens by four router
+// outputs in registers, so a weight it loads serves eight tokens and an activation four outputs; the warps' parts meet in shared
+// memory in a fixed order.
 template <typename T, int V>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x, const float* __restrict__ wr,
@@ -129,13 +130,12 @@ route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* _
                   float* __restrict__ extra_out, int groups, int keep) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ float smem[];                     // [kRouteWarps][kRouteTokens][E], mode 3: [..][2 E + groups]
+    extern __shared__ float smem[];                     // [kRouteTokens][E] (mode 3: [..][2 E + groups]), then a round's parts
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int64_t t0 = (static_cast<int64_t>(blockIdx.x) * kRouteWarps + warp) * kRouteTokens;
-    if (t0 >= n_tokens) return;
+    const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kRouteTokens;
     const int nt = static_cast<int>(n_tokens - t0 < kRouteTokens ? n_tokens - t0 : kRouteTokens);
     const int per = mode == 3 ? 2 * E + groups : E;
-    float* z = smem + static_cast<int64_t>(warp) * kRouteTokens * per;
+    float* part = smem + kRouteTokens * per;            // [kRouteWarps][kRouteTokens * 4]
     const T* xr[kRouteTokens];
 #pragma unroll
     for (int k = 0; k < kRouteTokens; ++k) xr[k] = x + (t0 + min(k, nt - 1)) * D;       // rows past the end repeat the last one
@@ -146,33 +146,51 @@ route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* _
         float d[kRouteTokens][4];
 #pragma unroll
         for (int k = 0; k < kRouteTokens; ++k) { d[k][0] = d[k][1] = d[k][2] = d[k][3] = 0.f; }
-        for (int i = lane * V; i < D; i += 32 * V) {
-            float wv[4][V], xv[kRouteTokens][V];
+        for (int i = (warp * 32 + lane) * V; i < D; i += kRouteWarps * 32 * V) {
+            float wv[4][V];
 #pragma unroll
             for (int q = 0; q < 4; ++q) route_load<V>(w[q] + i, wv[q]);
 #pragma unroll
-            for (int k = 0; k < kRouteTokens; ++k) route_load<V>(xr[k] + i, xv[k]);
-#pragma unroll
-            for (int k = 0; k < kRouteTokens; ++k)
+            for (int k = 0; k < kRouteTokens; ++k) {
+                float xv[V];
+                route_load<V>(xr[k] + i, xv);
 #pragma unroll
                 for (int q = 0; q < 4; ++q)
 #pragma unroll
-                    for (int v = 0; v < V; ++v) d[k][q] = fmaf(xv[k][v], wv[q][v], d[k][q]);
+                    for (int v = 0; v < V; ++v) d[k][q] = fmaf(xv[v], wv[q][v], d[k][q]);
+            }
         }
+        // 32 sums over 32 lanes: lane 4 k + q ends with the sum of (k, q), by a transposing butterfly
+        float r[kRouteTokens * 4];
 #pragma unroll
         for (int k = 0; k < kRouteTokens; ++k)
 #pragma unroll
-            for (int q = 0; q < 4; ++q) {
-                const float v = warp_sum(d[k][q]);
-                const int e = e0 + q;
-                if (lane == 0 && k < nt && e < E + extra) {
-                    if (e < E) z[k * per + e] = v + (bias && mode != 3 ? bias[e] : 0.f);
-                    else extra_out[(t0 + k) * extra + (e - E)] = v;
-                }
+            for (int q = 0; q < 4; ++q) r[k * 4 + q] = d[k][q];
+#pragma unroll
+        for (int half = 16; half > 0; half >>= 1) {
+            const bool up = (lane & half) != 0;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+                const float away = up ? r[i] : r[i + half], own = up ? r[i + half] : r[i];
+                r[i] = own + __shfl_xor_sync(0xffffffffu, away, half);
             }
+        }
+        __syncthreads();                                // the round before has been read
+        part[warp * 32 + lane] = r[0];
+        __syncthreads();
+        if (warp == 0) {
+            float v = 0.f;
+#pragma unroll
+            for (int g = 0; g < kRouteWarps; ++g) v += part[g * 32 + lane];
+            const int k = lane >> 2, e = e0 + (lane & 3);
+            if (k < nt && e < E + extra) {
+                if (e < E) smem[k * per + e] = v + (bias && mode != 3 ? bias[e] : 0.f);
+                else extra_out[(t0 + k) * extra + (e - E)] = v;
+            }
+        }
     }
-    __syncwarp();
-    for (int k = 0; k < nt; ++k) route_select(z + k * per, ids, weights, bias, t0 + k, E, top, mode, scale, groups, keep, lane);
+    __syncthreads();
+    for (int k = warp; k < nt; k += kRouteWarps) route_select(smem + k * per, ids, weights, bias, t0 + k, E, top, mode, scale, groups, keep, lane);
 }
 
 // Few tokens: a block per token; its warps take the router outputs in turn.
@@ -454,10 +472,11 @@ extern "C" int cvb_route_topk(int* ids, float* weights, const void* x, const flo
     if (top > E || E > 2048) return CVB_E_SHAPE;
     if (mode == 3 && (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups))) return CVB_E_SHAPE;
     const size_t row = static_cast<size_t>(mode == 3 ? 2 * E + groups : E) * sizeof(float);
-    if (row * kRouteWarps * kRouteTokens > 200 * 1024) return CVB_E_SIZE;
+    const size_t parts = static_cast<size_t>(kRouteWarps) * kRouteTokens * 4 * sizeof(float);
+    if (row * kRouteTokens + parts > 200 * 1024) return CVB_E_SIZE;
     const bool few = T <= 512;
     const bool four = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(wr)) & 15) == 0;
-    const size_t smem = few ? row : row * kRouteWarps * kRouteTokens;
+    const size_t smem = few ? row : row * kRouteTokens + parts;
 #define CALL_V(TY, V)                                                                                                         \
     do {                                                                                                                      \
         if (few) {                                                                                                            \
@@ -465,7 +484,7 @@ extern "C" int cvb_route_topk(int* ids, float* weights, const void* x, const flo
                           D, E, top, mode, scale, extra, extra_out, groups, keep);                                            \
         } else {                                                                                                              \
             if (smem > 48 * 1024) cudaFuncSetAttribute(route_topk_kernel<TY, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
-            launch_kernel(route_topk_kernel<TY, V>, dim3((T + kRouteWarps * kRouteTokens - 1) / (kRouteWarps * kRouteTokens)),                  \
+            launch_kernel(route_topk_kernel<TY, V>, dim3((T + kRouteTokens - 1) / kRouteTokens),                  \
                           dim3(kRouteWarps * 32), smem, stream, ids, weights, (const TY*)x, wr, bias, T, D, E, top, mode, scale, extra,         \
                           extra_out, groups, keep);                                                                           \
         }                                                                                                                     \

@@ -710,7 +710,8 @@ def delta_scan(out, qn, kn, vv, gg, bb, state: torch.Tensor, cu_seqlens, state_s
 # ---- gated linear attention (csrc/linear.cu) ------------------------------------------------------------------------------------
 
 _linear = None
-LINEAR_BLOCKS = 1184        # blocks of a scan that keep every SM busy
+LINEAR_BLOCKS = 592         # blocks of a scan that are resident together: four per SM
+LRU_BLOCKS = 1184           # the same for the gated recurrence
 LINEAR_MIN_CHUNK = 64
 
 
@@ -733,18 +734,21 @@ def linear_decay(z: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tenso
     return z
 
 
-def linear_chunk_tokens(num_tokens: int, num_heads: int, vdim: int) -> int:
+def _linear_blocks(num_heads: int, dim: int, vdim: int) -> int:
+    """Blocks per chunk: 64 columns of the state a block, 32 for more than 128 rows."""
+    return num_heads * -(-vdim // (64 if dim <= 128 else 32))
+
+
+def linear_chunk_tokens(num_tokens: int, num_heads: int, dim: int, vdim: int) -> int:
     """Tokens per chunk of a portion: as many chunks as it takes to keep every SM busy, none shorter than 64 tokens."""
-    per_chunk = num_heads * ((vdim + 31) // 32)
-    n = -(-num_tokens * per_chunk // LINEAR_BLOCKS)
-    return max(LINEAR_MIN_CHUNK, -(-n // 64) * 64)
+    n = -(-num_tokens * _linear_blocks(num_heads, dim, vdim) // LINEAR_BLOCKS)
+    return max(LINEAR_MIN_CHUNK, -(-n // 8) * 8)
 
 
-def linear_held_chunks(max_tokens: int, num_heads: int, vdim: int) -> int:
+def linear_held_chunks(max_tokens: int, num_heads: int, dim: int, vdim: int) -> int:
     """The most chunks that requests with more than one chunk can have in a step of up to `max_tokens` tokens: a request of n tokens has
     fewer than 2 n / len."""
-    per_chunk = num_heads * ((vdim + 31) // 32)
-    return min(2 * max_tokens // LINEAR_MIN_CHUNK, 2 * LINEAR_BLOCKS // per_chunk) + 2
+    return min(2 * max_tokens // LINEAR_MIN_CHUNK, 2 * LINEAR_BLOCKS // _linear_blocks(num_heads, dim, vdim)) + 2
 
 
 def linear_scan(out: torch.Tensor, packed: torch.Tensor, q_off: int, k_off: int, v_off: int, qk_scale: float, gg: torch.Tensor,
@@ -828,13 +832,13 @@ def _lru_check(packed, width, parts, y_off, x_off, vectors, ints):
 def lru_chunk_tokens(num_tokens: int, width: int) -> int:
     """Tokens per chunk of a request's portion: short enough that a long prompt's chunks fill the SMs, long enough that the chunks
     before a chunk are few."""
-    n = -(-num_tokens * (-(-width // 128)) // LINEAR_BLOCKS)
+    n = -(-num_tokens * (-(-width // 128)) // LRU_BLOCKS)
     return max(32, min(256, -(-n // 32) * 32))
 
 
 def lru_most_chunks(max_tokens: int, max_seqs: int, width: int) -> int:
     """The most chunks a step of up to `max_tokens` tokens of `max_seqs` requests can have."""
-    return max(LINEAR_BLOCKS // (-(-width // 128)), max_tokens // 256) + 2 + max_seqs
+    return max(LRU_BLOCKS // (-(-width // 128)), max_tokens // 256) + 2 + max_seqs
 
 
 def lru_conv(u: torch.Tensor, packed: torch.Tensor, y_off: int, x_off: int, parts: int, bias_x, conv_w, conv_b, state, seq_of_token, cu_seqlens,

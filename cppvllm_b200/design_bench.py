@@ -920,8 +920,8 @@ def sumevik_kernel_pairs(s, pk):
     vf, o32 = torch.zeros(T, HV, dtype=f32, device=d), torch.empty(T, HV, dtype=f32, device=d)
     y_lin = torch.empty(T, HV, dtype=bf, device=d)
     state = torch.zeros(2, H * dk * hd, dtype=f32, device=d)
-    chunk = ops.linear_chunk_tokens(T, H, hd)
-    held = ops.linear_held_chunks(T, H, hd)
+    chunk = ops.linear_chunk_tokens(T, H, dk, hd)
+    held = ops.linear_held_chunks(T, H, dk, hd)
     ends, decays = torch.empty(held * H * dk * hd, dtype=f32, device=d), torch.empty(held * H * dk, dtype=f32, device=d)
 
     def core(i):                                 # as parts/recurrent.py does for portions of prompts

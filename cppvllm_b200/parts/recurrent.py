@@ -276,10 +276,10 @@ class GatedLinearMixer(Mixer):
         ops.linear_decay(z, self.b_a2, self.tau)
         o = ws.rows("rec_o", T, H * dv, f32)
         q_lens = ctx.q_lens if ctx.q_lens is not None else [1] * S
-        chunk = ops.linear_chunk_tokens(T, H, dv)
+        chunk = ops.linear_chunk_tokens(T, H, dk, dv)
         ends = decays = None
         if max(q_lens) > chunk:
-            held = ops.linear_held_chunks(ws.max_tokens, H, dv)
+            held = ops.linear_held_chunks(ws.max_tokens, H, dk, dv)
             ends = ws.flat(f"linear_ends_{H}_{dk}_{dv}", held * H * dk * dv, f32)
             decays = ws.flat(f"linear_decays_{H}_{dk}_{dv}", held * H * dk, f32)
         ops.linear_scan(o, packed, q_off, k_off, v_off, qk_scale, z, state, ctx.cu_seqlens, ctx.state_slots, q_lens, H, dk, dv, chunk, ends, decays)

@@ -233,10 +233,10 @@ def test_members_of_a_pair_keep_one_cache_and_one_state():
 def test_chunk_scratch_is_large_enough(T, q_lens):
     """The buffers that are sized once for the largest step hold the chunks of every smaller one."""
     from cppvllm_b200.csrc import ops
-    for H, dv in ((1, 8), (6, 64), (16, 128), (64, 256)):
-        n = ops.linear_chunk_tokens(T, H, dv)
+    for H, dk, dv in ((1, 4, 8), (6, 48, 64), (16, 64, 128), (64, 300, 256)):
+        n = ops.linear_chunk_tokens(T, H, dk, dv)
         held = sum(c for c in (-(-q // n) for q in q_lens) if c > 1)
-        assert n % 8 == 0 and held <= ops.linear_held_chunks(max(T, 64), H, dv) and held <= ops.linear_held_chunks(8192, H, dv)
+        assert n % 8 == 0 and held <= ops.linear_held_chunks(max(T, 64), H, dk, dv) and held <= ops.linear_held_chunks(8192, H, dk, dv)
     for W in (24, 160, 1024, 4096):
         n = ops.lru_chunk_tokens(T, W)
         assert sum(-(-q // n) for q in q_lens) <= ops.lru_most_chunks(8192, len(q_lens), W)
