@@ -33,9 +33,7 @@
 
 namespace cvb {
 
-constexpr int kRouteWarps = 8;          // many tokens: warps per block, which share kRouteTokens tokens
-constexpr int kRouteTokens = 8;
-constexpr int kRouteFewWarps = 8;       // few tokens: the warps of a block share one token's router outputs out
+constexpr int kRouteWarps = 8;          // warps of a block, which share its tokens' rows out
 
 // The choice from the logits z [E] (shared memory of the calling warp; in mode 3 with 2 E + groups floats): see the top of this file.
 __device__ __forceinline__ void route_select(float* z, int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ bias,
@@ -120,70 +118,75 @@ template <int V> __device__ __forceinline__ void route_load(const __nv_bfloat16*
     } else f[0] = __bfloat162float(p[0]);
 }
 
-// Many tokens: a block takes kRouteTokens tokens, its warps a slice of D each.  A warp holds all the block's tokens by four router
-// outputs in registers, so a weight it loads serves eight tokens and an activation four outputs; the warps' parts meet in shared
-// memory in a fixed order.
-template <typename T, int V>
+// A block takes NT tokens, its warps a slice of D each.  A warp holds the block's tokens by NE router outputs in registers, so a
+// weight it loads serves NT tokens and an activation NE outputs; the warps' parts meet in shared memory in a fixed order.  NT = 8,
+// NE = 4 for many tokens; NT = 1, NE = 16 for few (every row of the router in flight at once).
+template <typename T, int V, int NT, int NE>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x, const float* __restrict__ wr,
                   const float* __restrict__ bias, int n_tokens, int D, int E, int top, int mode, float scale, int extra,
                   float* __restrict__ extra_out, int groups, int keep) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ float smem[];                     // [kRouteTokens][E] (mode 3: [..][2 E + groups]), then a round's parts
+    constexpr int NV = NT * NE, kSpan = 32 / NV;        // sums per warp and round; lanes that end with the same one
+    static_assert(NV == 16 || NV == 32, "a butterfly over the warp");
+    extern __shared__ float smem[];                     // [NT][E] (mode 3: [..][2 E + groups]), then a round's parts
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kRouteTokens;
-    const int nt = static_cast<int>(n_tokens - t0 < kRouteTokens ? n_tokens - t0 : kRouteTokens);
+    const int64_t t0 = static_cast<int64_t>(blockIdx.x) * NT;
+    const int nt = static_cast<int>(n_tokens - t0 < NT ? n_tokens - t0 : NT), n_out = E + extra;
     const int per = mode == 3 ? 2 * E + groups : E;
-    float* part = smem + kRouteTokens * per;            // [kRouteWarps][kRouteTokens * 4]
-    const T* xr[kRouteTokens];
+    float* part = smem + NT * per;                      // [kRouteWarps][NV]
+    const T* xr[NT];
 #pragma unroll
-    for (int k = 0; k < kRouteTokens; ++k) xr[k] = x + (t0 + min(k, nt - 1)) * D;       // rows past the end repeat the last one
-    for (int e0 = 0; e0 < E + extra; e0 += 4) {
-        const float* w[4];
+    for (int k = 0; k < NT; ++k) xr[k] = x + (t0 + min(k, nt - 1)) * D;       // rows past the end repeat the last one
+    for (int e0 = 0; e0 < n_out; e0 += NE) {
+        const float* w = wr + static_cast<int64_t>(e0) * D;
+        float r[NV];                                    // [token][output]
 #pragma unroll
-        for (int q = 0; q < 4; ++q) w[q] = wr + static_cast<int64_t>(min(e0 + q, E + extra - 1)) * D;
-        float d[kRouteTokens][4];
-#pragma unroll
-        for (int k = 0; k < kRouteTokens; ++k) { d[k][0] = d[k][1] = d[k][2] = d[k][3] = 0.f; }
+        for (int i = 0; i < NV; ++i) r[i] = 0.f;
+#pragma unroll 2
         for (int i = (warp * 32 + lane) * V; i < D; i += kRouteWarps * 32 * V) {
-            float wv[4][V];
+            float wv[NE][V];
 #pragma unroll
-            for (int q = 0; q < 4; ++q) route_load<V>(w[q] + i, wv[q]);
+            for (int q = 0; q < NE; ++q) {
+                if (e0 + q < n_out) route_load<V>(w + static_cast<int64_t>(q) * D + i, wv[q]);
+                else {
 #pragma unroll
-            for (int k = 0; k < kRouteTokens; ++k) {
+                    for (int v = 0; v < V; ++v) wv[q][v] = 0.f;
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < NT; ++k) {
                 float xv[V];
                 route_load<V>(xr[k] + i, xv);
 #pragma unroll
-                for (int q = 0; q < 4; ++q)
+                for (int q = 0; q < NE; ++q)
 #pragma unroll
-                    for (int v = 0; v < V; ++v) d[k][q] = fmaf(xv[v], wv[q][v], d[k][q]);
+                    for (int v = 0; v < V; ++v) r[k * NE + q] = fmaf(xv[v], wv[q][v], r[k * NE + q]);
             }
         }
-        // 32 sums over 32 lanes: lane 4 k + q ends with the sum of (k, q), by a transposing butterfly
-        float r[kRouteTokens * 4];
+        // NV sums over 32 lanes by a transposing butterfly: lane l ends with sum l / kSpan
+        int mask = 16;
 #pragma unroll
-        for (int k = 0; k < kRouteTokens; ++k)
-#pragma unroll
-            for (int q = 0; q < 4; ++q) r[k * 4 + q] = d[k][q];
-#pragma unroll
-        for (int half = 16; half > 0; half >>= 1) {
-            const bool up = (lane & half) != 0;
+        for (int half = NV / 2; half > 0; half >>= 1, mask >>= 1) {
+            const bool up = (lane & mask) != 0;
 #pragma unroll
             for (int i = 0; i < half; ++i) {
                 const float away = up ? r[i] : r[i + half], own = up ? r[i + half] : r[i];
-                r[i] = own + __shfl_xor_sync(0xffffffffu, away, half);
+                r[i] = own + __shfl_xor_sync(0xffffffffu, away, mask);
             }
         }
+#pragma unroll
+        for (; mask > 0; mask >>= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], mask);
         __syncthreads();                                // the round before has been read
-        part[warp * 32 + lane] = r[0];
+        if (lane % kSpan == 0) part[warp * NV + lane / kSpan] = r[0];
         __syncthreads();
-        if (warp == 0) {
+        if (warp == 0 && lane < NV) {
             float v = 0.f;
 #pragma unroll
-            for (int g = 0; g < kRouteWarps; ++g) v += part[g * 32 + lane];
-            const int k = lane >> 2, e = e0 + (lane & 3);
-            if (k < nt && e < E + extra) {
+            for (int g = 0; g < kRouteWarps; ++g) v += part[g * NV + lane];
+            const int k = lane / NE, e = e0 + lane % NE;
+            if (k < nt && e < n_out) {
                 if (e < E) smem[k * per + e] = v + (bias && mode != 3 ? bias[e] : 0.f);
                 else extra_out[(t0 + k) * extra + (e - E)] = v;
             }
@@ -191,39 +194,6 @@ route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* _
     }
     __syncthreads();
     for (int k = warp; k < nt; k += kRouteWarps) route_select(smem + k * per, ids, weights, bias, t0 + k, E, top, mode, scale, groups, keep, lane);
-}
-
-// Few tokens: a block per token; its warps take the router outputs in turn.
-template <typename T, int V>
-__global__ void __launch_bounds__(kRouteFewWarps * 32)
-route_topk_few_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x, const float* __restrict__ wr,
-                      const float* __restrict__ bias, int D, int E, int top, int mode, float scale, int extra,
-                      float* __restrict__ extra_out, int groups, int keep) {
-    pdl_trigger();
-    pdl_wait();
-    extern __shared__ float smem[];                     // [E], mode 3: [2 E + groups]
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int64_t t = blockIdx.x;
-    const T* xr = x + t * D;
-    for (int e = warp; e < E + extra; e += kRouteFewWarps) {
-        const float* w = wr + static_cast<int64_t>(e) * D;
-        float d = 0.f;
-#pragma unroll 8
-        for (int i = lane * V; i < D; i += 32 * V) {
-            float wv[V], xv[V];
-            route_load<V>(w + i, wv);
-            route_load<V>(xr + i, xv);
-#pragma unroll
-            for (int v = 0; v < V; ++v) d = fmaf(xv[v], wv[v], d);
-        }
-        d = warp_sum(d);
-        if (lane == 0) {
-            if (e < E) smem[e] = d + (bias && mode != 3 ? bias[e] : 0.f);
-            else extra_out[t * extra + (e - E)] = d;
-        }
-    }
-    __syncthreads();
-    if (warp == 0) route_select(smem, ids, weights, bias, t, E, top, mode, scale, groups, keep, lane);
 }
 
 constexpr int kExpertThreads = 256;
@@ -471,28 +441,23 @@ extern "C" int cvb_route_topk(int* ids, float* weights, const void* x, const flo
     if (mode < 0 || mode > 3) return CVB_E_SHAPE;
     if (top > E || E > 2048) return CVB_E_SHAPE;
     if (mode == 3 && (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups))) return CVB_E_SHAPE;
-    const size_t row = static_cast<size_t>(mode == 3 ? 2 * E + groups : E) * sizeof(float);
-    const size_t parts = static_cast<size_t>(kRouteWarps) * kRouteTokens * 4 * sizeof(float);
-    if (row * kRouteTokens + parts > 200 * 1024) return CVB_E_SIZE;
     const bool few = T <= 512;
+    const int nt = few ? 1 : 8;
+    const size_t smem = (static_cast<size_t>(nt) * (mode == 3 ? 2 * E + groups : E) + kRouteWarps * 32) * sizeof(float);
+    if (smem > 200 * 1024) return CVB_E_SIZE;
     const bool four = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(wr)) & 15) == 0;
-    const size_t smem = few ? row : row * kRouteTokens + parts;
-#define CALL_V(TY, V)                                                                                                         \
+#define CALL_N(TY, V, NT, NE)                                                                                                 \
     do {                                                                                                                      \
-        if (few) {                                                                                                            \
-            launch_kernel(route_topk_few_kernel<TY, V>, dim3(T), dim3(kRouteFewWarps * 32), smem, stream, ids, weights, (const TY*)x, wr, bias, \
-                          D, E, top, mode, scale, extra, extra_out, groups, keep);                                            \
-        } else {                                                                                                              \
-            if (smem > 48 * 1024) cudaFuncSetAttribute(route_topk_kernel<TY, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
-            launch_kernel(route_topk_kernel<TY, V>, dim3((T + kRouteTokens - 1) / kRouteTokens),                  \
-                          dim3(kRouteWarps * 32), smem, stream, ids, weights, (const TY*)x, wr, bias, T, D, E, top, mode, scale, extra,         \
-                          extra_out, groups, keep);                                                                           \
-        }                                                                                                                     \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(route_topk_kernel<TY, V, NT, NE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        launch_kernel(route_topk_kernel<TY, V, NT, NE>, dim3((T + NT - 1) / NT), dim3(kRouteWarps * 32), smem, stream, ids, weights,  \
+                      (const TY*)x, wr, bias, T, D, E, top, mode, scale, extra, extra_out, groups, keep);                       \
     } while (0)
+#define CALL_V(TY, V) if (few) CALL_N(TY, V, 1, 16); else CALL_N(TY, V, 8, 4)
 #define CALL(TY) if (four) { CALL_V(TY, 4); } else { CALL_V(TY, 1); }
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
 #undef CALL_V
+#undef CALL_N
     return launch_status();
 }
 
