@@ -13,7 +13,8 @@
 // of a kv head is `ew` >= hd elements wide, its first hd elements are the key and the vd elements from `voff` on are the
 // value (ew = hd, voff = 0: the key's leading elements; ew = hd + vd, voff = hd: a key with its own value behind it, of
 // any size).  With a distance table `bias` [H, bias_len] (float) the score receives bias[h, min(p - j, bias_len - 1)] after
-// the scale: a learned bias per head and distance, whose last entry serves every larger distance.
+// the scale: a learned bias per head and distance, whose last entry serves every larger distance.  With `sink` [H] the softmax's
+// denominator also holds exp(sink_h), a term without key or value; outputs are multiplied by `out_scale`.
 //
 // Formulas (reference kernels/paged_attention.cu:89-359 and model/model_architecture.cpp:134,147):
 //   query head h uses kv head h / (H / KV);  s_j = scale * q . k_j  for lo <= j <= p, others excluded;
@@ -34,7 +35,7 @@ paged_attention_general_kernel(T* __restrict__ out, const T* __restrict__ q, con
                                const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                                int H, int KV, int hd, int vd, int page_size, int window, int keep_first, int planes, int q_stride,
                                float scale, int num_pages, int ew, int voff_in_entry, const float* __restrict__ bias, int bias_len,
-                               int* __restrict__ err) {
+                               const float* __restrict__ sink, float out_scale, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ int64_t smem64[];
@@ -59,6 +60,7 @@ paged_attention_general_kernel(T* __restrict__ out, const T* __restrict__ q, con
 #pragma unroll
     for (int i = 0; i < kMaxDimsPerThread; ++i) acc[i] = 0.f;
     float m = -INFINITY, l = 0.f;
+    if (sink != nullptr) { m = sink[h]; l = 1.f; }
 
     const int kept = min(keep_first, lo);               // positions 0..kept-1 lie before the window and stay visible
     for (int run = kept > 0 ? 0 : 1; run < 2; ++run) {
@@ -107,7 +109,7 @@ paged_attention_general_kernel(T* __restrict__ out, const T* __restrict__ q, con
         __syncthreads();
     }
     }
-    const float inv_l = l > 0.f ? 1.f / l : 0.f;
+    const float inv_l = l > 0.f ? out_scale / l : 0.f;
 #pragma unroll
     for (int i = 0; i < kMaxDimsPerThread; ++i) {
         const int d = tid + i * kAttnThreads;
@@ -123,7 +125,7 @@ static int attention_general_launch(void* out, const void* q, const void* cache,
                                     int table_width, const int* seq_of_token, const int* positions, int T,
                                     int H, int KV, int hd, int vd, int page_size, int window, int keep_first, int planes,
                                     int q_stride, float scale, int num_pages, int ew, int voff, const float* bias, int bias_len,
-                                    int dtype, int* err_flag, cudaStream_t stream) {
+                                    const float* sink, float out_scale, int dtype, int* err_flag, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
     if (T < 0 || H <= 0 || KV <= 0 || hd <= 0 || page_size <= 0 || table_width <= 0 || num_pages <= 0)
         return CVB_E_SIZE;
@@ -137,7 +139,7 @@ static int attention_general_launch(void* out, const void* q, const void* cache,
 #define CALL(TY)                                                                                         \
     launch_kernel(paged_attention_general_kernel<TY>, dim3(grid), dim3(kAttnThreads), smem, stream,                             \
         (TY*)out, (const TY*)q, (const TY*)cache, block_tables, table_width, seq_of_token, positions, H, \
-        KV, hd, vd, page_size, window, keep_first, planes, q_stride, scale, num_pages, ew, voff, bias, bias_len, err_flag)
+        KV, hd, vd, page_size, window, keep_first, planes, q_stride, scale, num_pages, ew, voff, bias, bias_len, sink, out_scale, err_flag)
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
     return launch_status();
@@ -146,11 +148,11 @@ static int attention_general_launch(void* out, const void* q, const void* cache,
 extern "C" int cvb_paged_attention_general(void* out, const void* q, const void* cache, const int* block_tables,
                                            int table_width, const int* seq_of_token, const int* positions, int T,
                                            int H, int KV, int hd, int vd, int page_size, int window, int keep_first, int planes,
-                                           int q_stride, float scale, int num_pages, int dtype, int* err_flag,
-                                           cudaStream_t stream) {
+                                           int q_stride, float scale, int num_pages, const float* sink, float out_scale, int dtype,
+                                           int* err_flag, cudaStream_t stream) {
     if (vd <= 0 || vd > hd) return CVB_E_SHAPE;
     return attention_general_launch(out, q, cache, block_tables, table_width, seq_of_token, positions, T, H, KV, hd, vd, page_size,
-                                    window, keep_first, planes, q_stride, scale, num_pages, hd, 0, nullptr, 0, dtype, err_flag, stream);
+                                    window, keep_first, planes, q_stride, scale, num_pages, hd, 0, nullptr, 0, sink, out_scale, dtype, err_flag, stream);
 }
 
 // Entries [key (hd) | value (vd)] per kv head (pages [page, kv head, slot, hd + vd]) and an optional distance table.
@@ -160,5 +162,5 @@ extern "C" int cvb_paged_attention_entries(void* out, const void* q, const void*
                                            int num_pages, const float* bias, int bias_len, int dtype, int* err_flag,
                                            cudaStream_t stream) {
     return attention_general_launch(out, q, cache, block_tables, table_width, seq_of_token, positions, T, H, KV, hd, vd, page_size,
-                                    window, 0, 1, q_stride, scale, num_pages, hd + vd, hd, bias, bias_len, dtype, err_flag, stream);
+                                    window, 0, 1, q_stride, scale, num_pages, hd + vd, hd, bias, bias_len, nullptr, 1.f, dtype, err_flag, stream);
 }

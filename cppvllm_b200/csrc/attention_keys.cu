@@ -15,6 +15,8 @@
 // which makes every ldmatrix conflict-free for all head sizes that are multiples of 16.
 // The value may be narrower than the key (`vd` <= HD, a multiple of 16): only the first vd elements of a key are its value
 // (a latent vector with a positional part behind it); O += P K then stops at column vd and the output rows are [T, H, vd].
+// With `sink` [H] the softmax's denominator also holds exp(sink_h), a term without key or value: it starts a row's maximum and sum
+// (portions) or joins where the parts are merged, once (decoded tokens).  Outputs are multiplied by `out_scale`.
 #include "common.cuh"
 #include "sm100.cuh"
 #include "mma_tiles.cuh"
@@ -43,6 +45,8 @@ struct KeysAttnParams {
     int splits;
     float* parts;                       // [S, KV, splits, 16, HD + 2]
     float scale_log2;                   // scale * log2(e)
+    const float* sink;                  // [H] or null
+    float out_scale;
     int* err;
 };
 
@@ -135,6 +139,14 @@ attn_keys_kernel(const KeysAttnParams p) {
         row_hi[half] = pos_first + tok;
         row_lo[half] = p.window > 0 ? max(0, row_hi[half] - p.window + 1) : 0;
     }
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    if (p.sink != nullptr) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            m[half] = p.sink[kvh * g + (warp * 16 + (lane >> 2) + half * 8) % g] * kLog2eKeys;
+            l[half] = (lane & 3) == 0 ? 1.f : 0.f;        // the four threads of a row add their sums up at the end
+        }
+    }
     const bool warp_has_rows = warp * 16 < n_tok * g;
     const int warp_last_pos = pos_first + min(n_tok - 1, (warp * 16 + 15) / g);
     const int warp_first_pos = pos_first + min(n_tok - 1, (warp * 16) / g);
@@ -143,7 +155,6 @@ attn_keys_kernel(const KeysAttnParams p) {
     float o[HD / 8][4];
 #pragma unroll
     for (int dt = 0; dt < HD / 8; ++dt) { o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f; }
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     uint32_t qf[HD / 16][4];
 
     for (int it = 0; it < n_tiles; ++it) {
@@ -244,7 +255,7 @@ attn_keys_kernel(const KeysAttnParams p) {
         const int r = warp * 16 + (lane >> 2) + half * 8;
         const int tok = r / g;
         if (tok >= n_tok) continue;
-        const float inv = l[half] > 0.f ? 1.f / l[half] : 0.f;
+        const float inv = l[half] > 0.f ? p.out_scale / l[half] : 0.f;
         __nv_bfloat16* dst = p.out + (static_cast<int64_t>(cu0 + q0 + tok) * p.H + kvh * g + r % g) * p.vd;
 #pragma unroll
         for (int dt = 0; dt < HD / 8; ++dt) {
@@ -267,6 +278,18 @@ attn_keys_kernel(const KeysAttnParams p) {
 // dependencies), two warps per scheduler with half the instructions each overlap.
 constexpr int kDecWarps = 8;
 constexpr int kDecKeys = 32;                             // keys per tile of the decode form
+
+// A row's merged accumulator, maximum and sum become its output element; the sink joins here.
+__device__ __forceinline__ void keys_finish(const KeysAttnParams& p, int t, int head, int d, float mm, float ll, float acc) {
+    if (p.sink != nullptr) {
+        const float sk = p.sink[head] * kLog2eKeys;
+        const float top = fmaxf(mm, sk);
+        const float f = mm == -INFINITY ? 0.f : ex2(mm - top);
+        ll = ll * f + ex2(sk - top);
+        acc *= f;
+    }
+    p.out[(static_cast<int64_t>(t) * p.H + head) * p.vd + d] = __float2bfloat16_rn(ll > 0.f ? acc / ll * p.out_scale : 0.f);
+}
 
 template <int HD>
 __global__ void __launch_bounds__(kDecWarps * 32)
@@ -460,7 +483,7 @@ attn_keys_decode_kernel(const KeysAttnParams p) {
             acc += reinterpret_cast<const float*>(sK + w * 2 * kDecKeys * LD)[r * HD + d] * f;
         }
         if (p.splits == 1) {
-            p.out[(static_cast<int64_t>(t) * p.H + kvh * g + r) * p.vd + d] = __float2bfloat16_rn(ll > 0.f ? acc / ll : 0.f);
+            keys_finish(p, t, kvh * g + r, d, mm, ll, acc);
         } else {
             float* dst = p.parts + ((static_cast<int64_t>(seq) * p.KV + kvh) * p.splits + blockIdx.z) * 16 * (HD + 2) + r * (HD + 2);
             dst[d] = acc;
@@ -490,7 +513,7 @@ __global__ void attn_keys_merge_kernel(const KeysAttnParams p) {
             ll += row[HD + 1] * f;
             acc += row[d] * f;
         }
-        p.out[(static_cast<int64_t>(t) * p.H + kvh * g + r) * p.vd + d] = __float2bfloat16_rn(ll > 0.f ? acc / ll : 0.f);
+        keys_finish(p, t, kvh * g + r, d, mm, ll, acc);
     }
 }
 
@@ -533,7 +556,7 @@ extern "C" int cvb_attn_keys_supported(int H, int KV, int hd) {
 extern "C" int cvb_attn_keys_bf16(void* out, const void* q, int q_stride, const void* pages, const int* block_tables,
                                   int table_width, const int* cu_seqlens, const int* positions, int S, int num_tiles, int H,
                                   int KV, int hd, int vd, int page_size, int window, int keep_first, float scale, int num_pages,
-                                  int all_single, int splits, float* parts, int64_t parts_floats, int kv_phys, int* err_flag,
+                                  int all_single, int splits, float* parts, int64_t parts_floats, int kv_phys, const float* sink, float out_scale, int* err_flag,
                                   cudaStream_t stream) {
     if (num_tiles == 0 || S == 0) return CVB_OK;
     if (S < 0 || num_tiles < 0 || page_size <= 0 || table_width <= 0 || num_pages <= 0 || window < 0 || keep_first < 0) return CVB_E_SIZE;
@@ -555,6 +578,7 @@ extern "C" int cvb_attn_keys_bf16(void* out, const void* q, int q_stride, const 
     for (int sh = 0; sh < 31; ++sh)
         if ((1 << sh) == page_size) p.page_shift = sh;
     p.scale_log2 = scale * kLog2eKeys;
+    p.sink = sink; p.out_scale = out_scale;
     p.err = err_flag;
     p.splits = 1; p.parts = nullptr;
     if (all_single && H / KV <= 16 && splits > 1) {

@@ -4,7 +4,8 @@
 //   visible keys of the token at position p:  lo <= j <= p  with
 //       lo = 0                                   (all earlier tokens)
 //       lo = floor(p / C) * C                    `chunk` = C > 0: only the token's own chunk, counted from position 0
-//       lo = max(0, p - W + 1)                   `window` = W > 0: the last W tokens
+//       lo = max(0, p - W + 1)                   `window` = W > 0: the last W tokens; with `keep` = K > 0 also j < K: the first K tokens
+//                                                stay visible for ever
 //   and, with `pool` = P > 0 beside a window, one entry per block b of P tokens (positions bP .. bP + P - 1) that lies wholly
 //   before the window, bP + P - 1 <= p - W: the means of the block's keys and values as the cache holds them, kept in a
 //   second plane of the same pages at the place of position b.  Tokens and blocks share one softmax.
@@ -146,7 +147,8 @@ masked_qkv_prep_pairs_kernel(T* __restrict__ q_out, const T* __restrict__ packed
     }
 }
 
-// ---- 16 bytes per thread: head sizes whose chunk count is a power of two, a rotation in pairs (2i, 2i + 1) or none ------------
+// ---- 16 bytes per thread: head sizes whose chunk count is a power of two; a rotation in pairs (2i, 2i + 1), in pairs (i, i + rot / 2)
+// where half the rotation is whole chunks (the partner's chunk is read beside the own one), or none -----------------------------
 //
 // One thread owns one 16-byte chunk of a head (8 bf16 or 4 float elements, whole pairs); the dk / N threads of a query or key
 // head are neighbours in a warp, so the sum of squares is a butterfly over the group.  The threads of a token are laid out as
@@ -180,7 +182,7 @@ masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, 
                            const float* __restrict__ k_w, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                            const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ pages,
                            T* __restrict__ vfirst_out, const T* __restrict__ vfirst_in, const float* __restrict__ lam_p,
-                           int H, int G, int dk, int dv, int rot, int planes, int page_size, int max_pos, float eps,
+                           int H, int G, int dk, int dv, int rot, int interleaved, int planes, int page_size, int max_pos, float eps,
                            int64_t total_slots, int qk_pad, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
@@ -227,11 +229,22 @@ masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, 
     const bool live = idx < (H + G) * chk && (is_q || entry >= 0);
     const float* w = is_q ? q_w : k_w;
     float ss = 0.f;
+    const int half = rot >> 1;
+    const bool turned = cos_t != nullptr && c * N < rot;
+    const int mate = c * N < half ? c + half / N : c - half / N;          // the chunk of the partners (i, i + rot / 2)
+    float u[N];
     if (live) {
         Chunk16<T>::load(v, row + task * dk + c * N);   // key heads lie behind the query heads in the row
         if (bias != nullptr) {
 #pragma unroll
             for (int i = 0; i < N; ++i) v[i] += bias[task * dk + c * N + i];
+        }
+        if (turned && !interleaved) {
+            Chunk16<T>::load(u, row + task * dk + mate * N);
+            if (bias != nullptr) {
+#pragma unroll
+                for (int i = 0; i < N; ++i) u[i] += bias[task * dk + mate * N + i];
+            }
         }
 #pragma unroll
         for (int i = 0; i < N; ++i) ss = fmaf(v[i], v[i], ss);
@@ -242,11 +255,14 @@ masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, 
         if (live) {
 #pragma unroll
             for (int i = 0; i < N; ++i) v[i] = v[i] * inv * w[c * N + i];
+            if (turned && !interleaved) {
+#pragma unroll
+                for (int i = 0; i < N; ++i) u[i] = u[i] * inv * w[mate * N + i];
+            }
         }
     }
     if (!live) return;
-    const int half = rot >> 1;
-    if (cos_t != nullptr && c * N < rot) {
+    if (turned) {
         int pos = positions[t];
         if (pos < 0 || pos >= max_pos) {
             atomicExch(err, 3);
@@ -254,8 +270,18 @@ masked_qkv_prep_vec_kernel(T* __restrict__ q_out, const T* __restrict__ packed, 
         }
         const float* c_row = cos_t + static_cast<int64_t>(pos) * half;
         const float* s_row = sin_t + static_cast<int64_t>(pos) * half;
+        if (!interleaved) {
+            const bool low = c * N < half;
+            const int p0 = low ? c * N : c * N - half;
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                const float cs = c_row[p0 + i], sn = s_row[p0 + i];
+                v[i] = low ? v[i] * cs - u[i] * sn : v[i] * cs + u[i] * sn;
+            }
+        }
 #pragma unroll
         for (int i = 0; i < N; i += 2) {
+            if (!interleaved) break;
             const int pr = (c * N + i) >> 1;
             if (pr < half) {
                 const float cs = c_row[pr], sn = s_row[pr], x0 = v[i], x1 = v[i + 1];
@@ -400,7 +426,7 @@ constexpr int kMaskedThreads = 128;
 constexpr int kMaskedDimsPerThread = 8;
 
 struct MaskParams {
-    int chunk, window, pool;
+    int chunk, window, pool, keep;      // keep: with a window, the first tokens that stay visible
     float scale, softcap;
 };
 
@@ -443,8 +469,8 @@ attn_masked_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T
     if (sink != nullptr) { m = sink[h]; l = 1.f; }
     const float b1 = r1 != nullptr ? r1[h] : 0.f, b2 = r2 != nullptr ? r2[h] : 0.f;
     const int lo = first_visible(p, mp), nb = visible_blocks(p, mp);
-    for (int run = nb > 0 ? 0 : 1; run < 2; ++run) {
-        const int first = run == 0 ? 0 : lo, last = run == 0 ? nb - 1 : p, plane = run == 0 ? 1 : 0;
+    for (int run = 0; run < 3; ++run) {                 // the pooled blocks, the kept first tokens before `lo`, the tokens from `lo` on
+        const int first = run == 2 ? lo : 0, last = run == 0 ? nb - 1 : (run == 1 ? min(mp.keep, lo) - 1 : p), plane = run == 0 ? 1 : 0;
         for (int start = first; start <= last; start += kMaskedThreads) {
             const int j = start + tid;
             float s = -INFINITY;
@@ -462,7 +488,7 @@ attn_masked_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T
                     for (int e = 0; e < dk; ++e) d = fmaf(qs[e], to_float(kp[e]), d);
                     s = d * mp.scale;
                     if (mp.softcap > 0.f) s = mp.softcap * tanhf(s / mp.softcap);
-                    if (r1 != nullptr && run == 1) s -= b1 * log1pf(b2 * static_cast<float>(p - j));
+                    if (r1 != nullptr && run > 0) s -= b1 * log1pf(b2 * static_cast<float>(p - j));
                 }
             }
             const float tile_max = block_max(s, scratch);
@@ -570,8 +596,15 @@ attn_masked_kernel(const MaskedAttnParams p) {
     // both bounds grow with the position: the block's first token sees the earliest token, its last one the most blocks
     const int nb_max = visible_blocks(key_hi, p.mp);
     const int n_pool_tiles = (nb_max + kMTileKeys - 1) / kMTileKeys;
-    const int tok_tile0 = first_visible(pos_first, p.mp) / kMTileKeys;
-    const int n_tiles = n_pool_tiles + key_hi / kMTileKeys - tok_tile0 + 1;
+    const int key_lo = first_visible(pos_first, p.mp), keep = p.mp.keep;
+    const int tok_tile0 = key_lo / kMTileKeys;
+    const int n_kept = keep > 0 ? min((keep - 1) / kMTileKeys + 1, tok_tile0) : 0;      // tiles of kept first tokens, wholly before the others
+    const int n_tiles = n_pool_tiles + n_kept + key_hi / kMTileKeys - tok_tile0 + 1;
+    auto first_key = [&](int it) {
+        if (it < n_pool_tiles) return it * kMTileKeys;
+        it -= n_pool_tiles;
+        return (it < n_kept ? it : tok_tile0 + it - n_kept) * kMTileKeys;
+    };
 
     for (int i = threadIdx.x; i < kMTileRows * CQ; i += kMThreads) {
         const int r = i / CQ, c = i - r * CQ;
@@ -585,7 +618,7 @@ attn_masked_kernel(const MaskedAttnParams p) {
     const int ld_dr = kMThreads / CE, ld_dc = kMThreads - ld_dr * CE;
     auto load_tile = [&](int it, int stage) {
         const bool pooled = it < n_pool_tiles;
-        const int key0 = pooled ? it * kMTileKeys : (tok_tile0 + it - n_pool_tiles) * kMTileKeys;
+        const int key0 = first_key(it);
         const int hi = pooled ? nb_max - 1 : key_hi;
         const int plane = pooled ? 1 : 0;
         __nv_bfloat16* dst = sK + stage * kMTileKeys * LD;
@@ -594,7 +627,7 @@ attn_masked_kernel(const MaskedAttnParams p) {
         for (; r < kMTileKeys; r += ld_dr, c += ld_dc) {
             if (c >= CE) { c -= CE; ++r; if (r >= kMTileKeys) break; }
             const int j = key0 + r;
-            bool need = j <= hi;
+            bool need = j <= hi && (pooled || j >= key_lo || j < keep);      // pages before the window may have been given back
             const __nv_bfloat16* src = p.pages;
             if (need) {
                 int slot, off;
@@ -645,7 +678,7 @@ attn_masked_kernel(const MaskedAttnParams p) {
         if (it + 1 < n_tiles) load_tile(it + 1, (it + 1) & 1);
         cp_async_commit();
         const bool pooled = it < n_pool_tiles;
-        const int key0 = pooled ? it * kMTileKeys : (tok_tile0 + it - n_pool_tiles) * kMTileKeys;
+        const int key0 = first_key(it);
         cp_async_wait<1>();                               // everything but the newest group: the query tile and tile `it`
         __syncthreads();
         if (it == 0) {
@@ -655,7 +688,7 @@ attn_masked_kernel(const MaskedAttnParams p) {
                 ldm_x4(qf[ks], sQ + (warp * 16 + (lane & 15)) * LDQ + ks * 16 + (lane >> 4) * 8);
             }
         }
-        const bool wanted = pooled ? key0 < warp_nb : (key0 <= warp_last_pos && key0 + kMTileKeys - 1 >= warp_lo);
+        const bool wanted = pooled ? key0 < warp_nb : (key0 <= warp_last_pos && (key0 + kMTileKeys - 1 >= warp_lo || key0 < keep));
         if (warp_has_rows && wanted) {
             const __nv_bfloat16* tile = sK + (it & 1) * kMTileKeys * LD;
             float s[8][4];
@@ -680,7 +713,7 @@ attn_masked_kernel(const MaskedAttnParams p) {
                 for (int e = 0; e < 4; ++e) {
                     const int half = e >> 1;
                     const int j = key0 + nt * 8 + ((lane & 3) << 1) + (e & 1);
-                    const bool visible = pooled ? j < nb_t[half] : (j >= lo_t[half] && j <= ptok[half]);
+                    const bool visible = pooled ? j < nb_t[half] : ((j >= lo_t[half] || j < keep) && j <= ptok[half]);
                     float v = s[nt][e] * p.mp.scale;
                     if (cap > 0.f) v = cap * tanh_by_exp(v * inv_cap);
                     if (p.r1 != nullptr && !pooled) v -= b1[half] * __logf(1.f + b2[half] * static_cast<float>(max(ptok[half] - j, 0)));
@@ -826,8 +859,15 @@ attn_masked_decode_kernel(const MaskedAttnParams p) {
     const int* table = p.block_tables + static_cast<int64_t>(seq) * p.table_width;
     const int lo = first_visible(pos, p.mp), nb = visible_blocks(pos, p.mp);
     const int n_pool_tiles = (nb + kMDecKeys - 1) / kMDecKeys;
+    const int keep = p.mp.keep;
     const int tok_tile0 = lo / kMDecKeys;
-    const int n_tiles = n_pool_tiles + pos / kMDecKeys - tok_tile0 + 1;
+    const int n_kept = keep > 0 ? min((keep - 1) / kMDecKeys + 1, tok_tile0) : 0;
+    const int n_tiles = n_pool_tiles + n_kept + pos / kMDecKeys - tok_tile0 + 1;
+    auto first_key = [&](int it) {
+        if (it < n_pool_tiles) return it * kMDecKeys;
+        it -= n_pool_tiles;
+        return (it < n_kept ? it : tok_tile0 + it - n_kept) * kMDecKeys;
+    };
 
     for (int i = threadIdx.x; i < 16 * CQ; i += blockDim.x) {
         const int r = i / CQ, c = i - r * CQ;
@@ -841,7 +881,7 @@ attn_masked_decode_kernel(const MaskedAttnParams p) {
     const int ld_dr = 32 / CE, ld_dc = 32 - ld_dr * CE;
     auto load_tile = [&](int it, int stage) {
         const bool pooled = it < n_pool_tiles;
-        const int key0 = pooled ? it * kMDecKeys : (tok_tile0 + it - n_pool_tiles) * kMDecKeys;
+        const int key0 = first_key(it);
         const int hi = pooled ? nb - 1 : pos;
         const int plane = pooled ? 1 : 0;
         __nv_bfloat16* dst = my + stage * kMDecKeys * LD;
@@ -867,7 +907,7 @@ attn_masked_decode_kernel(const MaskedAttnParams p) {
         for (; r < kMDecKeys; r += ld_dr, c += ld_dc) {
             if (c >= CE) { c -= CE; ++r; if (r >= kMDecKeys) break; }
             const int j = key0 + r;
-            bool need = j <= hi;
+            bool need = j <= hi && (pooled || j >= lo || j < keep);
             const __nv_bfloat16* src = p.pages;
             if (need) {
                 int slot, off;
@@ -925,7 +965,7 @@ attn_masked_decode_kernel(const MaskedAttnParams p) {
         cp_async_wait<1>();
         __syncwarp();
         const bool pooled = it < n_pool_tiles;
-        const int key0 = pooled ? it * kMDecKeys : (tok_tile0 + it - n_pool_tiles) * kMDecKeys;
+        const int key0 = first_key(it);
         const __nv_bfloat16* tile = my + (n & 1) * kMDecKeys * LD;
         float s[kMDecKeys / 8][4];
 #pragma unroll
@@ -948,7 +988,7 @@ attn_masked_decode_kernel(const MaskedAttnParams p) {
             for (int e = 0; e < 4; ++e) {
                 const int half = e >> 1;
                 const int j = key0 + nt * 8 + ((lane & 3) << 1) + (e & 1);
-                const bool visible = pooled ? j < nb : (j >= lo && j <= pos);
+                const bool visible = pooled ? j < nb : ((j >= lo || j < keep) && j <= pos);
                 float v = s[nt][e] * p.mp.scale;
                 if (cap > 0.f) v = cap * tanh_by_exp(v * inv_cap);
                 if (p.r1 != nullptr && !pooled) v -= b1[half] * __logf(1.f + b2[half] * static_cast<float>(max(pos - j, 0)));
@@ -1108,13 +1148,13 @@ extern "C" int cvb_masked_qkv_prep(void* q_out, const void* packed, int T, int s
     const size_t smem = static_cast<size_t>(kPrepWarps) * dk * sizeof(float);
     if (smem > 48 * 1024 || grid.y > 65535) return CVB_E_SIZE;
     const bool turns = rot > 0 && cos_t != nullptr;
+    const int n16 = dtype == CVB_DTYPE_BF16 ? 8 : 4;
+    // 16 bytes per thread where a head is a power of two of such chunks and everything is aligned to them
     const bool pairs = dk % 2 == 0 && dv % 2 == 0 && stride % 2 == 0 && dk <= 64 * kPrepPairs && (interleaved || !turns)
                        && ((reinterpret_cast<uintptr_t>(packed) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(pages)
                             | reinterpret_cast<uintptr_t>(vfirst_out) | reinterpret_cast<uintptr_t>(vfirst_in)) & 7) == 0;
-    // 16 bytes per thread where a head is a power of two of such chunks and everything is aligned to them
-    const int n16 = dtype == CVB_DTYPE_BF16 ? 8 : 4;
     const int chk = dk / n16;
-    const bool vec16 = pairs && dk % n16 == 0 && dv % n16 == 0 && stride % n16 == 0 && chk <= 32 && (chk & (chk - 1)) == 0 && rot % 2 == 0
+    const bool vec16 = (interleaved || !turns || (rot / 2) % n16 == 0) && dk % n16 == 0 && dv % n16 == 0 && stride % n16 == 0 && chk <= 32 && (chk & (chk - 1)) == 0 && rot % 2 == 0
                        && ((reinterpret_cast<uintptr_t>(packed) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(pages)
                             | reinterpret_cast<uintptr_t>(vfirst_out) | reinterpret_cast<uintptr_t>(vfirst_in)) & 15) == 0;
     const int qk_pad = vec16 ? ((H + G) * chk + 31) / 32 * 32 : 0;
@@ -1123,7 +1163,7 @@ extern "C" int cvb_masked_qkv_prep(void* q_out, const void* packed, int T, int s
     if (vec16)                                                                                                            \
     launch_kernel(masked_qkv_prep_vec_kernel<TY>, grid16, dim3(128), 0, stream, (TY*)q_out, (const TY*)packed, stride, bias, q_w,           \
                   k_w, cos_t, sin_t, positions, slots, (TY*)pages, (TY*)vfirst_out, (const TY*)vfirst_in, lam, H, G, dk, dv, rot,    \
-                  planes, page_size, max_pos, eps, total_slots, qk_pad, err_flag);                                        \
+                  interleaved, planes, page_size, max_pos, eps, total_slots, qk_pad, err_flag);                                        \
     else if (pairs)                                                                                                       \
     launch_kernel(masked_qkv_prep_pairs_kernel<TY>, grid, dim3(kPrepWarps * 32), 0, stream, (TY*)q_out, (const TY*)packed, stride, bias, q_w, \
                   k_w, cos_t, sin_t, positions, slots, (TY*)pages, (TY*)vfirst_out, (const TY*)vfirst_in, lam, H, G, dk, dv, rot,    \
@@ -1152,17 +1192,17 @@ extern "C" int cvb_pool_entries(void* pages, const int* block_tables, int table_
 
 extern "C" int cvb_attn_masked_general(void* out, const void* q, const void* pages, const int* block_tables, int table_width,
                                        const int* seq_of_token, const int* positions, int T, int H, int G, int dk, int dv,
-                                       int page_size, int planes, int chunk, int window, int pool, float scale, float softcap,
+                                       int page_size, int planes, int chunk, int window, int pool, int keep, float scale, float softcap,
                                        const float* r1, const float* r2, const float* sink, const void* gate, int gate_stride,
                                        int gate_element, float out_scale, int out_stride, int num_pages, int dtype, int* err_flag, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
     if (T < 0 || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || page_size <= 0 || table_width <= 0 || num_pages <= 0) return CVB_E_SIZE;
     if (dv > kMaskedThreads * kMaskedDimsPerThread || H > 65535) return CVB_E_SIZE;
-    if (H % G || chunk < 0 || window < 0 || pool < 0 || (planes != 1 && planes != 2) || (pool > 0 && (planes != 2 || window <= 0)))
+    if (H % G || keep < 0 || (keep > 0 && window <= 0) || chunk < 0 || window < 0 || pool < 0 || (planes != 1 && planes != 2) || (pool > 0 && (planes != 2 || window <= 0)))
         return CVB_E_SHAPE;
     if ((r1 == nullptr) != (r2 == nullptr) || out_stride < H * dv) return CVB_E_SHAPE;
     if (gate != nullptr && gate_stride < (gate_element ? H * dv : H)) return CVB_E_SHAPE;
-    MaskParams mp{chunk, window, pool, scale, softcap};
+    MaskParams mp{chunk, window, pool, keep, scale, softcap};
     const size_t smem = kMaskedThreads * sizeof(int64_t) + (static_cast<size_t>(dk) + kMaskedThreads + 32) * sizeof(float);
     if (smem > 48 * 1024) return CVB_E_SIZE;
 #define CALL(TY)                                                                                                          \
@@ -1182,14 +1222,14 @@ extern "C" int cvb_attn_masked_supported(int H, int G, int dk, int dv) {
 
 extern "C" int cvb_attn_masked_bf16(void* out, const void* q, const void* pages, const int* block_tables, int table_width,
                                     const int* cu_seqlens, const int* positions, int S, int num_tiles, int H, int G, int dk, int dv,
-                                    int page_size, int planes, int chunk, int window, int pool, float scale, float softcap,
+                                    int page_size, int planes, int chunk, int window, int pool, int keep, float scale, float softcap,
                                     const float* r1, const float* r2, const float* sink, const void* gate, int gate_stride,
                                     int gate_element, float out_scale, int out_stride, int num_pages, int all_single, int splits, float* parts, int64_t parts_floats, int* err_flag,
                                     cudaStream_t stream) {
     if (num_tiles == 0 || S == 0) return CVB_OK;
     if (S < 0 || num_tiles < 0 || page_size <= 0 || table_width <= 0 || num_pages <= 0) return CVB_E_SIZE;
     if (!cvb_attn_masked_supported(H, G, dk, dv)) return CVB_E_UNSUPPORTED;
-    if (chunk < 0 || window < 0 || pool < 0 || (planes != 1 && planes != 2) || (pool > 0 && (planes != 2 || window <= 0))) return CVB_E_SHAPE;
+    if (keep < 0 || (keep > 0 && window <= 0) || chunk < 0 || window < 0 || pool < 0 || (planes != 1 && planes != 2) || (pool > 0 && (planes != 2 || window <= 0))) return CVB_E_SHAPE;
     if ((r1 == nullptr) != (r2 == nullptr)) return CVB_E_SHAPE;
     if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(pages)) & 15) return CVB_E_ALIGN;
     if (out_stride < H * dv || (gate != nullptr && gate_stride < (gate_element ? H * dv : H))) return CVB_E_SHAPE;
@@ -1209,7 +1249,7 @@ extern "C" int cvb_attn_masked_bf16(void* out, const void* q, const void* pages,
     p.page_shift = -1;
     for (int sh = 0; sh < 31; ++sh)
         if ((1 << sh) == page_size) p.page_shift = sh;
-    p.mp = MaskParams{chunk, window, pool, scale, softcap};
+    p.mp = MaskParams{chunk, window, pool, keep, scale, softcap};
     p.err = err_flag;
     p.splits = 1; p.parts = nullptr;
     const bool decode = all_single && H / G <= 16;        // every request brings one token: the kernel for decoded tokens

@@ -45,6 +45,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "recurrent": ["recurrent.cu"],
     "lru": ["lru.cu"],
     "linear": ["linear.cu"],
+    "ssd": ["ssd.cu"],
     "sandwich": ["sandwich.cu"],
     "hyper": ["hyper.cu"],
     "attn_masked": ["attention_masked.cu"],

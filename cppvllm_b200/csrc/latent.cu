@@ -9,6 +9,7 @@
 //   latent_q_assemble: the query that the attention kernel reads, per token and head: [q_abs | rot_p(q_rot)], where q_abs
 //                      (the unrotated query taken through the key up-projection, laid out [head, token, rank]) comes from a
 //                      batched product and q_rot is the head's positional part inside the packed query projection.
+//   latent_q_turn    : the same where the batched product has written q_abs to its place already: the turned parts alone.
 //   head_gate        : att[t, h, :] = T( o[h, t, :] * sigmoid(g[t, h]) ): one gate per token and head, and the move from the
 //                      batched product's [head, token, :] to rows of concatenated heads.  With `per_element` the gate has
 //                      one number per element of the concatenated heads: att[t, i] = T( o[..] * sigmoid(g[t, i]) ).
@@ -102,7 +103,34 @@ latent_q_assemble_kernel(T* __restrict__ q_out, const T* __restrict__ q_abs, con
 
 template <typename T>
 __global__ void __launch_bounds__(kLatentThreads)
-head_gate_kernel(T* __restrict__ out, const T* __restrict__ o, const T* __restrict__ gate, int gate_stride, int H, int vd, int T_total,
+latent_q_turn_kernel(T* __restrict__ q_out, const T* __restrict__ q, int q_stride, int H, int nope, int rank, int rot_width, int rot,
+                     const float* __restrict__ cos_t, const float* __restrict__ sin_t, int max_pos, const int* __restrict__ positions,
+                     int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t t = blockIdx.x;
+    int p = positions[t];
+    if (p < 0 || p >= max_pos) {
+        if (threadIdx.x == 0) atomicExch(err, 3);
+        p = p < 0 ? 0 : max_pos - 1;
+    }
+    const float* cs = cos_t + static_cast<int64_t>(p) * (rot / 2);
+    const float* sn = sin_t + static_cast<int64_t>(p) * (rot / 2);
+    for (int i = blockIdx.y * kLatentThreads + threadIdx.x; i < H * rot_width; i += gridDim.y * kLatentThreads) {
+        const int h = i / rot_width, e = i - h * rot_width;
+        const T* in = q + t * q_stride + h * (nope + rot_width) + nope;
+        float v = to_float(in[e]);
+        if (e < rot) {
+            const float c = cs[e >> 1], s = sn[e >> 1], other = to_float(in[e ^ 1]);
+            v = (e & 1) ? v * c + other * s : v * c - other * s;
+        }
+        q_out[(t * H + h) * (rank + rot_width) + rank + e] = from_float<T>(v);
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kLatentThreads)
+head_gate_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ o, const T* __restrict__ gate, int gate_stride, int H, int vd, int T_total,
                  int per_element) {
     pdl_trigger();
     pdl_wait();
@@ -110,7 +138,7 @@ head_gate_kernel(T* __restrict__ out, const T* __restrict__ o, const T* __restri
     for (int i = blockIdx.y * kLatentThreads + threadIdx.x; i < H * vd; i += gridDim.y * kLatentThreads) {
         const int h = i / vd, j = i - h * vd;
         const float z = to_float(gate[t * gate_stride + (per_element ? i : h)]);
-        out[t * H * vd + i] = from_float<T>(to_float(o[(static_cast<int64_t>(h) * T_total + t) * vd + j]) * (1.f / (1.f + expf(-z))));
+        out[t * out_stride + i] = from_float<T>(to_float(o[(static_cast<int64_t>(h) * T_total + t) * vd + j]) * (1.f / (1.f + expf(-z))));
     }
 }
 
@@ -150,12 +178,26 @@ extern "C" int cvb_latent_q_assemble(void* q_out, const void* q_abs, const void*
     return launch_status();
 }
 
-extern "C" int cvb_head_gate(void* out, const void* o, const void* gate, int T, int gate_stride, int H, int vd, int per_element,
+extern "C" int cvb_latent_q_turn(void* q_out, const void* q, int T, int q_stride, int H, int nope, int rank, int rot_width, int rot,
+                                 const float* cos_t, const float* sin_t, int max_pos, const int* positions, int dtype, int* err_flag,
+                                 cudaStream_t stream) {
+    if (T == 0 || rot_width == 0) return CVB_OK;
+    if (T < 0 || H <= 0 || nope <= 0 || rank <= 0 || rot_width < 0 || max_pos <= 0) return CVB_E_SIZE;
+    if (rot < 0 || rot > rot_width || rot % 2 || q_stride < H * (nope + rot_width)) return CVB_E_SHAPE;
+    const int per_row = (H * rot_width + kLatentThreads - 1) / kLatentThreads;
+#define CALL(TY) launch_kernel(latent_q_turn_kernel<TY>, dim3(T, per_row < 64 ? per_row : 64), dim3(kLatentThreads), 0, stream, (TY*)q_out, \
+                               (const TY*)q, q_stride, H, nope, rank, rot_width, rot, cos_t, sin_t, max_pos, positions, err_flag)
+    CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+    return launch_status();
+}
+
+extern "C" int cvb_head_gate(void* out, int out_stride, const void* o, const void* gate, int T, int gate_stride, int H, int vd, int per_element,
                              int dtype, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
-    if (T < 0 || H <= 0 || vd <= 0 || gate_stride < (per_element ? H * vd : H)) return CVB_E_SIZE;
+    if (T < 0 || H <= 0 || vd <= 0 || out_stride < H * vd || gate_stride < (per_element ? H * vd : H)) return CVB_E_SIZE;
     const int per_row = (H * vd + kLatentThreads - 1) / kLatentThreads;
-#define CALL(TY) launch_kernel(head_gate_kernel<TY>, dim3(T, per_row < 64 ? per_row : 64), dim3(kLatentThreads), 0, stream, (TY*)out, (const TY*)o, (const TY*)gate, \
+#define CALL(TY) launch_kernel(head_gate_kernel<TY>, dim3(T, per_row < 64 ? per_row : 64), dim3(kLatentThreads), 0, stream, (TY*)out, out_stride, (const TY*)o, (const TY*)gate, \
                                gate_stride, H, vd, T, per_element)
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL

@@ -217,7 +217,7 @@ def _resid32_lib():
     if _resid32 is None:
         lib = load_library("resid32")
         for name in ("cvb_embed_positions", "cvb_resid_update", "cvb_gelu_tanh", "cvb_write_rows", "cvb_norm_add", "cvb_bias_act",
-                     "cvb_gated_norm"):
+                     "cvb_gated_norm", "cvb_tanh_update", "cvb_stream_concat"):
             getattr(lib, name).restype = c_int
         _resid32 = lib
     return _resid32
@@ -269,6 +269,42 @@ def resid_update(h: torch.Tensor, deltas=(), rows: Optional[torch.Tensor] = None
     _check(_resid32_lib().cvb_resid_update(_ptr(h), _ptr(d1), _ptr(d2), _ptr(rows), _ptr(vector), _ptr(norm_weight), _ptr(out),
                                            c_int(T), c_int(D), c_float(eps), c_int(dtype_code(act)), _stream()), "resid_update")
     return out if out is not None else h
+
+
+def _stream_deltas(what: str, h: torch.Tensor, deltas, act: torch.dtype):
+    deltas = tuple(d for d in deltas if d is not None)
+    if len(deltas) > 2:
+        raise KernelError(f"{what}: at most two deltas")
+    for d in deltas:
+        if d.shape != h.shape or d.dtype != act:
+            raise KernelError(f"{what}: deltas must be shaped like h and share the output's element type")
+    return (deltas + (None, None))[:2]
+
+
+def tanh_update(h: torch.Tensor, deltas, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """h (float32 [T, D], in place) <- h + (deltas[0] + deltas[1]) (up to two deltas of out's element type); out <- tanh(alpha h) * weight + bias,
+    rounded once; alpha, weight [D] and bias [D] float32."""
+    d1, d2 = _stream_deltas("tanh_update", h, deltas, out.dtype)
+    _cuda(h, d1, d2, alpha, weight, bias, out); _contig(h, d1, d2, alpha, weight, bias, out)
+    T, D = h.shape
+    if (h.dtype != torch.float32 or out.shape != h.shape or any(t.dtype != torch.float32 for t in (alpha, weight, bias)) or alpha.numel() != 1
+            or weight.numel() != D or bias.numel() != D):
+        raise KernelError("tanh_update: h float32 [T, D], out [T, D]; alpha one float32, weight and bias float32 [D]")
+    _check(_resid32_lib().cvb_tanh_update(_ptr(h), _ptr(d1), _ptr(d2), _ptr(alpha), _ptr(weight), _ptr(bias), _ptr(out), c_int(T), c_int(D),
+                                          c_int(dtype_code(out.dtype)), _stream()), "tanh_update")
+    return out
+
+
+def stream_concat(out: torch.Tensor, h: torch.Tensor, deltas, rows: torch.Tensor) -> torch.Tensor:
+    """out [T, 2 D] <- [h + (deltas[0] + deltas[1]) | rows], rounded once to out's element type; h and rows float32 [T, D]."""
+    d1, d2 = _stream_deltas("stream_concat", h, deltas, out.dtype)
+    _cuda(out, h, d1, d2, rows); _contig(out, h, d1, d2, rows)
+    T, D = h.shape
+    if h.dtype != torch.float32 or rows.dtype != torch.float32 or rows.shape != h.shape or out.shape != (T, 2 * D):
+        raise KernelError("stream_concat: h and rows float32 [T, D], out [T, 2 D]")
+    _check(_resid32_lib().cvb_stream_concat(_ptr(out), _ptr(h), _ptr(d1), _ptr(d2), _ptr(rows), c_int(T), c_int(D),
+                                            c_int(dtype_code(out.dtype)), _stream()), "stream_concat")
+    return out
 
 
 def gelu_tanh(out: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
@@ -408,19 +444,19 @@ def glu_clamped(out: torch.Tensor, gate_up: torch.Tensor, limit: float, alpha: f
     T, I = out.shape
     if gate_up.shape != (T, 2 * I) or gate_up.dtype != out.dtype:
         raise KernelError("glu_clamped: gate_up must be [T, 2I] for out [T, I]")
-    _check(_sandwich_lib().cvb_glu_act(_ptr(out), _ptr(gate_up), c_int(T), c_int(I), c_int(0), c_float(limit), c_float(alpha),
-                                       c_int(dtype_code(out.dtype)), _stream()), "glu_clamped")
+    _check(_sandwich_lib().cvb_glu_act(_ptr(out), c_int(I), _ptr(gate_up), c_int(2 * I), c_int(T), c_int(I), c_int(0), c_float(limit),
+                                       c_float(alpha), c_float(1.0), c_int(dtype_code(out.dtype)), _stream()), "glu_clamped")
     return out
 
 
-def geglu(out: torch.Tensor, gate_up: torch.Tensor) -> torch.Tensor:
-    """out = gelu_tanh(gate) * up; gate_up [T, 2 I] (gate columns, then up)."""
-    _cuda(out, gate_up); _contig(out, gate_up)
+def geglu(out: torch.Tensor, gate_up: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+    """out = scale * gelu_tanh(gate) * up; gate_up [T, 2 I] (gate columns, then up).  Both may be column ranges of wider rows."""
+    _cuda(out, gate_up)
     T, I = out.shape
-    if gate_up.shape != (T, 2 * I) or gate_up.dtype != out.dtype:
+    if gate_up.shape != (T, 2 * I) or gate_up.dtype != out.dtype or out.stride(1) != 1 or gate_up.stride(1) != 1:
         raise KernelError("geglu: gate_up must be [T, 2I] for out [T, I]")
-    _check(_sandwich_lib().cvb_glu_act(_ptr(out), _ptr(gate_up), c_int(T), c_int(I), c_int(1), c_float(0.0), c_float(0.0),
-                                       c_int(dtype_code(out.dtype)), _stream()), "geglu")
+    _check(_sandwich_lib().cvb_glu_act(_ptr(out), c_int(out.stride(0)), _ptr(gate_up), c_int(gate_up.stride(0)), c_int(T), c_int(I), c_int(1),
+                                       c_float(0.0), c_float(0.0), c_float(scale), c_int(dtype_code(out.dtype)), _stream()), "geglu")
     return out
 
 
@@ -541,7 +577,7 @@ def _latent_lib():
     global _latent
     if _latent is None:
         lib = load_library("latent")
-        for name in ("cvb_latent_prep", "cvb_latent_q_assemble", "cvb_head_gate"):
+        for name in ("cvb_latent_prep", "cvb_latent_q_assemble", "cvb_latent_q_turn", "cvb_head_gate"):
             getattr(lib, name).restype = c_int
         _latent = lib
     return _latent
@@ -555,8 +591,10 @@ def latent_prep(packed: torch.Tensor, cq_out: Optional[torch.Tensor], q_off: int
     [RMSNorm(packed[kv_off : kv_off + rank]) * kv_weight | rotation of the rot_width elements behind them] (their first `rot`
     elements turn in pairs (2i, 2i+1) by cos/sin[position]).  `cq_out` or `pages` may be None."""
     _cuda(packed, cq_out, q_weight, pages, kv_weight, cos, sin, positions, slots)
-    _contig(packed, cq_out, q_weight, pages, kv_weight, cos, sin, positions, slots)
+    _contig(cq_out, q_weight, pages, kv_weight, cos, sin, positions, slots)
     T = packed.shape[0]
+    if packed.stride(1) != 1:
+        raise KernelError("latent_prep: packed rows have unit column stride")
     for t in (cq_out, pages):
         if t is not None and t.dtype != packed.dtype:
             raise KernelError("latent_prep: outputs share the packed rows' element type")
@@ -569,7 +607,7 @@ def latent_prep(packed: torch.Tensor, cq_out: Optional[torch.Tensor], q_off: int
         raise KernelError("latent_prep: a cache write needs slots and angle tables [positions, rot / 2]")
     total_slots = pages.numel() // (rank + rot_width) if pages is not None else 0
     _check(_latent_lib().cvb_latent_prep(
-        _ptr(cq_out), _ptr(pages), _ptr(packed), c_int(T), c_int(packed.shape[1]), c_int(q_off), c_int(q_rank), _ptr(q_weight),
+        _ptr(cq_out), _ptr(pages), _ptr(packed), c_int(T), c_int(packed.stride(0)), c_int(q_off), c_int(q_rank), _ptr(q_weight),
         c_int(kv_off), c_int(rank), c_int(rot_width), c_int(rot), _ptr(kv_weight), _ptr(cos), _ptr(sin),
         c_int(cos.shape[0] if cos is not None else 1), _ptr(positions), _ptr(slots), c_int64(total_slots), c_float(eps),
         c_int(dtype_code(packed.dtype)), _ptr(error_flag(packed.device)), _stream()), "latent_prep")
@@ -591,16 +629,30 @@ def latent_q_assemble(q_out: torch.Tensor, q_abs: torch.Tensor, q: torch.Tensor,
     return q_out
 
 
+def latent_q_turn(q_out: torch.Tensor, q: torch.Tensor, num_heads: int, nope: int, rank: int, rot_width: int, rot: int, cos: torch.Tensor,
+                  sin: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """q_out[t, h, rank:] = rotation of q[t, h, nope : nope + rot_width]; q_out[t, h, :rank] is left as it is."""
+    _cuda(q_out, q, cos, sin, positions); _contig(q_out, q, cos, sin, positions)
+    T = q.shape[0]
+    if (q_out.dtype != q.dtype or cos.dtype != torch.float32 or sin.dtype != torch.float32 or positions.dtype != torch.int32
+            or q_out.numel() != T * num_heads * (rank + rot_width) or (rot > 0 and cos.shape[1] != rot // 2)):
+        raise KernelError("latent_q_turn: q [T, H * (nope + rot_width)], q_out [T, H, rank + rot_width]")
+    _check(_latent_lib().cvb_latent_q_turn(
+        _ptr(q_out), _ptr(q), c_int(T), c_int(q.shape[1]), c_int(num_heads), c_int(nope), c_int(rank), c_int(rot_width), c_int(rot), _ptr(cos),
+        _ptr(sin), c_int(cos.shape[0]), _ptr(positions), c_int(dtype_code(q.dtype)), _ptr(error_flag(q.device)), _stream()), "latent_q_turn")
+    return q_out
+
+
 def head_gate(out: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, num_heads: int, vdim: int, per_element: bool = False) -> torch.Tensor:
-    """out[t, h * vdim + j] = o[h, t, j] * sigmoid(gate[t, h]); gate is a view of H columns inside rows of gate.stride(0).
+    """out[t, h * vdim + j] = o[h, t, j] * sigmoid(gate[t, h]); gate is a view of H columns inside rows of gate.stride(0), out one of H * vdim.
     `per_element`: the gate has H * vdim columns, one per element: out[t, i] = o[..] * sigmoid(gate[t, i])."""
-    _cuda(out, o, gate); _contig(out, o)
+    _cuda(out, o, gate); _contig(o)
     T = out.shape[0]
     cols = num_heads * vdim if per_element else num_heads
     if (out.dtype != o.dtype or gate.dtype != o.dtype or out.shape[1] != num_heads * vdim or o.numel() != T * num_heads * vdim
-            or gate.shape != (T, cols) or gate.stride(1) != 1):
+            or gate.shape != (T, cols) or gate.stride(1) != 1 or out.stride(1) != 1):
         raise KernelError("head_gate: o [H, T, vdim], out [T, H * vdim], gate [T, H] (or [T, H * vdim]) of one element type")
-    _check(_latent_lib().cvb_head_gate(_ptr(out), _ptr(o), _ptr(gate), c_int(T), c_int(gate.stride(0)), c_int(num_heads), c_int(vdim),
+    _check(_latent_lib().cvb_head_gate(_ptr(out), c_int(out.stride(0)), _ptr(o), _ptr(gate), c_int(T), c_int(gate.stride(0)), c_int(num_heads), c_int(vdim),
                                        c_int(1 if per_element else 0), c_int(dtype_code(o.dtype)), _stream()), "head_gate")
     return out
 
@@ -614,7 +666,7 @@ def _recurrent_lib():
     global _recurrent
     if _recurrent is None:
         lib = load_library("recurrent")
-        for name in ("cvb_lightning_prep", "cvb_lightning_scan", "cvb_delta_prep", "cvb_conv_history", "cvb_delta_scan"):
+        for name in ("cvb_lightning_prep", "cvb_lightning_scan", "cvb_delta_prep", "cvb_conv_history", "cvb_delta_scan", "cvb_skip_scan"):
             getattr(lib, name).restype = c_int
         _recurrent = lib
     return _recurrent
@@ -704,6 +756,147 @@ def delta_scan(out, qn, kn, vv, gg, bb, state: torch.Tensor, cu_seqlens, state_s
                                            _ptr(state_slots), c_int(n_slots), c_int(num_seqs), c_int(num_heads), c_int(num_kv_heads),
                                            c_int(dim), c_int(vdim), c_int(dim if decay_dim is None else int(decay_dim)),
                                            _ptr(error_flag(out.device)), _stream()), "delta_scan")
+    return out
+
+
+def skip_scan(out, q, k, v, log_decay, step, skip, state: torch.Tensor, cu_seqlens, state_slots, num_seqs: int, num_heads: int, num_groups: int,
+              dim: int, vdim: int) -> torch.Tensor:
+    """Per request and head: S <- exp(log_decay) S + step k v^T, out = S^T q + skip_h v; q and k [T, groups * dim], v [T, H * vdim] column ranges of
+    float32 rows of one stride; log_decay, step float32 [T, H]; skip float32 [H].  out float32 [T, H * vdim]."""
+    _cuda(out, q, k, v, log_decay, step, skip, state, cu_seqlens, state_slots); _contig(out, log_decay, step, skip, cu_seqlens, state_slots)
+    sp, sf, n_slots = _state_args(state)
+    T = v.shape[0]
+    if (any(t.dtype != torch.float32 for t in (out, q, k, v, log_decay, step, skip)) or out.shape != (T, num_heads * vdim) or v.shape != out.shape
+            or q.shape != (T, num_groups * dim) or k.shape != q.shape or any(t.stride() != v.stride() or t.stride(1) != 1 for t in (q, k, v))
+            or log_decay.shape != (T, num_heads) or step.shape != log_decay.shape or skip.numel() != num_heads):
+        raise KernelError("skip_scan: float32 rows q, k [T, groups * dim], v [T, H * vdim] of one stride; log_decay, step [T, H]; skip [H]")
+    _check(_recurrent_lib().cvb_skip_scan(_ptr(out), _ptr(q), _ptr(k), _ptr(v), c_int64(v.stride(0)), _ptr(log_decay), _ptr(step), _ptr(skip), sp, sf,
+                                          _ptr(cu_seqlens), _ptr(state_slots), c_int(n_slots), c_int(num_seqs), c_int(num_heads), c_int(num_groups),
+                                          c_int(dim), c_int(vdim), _ptr(error_flag(out.device)), _stream()), "skip_scan")
+    return out
+
+
+# ---- state-space recurrence (csrc/ssd.cu) -----------------------------------------------------------------------------------------
+
+_ssd = None
+SSD_CHUNK = 64              # tokens per chunk of the tensor-core form
+
+
+def _ssd_lib():
+    global _ssd
+    if _ssd is None:
+        lib = load_library("ssd")
+        for name in ("cvb_ssd_prep", "cvb_ssd_ring", "cvb_ssd_chunks", "cvb_ssd_step", "cvb_ssd_norm"):
+            getattr(lib, name).restype = c_int
+        _ssd = lib
+    return _ssd
+
+
+def _ssd_check(what, packed, conv_w, conv_b, dt_bias, neg_a, num_heads, groups, dim, vdim, ints):
+    C = num_heads * vdim + 2 * groups * dim
+    if (packed.stride(1) != 1 or conv_w.dim() != 2 or conv_w.shape[1] != C or conv_b.numel() != C or dt_bias.numel() != num_heads
+            or neg_a.numel() != num_heads or any(t.dtype != torch.float32 for t in (conv_w, conv_b, dt_bias, neg_a))):
+        raise KernelError(f"{what}: conv_w float32 [taps, channels], conv_b [channels], dt_bias and neg_a [H]; packed rows of unit column stride")
+    if any(t.dtype != torch.int32 for t in ints):
+        raise KernelError(f"{what}: index tensors are int32")
+    return C
+
+
+def ssd_prep(u: torch.Tensor, dt: torch.Tensor, log_decay: torch.Tensor, packed: torch.Tensor, u_off: int, dt_off: int, conv_w, conv_b, dt_bias, neg_a,
+             state: torch.Tensor, seq_of_token, cu_seqlens, state_slots, positions, num_heads: int, groups: int, dim: int, vdim: int) -> None:
+    """Per token: u [T, H vdim + 2 G dim] = silu(causal convolution of packed[:, u_off:] + conv_b) (float32 or packed's element type), dt =
+    softplus(packed[:, dt_off + h] + dt_bias), log_decay = neg_a dt (float32 [T, H]).  conv_w is [taps, channels], the last row on the current
+    token; what lies before the portion comes from the ring behind S in the request's state row (csrc/ssd.cu)."""
+    _cuda(u, dt, log_decay, packed, conv_w, conv_b, dt_bias, neg_a, state, seq_of_token, cu_seqlens, state_slots, positions)
+    _contig(u, dt, log_decay, conv_w, conv_b, dt_bias, neg_a, seq_of_token, cu_seqlens, state_slots, positions)
+    C = _ssd_check("ssd_prep", packed, conv_w, conv_b, dt_bias, neg_a, num_heads, groups, dim, vdim, (seq_of_token, cu_seqlens, state_slots, positions))
+    sp, sf, n_slots = _state_args(state)
+    T = packed.shape[0]
+    if u.shape != (T, C) or dt.shape != (T, num_heads) or log_decay.shape != dt.shape or dt.dtype != torch.float32 or log_decay.dtype != torch.float32:
+        raise KernelError("ssd_prep: u [T, channels]; dt and log_decay float32 [T, H]")
+    _check(_ssd_lib().cvb_ssd_prep(
+        _ptr(u), _ptr(dt), _ptr(log_decay), _ptr(packed), c_int(T), c_int(packed.stride(0)), c_int(u_off), c_int(dt_off), _ptr(conv_w), _ptr(conv_b),
+        c_int(conv_w.shape[0]), _ptr(dt_bias), _ptr(neg_a), sp, sf, _ptr(seq_of_token), _ptr(cu_seqlens), _ptr(state_slots), _ptr(positions),
+        c_int(n_slots), c_int(num_heads), c_int(groups), c_int(dim), c_int(vdim), c_int(dtype_code(packed.dtype)), c_int(dtype_code(u.dtype)),
+        _ptr(error_flag(u.device)), _stream()), "ssd_prep")
+
+
+def ssd_ring(state: torch.Tensor, packed: torch.Tensor, u_off: int, dt_off: int, taps: int, cu_seqlens, state_slots, positions, num_seqs: int,
+             num_heads: int, groups: int, dim: int, vdim: int) -> None:
+    """The last taps - 1 raw inputs of every request's portion into the ring of its state row."""
+    _cuda(state, packed, cu_seqlens, state_slots, positions); _contig(cu_seqlens, state_slots, positions)
+    sp, sf, n_slots = _state_args(state)
+    _check(_ssd_lib().cvb_ssd_ring(sp, sf, _ptr(packed), c_int(packed.stride(0)), c_int(u_off), c_int(dt_off), c_int(taps), _ptr(cu_seqlens),
+                                   _ptr(state_slots), _ptr(positions), c_int(n_slots), c_int(num_seqs), c_int(num_heads), c_int(groups), c_int(dim),
+                                   c_int(vdim), c_int(dtype_code(packed.dtype)), _ptr(error_flag(packed.device)), _stream()), "ssd_ring",
+           kernels=1 if taps > 1 else 0)
+
+
+def ssd_chunks_supported(dtype: torch.dtype, dim: int, vdim: int) -> bool:
+    """Whether the tensor-core form takes the sizes: bf16, state and value sizes in steps of 16, state sizes up to 256."""
+    return dtype == torch.bfloat16 and dim % 16 == 0 and dim <= 256 and vdim % 16 == 0
+
+
+def ssd_held_chunks(max_tokens: int) -> int:
+    """The most chunks that requests with more than one chunk can have in a step of up to `max_tokens` tokens: a request of n tokens has
+    fewer than 2 n / 64."""
+    return 2 * max_tokens // SSD_CHUNK + 2
+
+
+def ssd_chunks(y: torch.Tensor, u: torch.Tensor, dt: torch.Tensor, log_decay: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, cu_seqlens,
+               state_slots, q_lens, num_heads: int, groups: int, dim: int, vdim: int, ends: Optional[torch.Tensor] = None,
+               decays: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per request and head: S <- exp(log_decay) S + dt B x^T, y = S^T C + skip_h x over the request's tokens of this step, in chunks of 64 tokens on
+    the tensor cores; u bf16 [T, H vdim + 2 G dim] rows [x | B | C]; y float32 [T, H * vdim].  Portions of more than 64 tokens go through `ends`
+    (float32, H dim vdim per chunk of such a portion) and `decays` (float32, H per chunk)."""
+    _cuda(y, u, dt, log_decay, skip, state, cu_seqlens, state_slots, ends, decays); _contig(y, u, dt, log_decay, skip, cu_seqlens, state_slots, ends, decays)
+    sp, sf, n_slots = _state_args(state)
+    T = u.shape[0]
+    if (u.dtype != torch.bfloat16 or u.shape[1] != num_heads * vdim + 2 * groups * dim or y.shape != (T, num_heads * vdim) or dt.shape != (T, num_heads)
+            or log_decay.shape != dt.shape or skip.numel() != num_heads or cu_seqlens.dtype != torch.int32 or state_slots.dtype != torch.int32
+            or any(t is not None and t.dtype != torch.float32 for t in (y, dt, log_decay, skip, ends, decays))):
+        raise KernelError("ssd_chunks: u bf16 [T, channels]; y float32 [T, H * vdim]; dt, log_decay float32 [T, H]; skip float32 [H]")
+    per = [-(-n // SSD_CHUNK) for n in q_lens]
+    held = sum(c for c in per if c > 1)
+    _check(_ssd_lib().cvb_ssd_chunks(
+        _ptr(y), _ptr(u), _ptr(dt), _ptr(log_decay), _ptr(skip), _ptr(ends), c_int64(ends.numel() if ends is not None else 0), _ptr(decays),
+        c_int64(decays.numel() if decays is not None else 0), sp, sf, c_int(n_slots), _ptr(cu_seqlens), _ptr(state_slots), c_int(len(per)),
+        c_int(sum(per)), c_int(held), c_int(num_heads), c_int(groups), c_int(dim), c_int(vdim), _ptr(error_flag(u.device)), _stream()),
+        "ssd_chunks", kernels=3 if held else 1)
+    return y
+
+
+def ssd_step_supported(dim: int, vdim: int) -> bool:
+    """Whether the one-kernel form of a step of decoded tokens holds a head's vectors in shared memory."""
+    return (vdim + 2 * dim + max(1024, vdim)) * 4 <= 48 * 1024
+
+
+def ssd_step(y: torch.Tensor, packed: torch.Tensor, u_off: int, dt_off: int, conv_w, conv_b, dt_bias, neg_a, skip, state: torch.Tensor, cu_seqlens,
+             state_slots, positions, num_seqs: int, num_heads: int, groups: int, dim: int, vdim: int) -> torch.Tensor:
+    """A step of one token per request: convolutions, ring, dt, decay, S <- exp(log_decay) S + dt B x^T, y = S^T C + skip_h x (float32)."""
+    _cuda(y, packed, conv_w, conv_b, dt_bias, neg_a, skip, state, cu_seqlens, state_slots, positions)
+    _contig(y, conv_w, conv_b, dt_bias, neg_a, skip, cu_seqlens, state_slots, positions)
+    _ssd_check("ssd_step", packed, conv_w, conv_b, dt_bias, neg_a, num_heads, groups, dim, vdim, (cu_seqlens, state_slots, positions))
+    sp, sf, n_slots = _state_args(state)
+    if y.dtype != torch.float32 or y.shape != (packed.shape[0], num_heads * vdim) or skip.dtype != torch.float32 or skip.numel() != num_heads:
+        raise KernelError("ssd_step: y float32 [S, H * vdim]; skip float32 [H]")
+    _check(_ssd_lib().cvb_ssd_step(
+        _ptr(y), _ptr(packed), c_int(packed.stride(0)), c_int(u_off), c_int(dt_off), _ptr(conv_w), _ptr(conv_b), c_int(conv_w.shape[0]), _ptr(dt_bias),
+        _ptr(neg_a), _ptr(skip), sp, sf, _ptr(cu_seqlens), _ptr(state_slots), _ptr(positions), c_int(n_slots), c_int(num_seqs), c_int(num_heads),
+        c_int(groups), c_int(dim), c_int(vdim), c_int(dtype_code(packed.dtype)), _ptr(error_flag(y.device)), _stream()), "ssd_step")
+    return y
+
+
+def gate_norm(out: torch.Tensor, y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, scale: float = 1.0) -> torch.Tensor:
+    """out = scale * RMSNorm(y * silu(gate)) * weight over `parts` equal parts of the row, each by its own root mean square; y float32 [T, n], weight
+    float32 [n]; out and gate [T, n] of one element type, column ranges of wider rows."""
+    _cuda(out, y, gate, weight); _contig(y, weight)
+    T, n = y.shape
+    if (y.dtype != torch.float32 or weight.dtype != torch.float32 or weight.numel() != n or n % parts or out.shape != y.shape or gate.shape != y.shape
+            or gate.dtype != out.dtype or out.stride(1) != 1 or gate.stride(1) != 1):
+        raise KernelError("gate_norm: y float32 [T, n], weight float32 [n]; out and gate [T, n] of the activations' type")
+    _check(_ssd_lib().cvb_ssd_norm(_ptr(out), c_int(out.stride(0)), _ptr(y), _ptr(gate), c_int(gate.stride(0)), _ptr(weight), c_int(T), c_int(parts),
+                                   c_int(n // parts), c_float(eps), c_float(scale), c_int(dtype_code(out.dtype)), _stream()), "gate_norm")
     return out
 
 
@@ -970,7 +1163,8 @@ def attn_keys_tiles(q_lens, num_heads: int, num_kv_heads: int) -> int:
 def attn_keys_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, block_tables: torch.Tensor, cu_seqlens: torch.Tensor,
                    positions: torch.Tensor, num_seqs: int, num_tiles: int, num_heads: int, num_kv_heads: int, head_dim: int,
                    page_size: int, scale: float, window: int = 0, keep_first: int = 0, all_single: bool = False, splits: int = 1,
-                   scratch: Optional[torch.Tensor] = None, value_dim: Optional[int] = None, kv_heads_in_pages: int = 0) -> torch.Tensor:
+                   scratch: Optional[torch.Tensor] = None, value_dim: Optional[int] = None, kv_heads_in_pages: int = 0,
+                   sink: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
     """Attention of prompt portions and decoded tokens over pages [kv head, slot, head_dim] whose keys are also the
     values; `q` may be the packed output of a projection (rows of q.shape[1] elements, queries first).  `all_single`:
     every request brings exactly one token (a decode step): a block per (request, kv head) whose warps share out the key
@@ -978,8 +1172,11 @@ def attn_keys_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, bloc
     attn_keys_scratch_floats elements) and a merge kernel.  `value_dim` (a multiple of 16): only the first value_dim elements
     of a key are its value; out is [T, H * value_dim].  `kv_heads_in_pages` (a divisor of num_kv_heads): the pages hold fewer
     kv heads than the grid walks, the query heads of one stored head being dealt with as several groups (a decode step of more
-    than 16 query heads per stored head)."""
-    _cuda(out, q, pages, block_tables, cu_seqlens, positions); _contig(out, q, pages, block_tables, cu_seqlens, positions)
+    than 16 query heads per stored head).  `sink` (float32 [H]): exp(sink_h) joins the softmax's denominator; `out_scale` multiplies the
+    output."""
+    _cuda(out, q, pages, block_tables, cu_seqlens, positions, sink); _contig(out, q, pages, block_tables, cu_seqlens, positions, sink)
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != num_heads):
+        raise KernelError("attn_keys_bf16: sink is float32 [H]")
     if q.dtype != torch.bfloat16 or pages.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("attn_keys_bf16 takes bf16 queries, pages and output")
     if block_tables.dtype != torch.int32 or block_tables.dim() != 2 or cu_seqlens.dtype != torch.int32 or positions.dtype != torch.int32:
@@ -993,7 +1190,7 @@ def attn_keys_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, bloc
         c_int(head_dim if value_dim is None else value_dim), c_int(page_size), c_int(window), c_int(keep_first), c_float(scale),
         c_int(num_pages), c_int(1 if all_single else 0),
         c_int(splits), _ptr(scratch), c_int64(scratch.numel() if scratch is not None else 0), c_int(kv_heads_in_pages),
-        _ptr(error_flag(q.device)), _stream()), "attn_keys_bf16", kernels=2 if all_single and splits > 1 else 1)
+        _ptr(sink), c_float(out_scale), _ptr(error_flag(q.device)), _stream()), "attn_keys_bf16", kernels=2 if all_single and splits > 1 else 1)
     return out
 
 
@@ -1323,7 +1520,7 @@ def pool_entries(pages: torch.Tensor, block_tables: torch.Tensor, seq_of_token: 
 def attn_masked_general(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, block_tables: torch.Tensor,
                         seq_of_token: torch.Tensor, positions: torch.Tensor, num_tokens: int, num_heads: int, num_kv_heads: int,
                         dim: int, vdim: int, page_size: int, scale: float, planes: int = 1, chunk: int = 0, window: int = 0,
-                        pool: int = 0, softcap: float = 0.0, r1: Optional[torch.Tensor] = None, r2: Optional[torch.Tensor] = None,
+                        pool: int = 0, keep_first: int = 0, softcap: float = 0.0, r1: Optional[torch.Tensor] = None, r2: Optional[torch.Tensor] = None,
                         sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
     """out [T, H * vdim] (a column range of wider rows will do): one block per (token, query head), any sizes, float32 or bf16 (see csrc/attention_masked.cu).
     `gate` [T, H] (a view with unit column stride): the head's output is multiplied by sigmoid(gate[t, h]); a gate of H * vdim columns
@@ -1346,7 +1543,7 @@ def attn_masked_general(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor,
     _check(_attn_masked_lib().cvb_attn_masked_general(
         _ptr(out), _ptr(q), _ptr(pages), _ptr(block_tables), c_int(block_tables.shape[1]), _ptr(seq_of_token), _ptr(positions),
         c_int(T), c_int(H), c_int(G), c_int(dim), c_int(vdim), c_int(page_size), c_int(planes), c_int(chunk), c_int(window),
-        c_int(pool), c_float(scale), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate),
+        c_int(pool), c_int(keep_first), c_float(scale), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate),
         c_int(gate.stride(0) if gate is not None else 0), c_int(1 if per_element else 0), c_float(out_scale), c_int(out.stride(0)),
         c_int(num_pages), c_int(dtype_code(q.dtype)), _ptr(error_flag(q.device)), _stream()), "attn_masked_general")
     return out
@@ -1380,7 +1577,7 @@ def attn_masked_decode_splits(num_seqs: int, num_kv_heads: int, visible_keys: in
 
 def attn_masked_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, block_tables: torch.Tensor, cu_seqlens: torch.Tensor,
                      positions: torch.Tensor, num_seqs: int, num_tiles: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int,
-                     page_size: int, scale: float, planes: int = 1, chunk: int = 0, window: int = 0, pool: int = 0,
+                     page_size: int, scale: float, planes: int = 1, chunk: int = 0, window: int = 0, pool: int = 0, keep_first: int = 0,
                      softcap: float = 0.0, r1: Optional[torch.Tensor] = None, r2: Optional[torch.Tensor] = None,
                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, all_single: bool = False,
                      splits: int = 1, scratch: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
@@ -1409,7 +1606,7 @@ def attn_masked_bf16(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, bl
     _check(_attn_masked_lib().cvb_attn_masked_bf16(
         _ptr(out), _ptr(q), _ptr(pages), _ptr(block_tables), c_int(block_tables.shape[1]), _ptr(cu_seqlens), _ptr(positions),
         c_int(num_seqs), c_int(num_tiles), c_int(H), c_int(num_kv_heads), c_int(dim), c_int(vdim), c_int(page_size), c_int(planes),
-        c_int(chunk), c_int(window), c_int(pool), c_float(scale), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate),
+        c_int(chunk), c_int(window), c_int(pool), c_int(keep_first), c_float(scale), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate),
         c_int(gate.stride(0) if gate is not None else 0), c_int(1 if per_element else 0), c_float(out_scale), c_int(out.stride(0)),
         c_int(num_pages), c_int(1 if all_single else 0), c_int(splits), _ptr(scratch),
         c_int64(scratch.numel() if scratch is not None else 0), _ptr(error_flag(q.device)), _stream()), "attn_masked_bf16",
@@ -1463,14 +1660,16 @@ def paged_attention_general(out: torch.Tensor, q: torch.Tensor, cache: torch.Ten
                             seq_of_token: torch.Tensor, positions: torch.Tensor, num_heads: int, num_kv_heads: int,
                             head_dim: int, page_size: int, scale: float, window: int = 0,
                             num_tokens: Optional[int] = None, keep_first: int = 0, keys_are_values: bool = False,
-                            value_dim: Optional[int] = None) -> torch.Tensor:
+                            value_dim: Optional[int] = None, sink: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
     """One block per (token, query head); any head size.  `keep_first`: positions 0..keep_first-1 stay visible behind the
     window.  `keys_are_values`: pages are [kv head, slot, head_dim] and a key is also its value (else [K|V, kv head, slot,
     head_dim]).  `q` may be the packed output of a projection: rows of q.shape[1] elements whose first H * head_dim are
     the queries.  `value_dim` (with keys_are_values): only the first value_dim elements of a key are its value; out is
-    [T, H, value_dim]."""
-    _cuda(out, q, cache, block_tables, seq_of_token, positions)
-    _contig(out, q, cache, block_tables, seq_of_token, positions)
+    [T, H, value_dim].  `sink` (float32 [H]): exp(sink_h) joins the softmax's denominator; `out_scale` multiplies the output."""
+    _cuda(out, q, cache, block_tables, seq_of_token, positions, sink)
+    _contig(out, q, cache, block_tables, seq_of_token, positions, sink)
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != num_heads):
+        raise KernelError("paged_attention: sink is float32 [H]")
     T = q.shape[0] if num_tokens is None else num_tokens
     if q.dtype != cache.dtype or out.dtype != q.dtype:
         raise KernelError("paged_attention: q, out and the cache pages must share one element type")
@@ -1493,7 +1692,7 @@ def paged_attention_general(out: torch.Tensor, q: torch.Tensor, cache: torch.Ten
         _ptr(out), _ptr(q), _ptr(cache), _ptr(block_tables), c_int(block_tables.shape[1]), _ptr(seq_of_token),
         _ptr(positions), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(vd), c_int(page_size),
         c_int(window), c_int(keep_first), c_int(planes), c_int(q_stride), c_float(scale), c_int(num_pages),
-        c_int(dtype_code(q.dtype)),
+        _ptr(sink), c_float(out_scale), c_int(dtype_code(q.dtype)),
         _ptr(error_flag(q.device)), _stream()), "paged_attention_general")
     return out
 

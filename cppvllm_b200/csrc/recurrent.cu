@@ -9,6 +9,8 @@
 //   conv_history   : the last taps - 1 raw inputs of every request's portion become the history of its next one
 //   delta_scan     : S <- diag(g) S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q      (query/key head h / (H / G))
 //                    The decay is one number per head and key channel, or (`gd` = 1) one number per head: S <- g S.
+//   skip_scan      : S <- e^a S + b k v^T;  o = S^T q + d_h v       a and b one number per token and head (query/key head h / (H / G)),
+//                    d one per head; q, k, v column ranges of float rows (the state-space rule of ssd.cu in float, any sizes)
 //
 // S is [dk, dv] per (request, head), float, in the request's state slot; portions of any length continue where the
 // state stands, one token after the other in the same order of operations, so cutting a sequence changes no bit.
@@ -53,18 +55,21 @@ __global__ void lightning_prep_kernel(float* __restrict__ qf, float* __restrict_
 // (rows r * kScanLanes + lane part) and add their parts up by shuffles.  The tokens' q, k (and g), v (and b) travel through
 // two stages of shared memory by cp.async, kScanChunk tokens a stage, so that the next tokens arrive while these are used.
 // MODE 1: S <- diag(g) S; u = b (v - S^T k); S <- S + k u^T; o = S^T q.  MODE 2: the same with one decay per head and token
-// (S <- g S).  MODE 0: S <- d S + k v^T; o = S^T q.
+// (S <- g S).  MODE 0: S <- d S + k v^T; o = S^T q.  MODE 3: S <- e^g S + b k v^T; o = S^T q + d v, g and b per head and token.
+// Rows of q, k (of v) are `qk_stride` (`v_stride`) floats apart.
 template <int KPT, int MODE>
 __global__ void __launch_bounds__(kScanThreads)
 recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vv,
                       const float* __restrict__ gg, const float* __restrict__ bb, const float* __restrict__ decay,
                       float* __restrict__ state, int64_t state_floats, const int* __restrict__ cu_seqlens,
-                      const int* __restrict__ state_slots, int num_slots, int H, int G, int dk, int dv, int* __restrict__ err) {
+                      const int* __restrict__ state_slots, int num_slots, int H, int G, int dk, int dv, int64_t qk_stride, int64_t v_stride,
+                      int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
     constexpr int dkp = KPT * kScanLanes;
-    constexpr bool DELTA = MODE != 0;
+    constexpr bool DELTA = MODE == 1 || MODE == 2;
+    constexpr bool PER_HEAD = MODE == 2 || MODE == 3;                       // one decay per head and token
     constexpr int kArrays = MODE == 1 ? 3 : 2;
     constexpr int kStage = kArrays * kScanChunk * dkp + kScanChunk * kScanCols + 2 * kScanChunk;
     const int s = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * kScanCols;
@@ -86,7 +91,7 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
         S[r] = (i < dk && j < dv) ? st[static_cast<int64_t>(i) * dv + j] : 0.f;
     }
     const float d = DELTA ? 1.f : decay[h];
-    const bool vec = (dk & 3) == 0 && (dv & 3) == 0;
+    const bool vec = (dk & 3) == 0 && (dv & 3) == 0 && (qk_stride & 3) == 0 && (v_stride & 3) == 0;
 
     auto load = [&](int t0, int stage) {
         const int n = min(kScanChunk, end - t0);
@@ -95,35 +100,35 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
         float* gs = ks + kScanChunk * dkp;                                  // MODE 1 only
         float* vs = qs + kArrays * kScanChunk * dkp;
         float* bs = vs + kScanChunk * kScanCols;
-        float* g1 = bs + kScanChunk;                                        // MODE 2 only: one decay per token
+        float* g1 = bs + kScanChunk;                                        // MODE 2 and 3: one decay per token
         if (vec) {
             const int dk4 = dk >> 2;
             for (int idx = tid; idx < n * dk4; idx += kScanThreads) {
                 const int tt = idx / dk4, i = (idx - tt * dk4) * 4;
                 const int64_t tok = t0 + tt;
-                cp_async16(qs + tt * dkp + i, qn + (tok * G + kvh) * dk + i, true);
-                cp_async16(ks + tt * dkp + i, kn + (tok * G + kvh) * dk + i, true);
+                cp_async16(qs + tt * dkp + i, qn + tok * qk_stride + kvh * dk + i, true);
+                cp_async16(ks + tt * dkp + i, kn + tok * qk_stride + kvh * dk + i, true);
                 if (MODE == 1) cp_async16(gs + tt * dkp + i, gg + (tok * H + h) * dk + i, true);
             }
             for (int idx = tid; idx < n * (kScanCols / 4); idx += kScanThreads) {
                 const int tt = idx / (kScanCols / 4), c = (idx - tt * (kScanCols / 4)) * 4;
-                if (j0 + c < dv) cp_async16(vs + tt * kScanCols + c, vv + (static_cast<int64_t>(t0 + tt) * H + h) * dv + j0 + c, true);
+                if (j0 + c < dv) cp_async16(vs + tt * kScanCols + c, vv + static_cast<int64_t>(t0 + tt) * v_stride + h * dv + j0 + c, true);
             }
         } else {
             for (int idx = tid; idx < n * dk; idx += kScanThreads) {
                 const int tt = idx / dk, i = idx - tt * dk;
                 const int64_t tok = t0 + tt;
-                cp_async4(qs + tt * dkp + i, qn + (tok * G + kvh) * dk + i);
-                cp_async4(ks + tt * dkp + i, kn + (tok * G + kvh) * dk + i);
+                cp_async4(qs + tt * dkp + i, qn + tok * qk_stride + kvh * dk + i);
+                cp_async4(ks + tt * dkp + i, kn + tok * qk_stride + kvh * dk + i);
                 if (MODE == 1) cp_async4(gs + tt * dkp + i, gg + (tok * H + h) * dk + i);
             }
             for (int idx = tid; idx < n * kScanCols; idx += kScanThreads) {
                 const int tt = idx / kScanCols, c = idx - tt * kScanCols;
-                if (j0 + c < dv) cp_async4(vs + tt * kScanCols + c, vv + (static_cast<int64_t>(t0 + tt) * H + h) * dv + j0 + c);
+                if (j0 + c < dv) cp_async4(vs + tt * kScanCols + c, vv + static_cast<int64_t>(t0 + tt) * v_stride + h * dv + j0 + c);
             }
         }
-        if (DELTA && tid < n) cp_async4(bs + tid, bb + static_cast<int64_t>(t0 + tid) * H + h);
-        if (MODE == 2 && tid < n) cp_async4(g1 + tid, gg + static_cast<int64_t>(t0 + tid) * H + h);
+        if ((DELTA || MODE == 3) && tid < n) cp_async4(bs + tid, bb + static_cast<int64_t>(t0 + tid) * H + h);
+        if (PER_HEAD && tid < n) cp_async4(g1 + tid, gg + static_cast<int64_t>(t0 + tid) * H + h);
     };
 
     if (begin < end) load(begin, 0);
@@ -165,16 +170,17 @@ recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qn, con
                     if (r & 1) o1 = fmaf(S[r], qq[r * kScanLanes], o1); else o0 = fmaf(S[r], qq[r * kScanLanes], o0);
                 }
             } else {
+                const float gh = MODE == 3 ? expf(g1[tt]) : d, vb = MODE == 3 ? bs[tt] * v : v;
 #pragma unroll
                 for (int r = 0; r < KPT; ++r) {
-                    S[r] = fmaf(d, S[r], kq[r * kScanLanes] * v);
+                    S[r] = fmaf(gh, S[r], kq[r * kScanLanes] * vb);
                     if (r & 1) o1 = fmaf(S[r], qq[r * kScanLanes], o1); else o0 = fmaf(S[r], qq[r * kScanLanes], o0);
                 }
             }
             float o = o0 + o1;
 #pragma unroll
             for (int m = 1; m < kScanLanes; m <<= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
-            if (part == 0 && j < dv) out[(static_cast<int64_t>(t0 + tt) * H + h) * dv + j] = o;
+            if (part == 0 && j < dv) out[(static_cast<int64_t>(t0 + tt) * H + h) * dv + j] = MODE == 3 ? fmaf(d, v, o) : o;
         };
         if (n == kScanChunk) {                                               // unrolled: the tokens' shuffles and loads overlap
 #pragma unroll
@@ -289,7 +295,7 @@ using namespace cvb;
 template <int KPT, int MODE>
 static int launch_scan(float* out, const float* qn, const float* kn, const float* vv, const float* gg, const float* bb, const float* decay,
                        float* state, int64_t state_floats, const int* cu_seqlens, const int* state_slots, int num_slots, int S, int H, int G,
-                       int dk, int dv, int* err_flag, cudaStream_t stream) {
+                       int dk, int dv, int64_t qk_stride, int64_t v_stride, int* err_flag, cudaStream_t stream) {
     constexpr int arrays = MODE == 1 ? 3 : 2;
     const size_t smem = static_cast<size_t>(2) * (arrays * kScanChunk * KPT * kScanLanes + kScanChunk * kScanCols + 2 * kScanChunk) * sizeof(float);
     static bool raised = false;
@@ -300,7 +306,7 @@ static int launch_scan(float* out, const float* qn, const float* kn, const float
     }
     const dim3 grid(S, H, (dv + kScanCols - 1) / kScanCols);
     launch_kernel(recurrent_scan_kernel<KPT, MODE>, grid, dim3(kScanThreads), smem, stream, out, qn, kn, vv, gg, bb, decay, state,
-                  state_floats, cu_seqlens, state_slots, num_slots, H, G, dk, dv, err_flag);
+                  state_floats, cu_seqlens, state_slots, num_slots, H, G, dk, dv, qk_stride, v_stride, err_flag);
     return launch_status();
 }
 
@@ -329,7 +335,7 @@ extern "C" int cvb_lightning_scan(float* out, const float* qf, const float* kf, 
     if (state_floats < static_cast<int64_t>(H) * dk * dv) return CVB_E_SHAPE;
     if (!aligned16(qf) || !aligned16(kf) || !aligned16(vf)) return CVB_E_ALIGN;
 #define CALL_K(KPT) return launch_scan<KPT, 0>(out, qf, kf, vf, nullptr, nullptr, decay, state, state_floats, cu_seqlens, state_slots, \
-                                                   num_slots, S, H, H, dk, dv, err_flag, stream)
+                                                   num_slots, S, H, H, dk, dv, static_cast<int64_t>(H) * dk, static_cast<int64_t>(H) * dv, err_flag, stream)
     CVB_DISPATCH_KPT(dk, CALL_K);
 #undef CALL_K
 }
@@ -377,12 +383,28 @@ extern "C" int cvb_delta_scan(float* out, const float* qn, const float* kn, cons
     if (!aligned16(qn) || !aligned16(kn) || !aligned16(vv) || !aligned16(gg)) return CVB_E_ALIGN;
     if (gd == 1 && dk != 1) {
 #define CALL_K(KPT) return launch_scan<KPT, 2>(out, qn, kn, vv, gg, bb, nullptr, state, state_floats, cu_seqlens, state_slots, num_slots, \
-                                               S, H, G, dk, dv, err_flag, stream)
+                                               S, H, G, dk, dv, static_cast<int64_t>(G) * dk, static_cast<int64_t>(H) * dv, err_flag, stream)
         CVB_DISPATCH_KPT(dk, CALL_K);
 #undef CALL_K
     }
 #define CALL_K(KPT) return launch_scan<KPT, 1>(out, qn, kn, vv, gg, bb, nullptr, state, state_floats, cu_seqlens, state_slots, num_slots, \
-                                               S, H, G, dk, dv, err_flag, stream)
+                                               S, H, G, dk, dv, static_cast<int64_t>(G) * dk, static_cast<int64_t>(H) * dv, err_flag, stream)
+    CVB_DISPATCH_KPT(dk, CALL_K);
+#undef CALL_K
+}
+
+// Rows of q, k and v are `stride` floats apart; a and b [T, H].
+extern "C" int cvb_skip_scan(float* out, const float* q, const float* k, const float* v, int64_t stride, const float* a, const float* b, const float* d,
+                             float* state, int64_t state_floats, const int* cu_seqlens, const int* state_slots, int num_slots, int S, int H,
+                             int G, int dk, int dv, int* err_flag, cudaStream_t stream) {
+    if (S == 0) return CVB_OK;
+    if (S < 0 || H <= 0 || H > 65535 || G <= 0 || dk <= 0 || dk > 512 || dv <= 0 || num_slots <= 0) return CVB_E_SIZE;
+    if (H % G || state_floats < static_cast<int64_t>(H) * dk * dv || stride < static_cast<int64_t>(G) * dk || stride < static_cast<int64_t>(H) * dv) return CVB_E_SHAPE;
+    // whole 16-byte pieces only where every row starts on one: the kernel decides by the sizes, so the bases have to agree
+    if ((dk & 3) == 0 && (dv & 3) == 0 && (stride & 3) == 0 && !(aligned16(q) && aligned16(k) && aligned16(v))) return CVB_E_ALIGN;
+#define CALL_K(KPT) return launch_scan<KPT, 3>(out, q, k, v, a, b, d, state, state_floats, cu_seqlens, state_slots, num_slots, S, H, G, dk, dv, \
+                                               stride, stride, err_flag, stream)
+    if (dk > 256) { CALL_K(64); }
     CVB_DISPATCH_KPT(dk, CALL_K);
 #undef CALL_K
 }

@@ -6,6 +6,8 @@
 //                     with a norm weight w also  out[t, :] = T( h * (1 / sqrt(mean(h^2) + eps)) * w ): RMSNorm with one
 //                     rounding, at the store.  One kernel serves the plain norm, the residual add fused with the next
 //                     norm, and the input of a repeated pass (the embedding output and a per-pass vector added).
+//   tanh_update     : h as above (deltas only), and  out[t, :] = T( tanh(alpha h) * w + b ): a norm without statistics
+//   stream_concat   : out[t, :] = [T(h + (d1 + d2)) | T(e)]: what a product over the stream and a second 32-bit row reads
 //   gelu_tanh       : out = T( 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) ), z = float(x)
 //   write_rows      : rows of a packed projection into cache pages [page, heads, slot in page, width] (a cache that
 //                     holds one vector per token and head: keys that also serve as values)
@@ -139,6 +141,106 @@ resid_update_vec_kernel(float* h, const T* __restrict__ d1, const T* __restrict_
             o[3] = from_float<T>(val[k].w * inv * ww.w);
         }
     }
+}
+
+// h <- h + (d1 + d2);  out = tanh(alpha h) w + b: element by element
+template <typename T>
+__global__ void __launch_bounds__(256)
+tanh_update_kernel(float* h, const T* __restrict__ d1, const T* __restrict__ d2, const float* __restrict__ alpha, const float* __restrict__ w,
+                   const float* __restrict__ b, T* __restrict__ out, int D, int64_t n) {
+    pdl_trigger();
+    pdl_wait();
+    const float a = alpha[0];
+    for (int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x; i < n; i += static_cast<int64_t>(gridDim.x) * 256) {
+        float v = h[i];
+        if (d1) {
+            float d = to_float(d1[i]);
+            if (d2) d += to_float(d2[i]);
+            v += d;
+            h[i] = v;
+        }
+        const int c = static_cast<int>(i % D);
+        out[i] = from_float<T>(fmaf(tanhf(a * v), w[c], b[c]));
+    }
+}
+
+// The same, eight elements a thread
+template <typename T>
+__global__ void __launch_bounds__(256)
+tanh_update_vec_kernel(float* h, const T* __restrict__ d1, const T* __restrict__ d2, const float* __restrict__ alpha, const float* __restrict__ w,
+                       const float* __restrict__ b, T* __restrict__ out, int D, int64_t n) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) * 8;
+    if (i >= n) return;
+    const int c = static_cast<int>(i % D);
+    float v[8], ww[8], bb[8];
+    load8(v, h + i);
+    load8(ww, w + c);
+    load8(bb, b + c);
+    const float a = alpha[0];
+    if (d1) {
+        float x[8];
+        load8(x, d1 + i);
+        if (d2) {
+            float y[8];
+            load8(y, d2 + i);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) x[k] += y[k];
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] += x[k];
+        store8(h + i, v);
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v[k] = fmaf(tanhf(a * v[k]), ww[k], bb[k]);
+    store8(out + i, v);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+stream_concat_kernel(T* __restrict__ out, const float* __restrict__ h, const T* __restrict__ d1, const T* __restrict__ d2, const float* __restrict__ e,
+                     int D, int64_t n) {
+    pdl_trigger();
+    pdl_wait();
+    for (int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x; i < n; i += static_cast<int64_t>(gridDim.x) * 256) {
+        const int64_t t = i / D;
+        float v = h[i];
+        if (d1) {
+            float d = to_float(d1[i]);
+            if (d2) d += to_float(d2[i]);
+            v += d;
+        }
+        out[i + t * D] = from_float<T>(v);
+        out[i + (t + 1) * D] = from_float<T>(e[i]);
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+stream_concat_vec_kernel(T* __restrict__ out, const float* __restrict__ h, const T* __restrict__ d1, const T* __restrict__ d2, const float* __restrict__ e,
+                         int D, int64_t n) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) * 8;
+    if (i >= n) return;
+    const int64_t t = i / D;
+    float v[8], x[8], y[8];
+    load8(v, h + i);
+    load8(y, e + i);
+    if (d1) {
+        load8(x, d1 + i);
+        if (d2) {
+            float z[8];
+            load8(z, d2 + i);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) x[k] += z[k];
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] += x[k];
+    }
+    store8(out + i + t * D, v);
+    store8(out + i + (t + 1) * D, y);
 }
 
 __device__ __forceinline__ float gelu_tanh_of(float z) {
@@ -434,6 +536,42 @@ extern "C" int cvb_resid_update(float* h, const void* d1, const void* d2, const 
                               (const TY*)d2, e, vec, w, (TY*)out, D, eps);                                                \
     else launch_kernel(resid_update_kernel<TY>, dim3(T), dim3(kUpdateThreads), 0, stream, h, (const TY*)d1, (const TY*)d2, \
                        e, vec, w, (TY*)out, D, eps)
+    CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+    return launch_status();
+}
+
+extern "C" int cvb_tanh_update(float* h, const void* d1, const void* d2, const float* alpha, const float* w, const float* b, void* out, int T, int D,
+                               int dtype, cudaStream_t stream) {
+    if (T == 0) return CVB_OK;
+    if (T < 0 || D <= 0) return CVB_E_SIZE;
+    if ((d2 != nullptr && d1 == nullptr) || h == nullptr || alpha == nullptr || w == nullptr || b == nullptr || out == nullptr) return CVB_E_SHAPE;
+    auto al = [](const void* p) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int64_t n = static_cast<int64_t>(T) * D, want = (n + 255) / 256;
+    const bool vec = D % 8 == 0 && al(h) && al(d1) && al(d2) && al(w) && al(b) && al(out);
+#define CALL(TY)                                                                                                              \
+    if (vec) launch_kernel(tanh_update_vec_kernel<TY>, dim3(static_cast<unsigned>((n / 8 + 255) / 256)), dim3(256), 0, stream, h, (const TY*)d1,   \
+                           (const TY*)d2, alpha, w, b, (TY*)out, D, n);                                                       \
+    else launch_kernel(tanh_update_kernel<TY>, dim3(static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16)), dim3(256), 0, stream, h,            \
+                       (const TY*)d1, (const TY*)d2, alpha, w, b, (TY*)out, D, n)
+    CVB_DISPATCH_DTYPE(dtype, CALL);
+#undef CALL
+    return launch_status();
+}
+
+extern "C" int cvb_stream_concat(void* out, const float* h, const void* d1, const void* d2, const float* e, int T, int D, int dtype,
+                                 cudaStream_t stream) {
+    if (T == 0) return CVB_OK;
+    if (T < 0 || D <= 0) return CVB_E_SIZE;
+    if ((d2 != nullptr && d1 == nullptr) || h == nullptr || e == nullptr || out == nullptr) return CVB_E_SHAPE;
+    auto al = [](const void* p) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int64_t n = static_cast<int64_t>(T) * D, want = (n + 255) / 256;
+    const bool vec = D % 8 == 0 && al(h) && al(d1) && al(d2) && al(e) && al(out);
+#define CALL(TY)                                                                                                              \
+    if (vec) launch_kernel(stream_concat_vec_kernel<TY>, dim3(static_cast<unsigned>((n / 8 + 255) / 256)), dim3(256), 0, stream, (TY*)out, h,      \
+                           (const TY*)d1, (const TY*)d2, e, D, n);                                                            \
+    else launch_kernel(stream_concat_kernel<TY>, dim3(static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16)), dim3(256), 0, stream, (TY*)out, h, \
+                       (const TY*)d1, (const TY*)d2, e, D, n)
     CVB_DISPATCH_DTYPE(dtype, CALL);
 #undef CALL
     return launch_status();

@@ -166,20 +166,20 @@ __device__ __forceinline__ float glu_of(float g, float u, float limit, float alp
 }
 
 template <typename T, int ACT>
-__global__ void glu_act_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n, int I, float limit, float alpha) {
+__global__ void glu_act_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ gu, int gu_stride, int64_t n, int I, float limit, float alpha, float scale) {
     pdl_trigger();
     pdl_wait();
     for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
          i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
         const int64_t t = i / I;
         const int c = static_cast<int>(i - t * I);
-        out[i] = from_float<T>(glu_of<ACT>(to_float(gu[t * 2 * I + c]), to_float(gu[t * 2 * I + I + c]), limit, alpha));
+        out[t * out_stride + c] = from_float<T>(glu_of<ACT>(to_float(gu[t * gu_stride + c]), to_float(gu[t * gu_stride + I + c]), limit, alpha) * scale);
     }
 }
 
 // 16 bytes of gate and of up per thread: I is a multiple of the chunk and all rows start on 16 bytes
 template <typename T, int ACT>
-__global__ void glu_act_vec_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n_chunks, int I, float limit, float alpha) {
+__global__ void glu_act_vec_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ gu, int gu_stride, int64_t n_chunks, int I, float limit, float alpha, float scale) {
     pdl_trigger();
     pdl_wait();
     constexpr int N = 16 / sizeof(T);
@@ -189,11 +189,11 @@ __global__ void glu_act_vec_kernel(T* __restrict__ out, const T* __restrict__ gu
     const int64_t t = k / per_row;
     const int c = static_cast<int>(k - t * per_row) * N;
     alignas(16) T g[N], u[N], o[N];
-    *reinterpret_cast<uint4*>(g) = *reinterpret_cast<const uint4*>(gu + t * 2 * I + c);
-    *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(gu + t * 2 * I + I + c);
+    *reinterpret_cast<uint4*>(g) = *reinterpret_cast<const uint4*>(gu + t * gu_stride + c);
+    *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(gu + t * gu_stride + I + c);
 #pragma unroll
-    for (int i = 0; i < N; ++i) o[i] = from_float<T>(glu_of<ACT>(to_float(g[i]), to_float(u[i]), limit, alpha));
-    *reinterpret_cast<uint4*>(out + t * I + c) = *reinterpret_cast<const uint4*>(o);
+    for (int i = 0; i < N; ++i) o[i] = from_float<T>(glu_of<ACT>(to_float(g[i]), to_float(u[i]), limit, alpha) * scale);
+    *reinterpret_cast<uint4*>(out + t * out_stride + c) = *reinterpret_cast<const uint4*>(o);
 }
 
 template <typename T>
@@ -293,20 +293,22 @@ extern "C" int cvb_gated_norm_add(float* h, const void* y, const void* z, const 
     return launch_status();
 }
 
-extern "C" int cvb_glu_act(void* out, const void* gate_up, int T, int I, int act, float limit, float alpha, int dtype, cudaStream_t stream) {
+// Rows of out and gate_up may lie inside wider rows; the outputs are multiplied by `scale`.
+extern "C" int cvb_glu_act(void* out, int out_stride, const void* gate_up, int gu_stride, int T, int I, int act, float limit, float alpha, float scale,
+                           int dtype, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
     if (T < 0 || I <= 0) return CVB_E_SIZE;
-    if (act < 0 || act > 1) return CVB_E_SHAPE;
+    if (act < 0 || act > 1 || out_stride < I || gu_stride < 2 * I) return CVB_E_SHAPE;
     const int64_t n = static_cast<int64_t>(T) * I, want = (n + 255) / 256;
     const unsigned blocks = static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16);
     const bool aligned = ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(gate_up)) & 15) == 0;
 #define CALL_ACT(TY, ACT)                                                                                                                 \
-    if (aligned && I % (16 / (int)sizeof(TY)) == 0) {                                                                                     \
+    if (aligned && I % (16 / (int)sizeof(TY)) == 0 && out_stride % (16 / (int)sizeof(TY)) == 0 && gu_stride % (16 / (int)sizeof(TY)) == 0) {                                                                                      \
         const int64_t nc = n / (16 / (int)sizeof(TY));                                                                                    \
         launch_kernel(glu_act_vec_kernel<TY, ACT>, dim3(static_cast<unsigned>((nc + 255) / 256)), dim3(256), 0, stream, (TY*)out,         \
-                      (const TY*)gate_up, nc, I, limit, alpha);                                                                           \
+                      out_stride, (const TY*)gate_up, gu_stride, nc, I, limit, alpha, scale);                                                                           \
     } else                                                                                                                                \
-        launch_kernel(glu_act_kernel<TY, ACT>, dim3(blocks), dim3(256), 0, stream, (TY*)out, (const TY*)gate_up, n, I, limit, alpha)
+        launch_kernel(glu_act_kernel<TY, ACT>, dim3(blocks), dim3(256), 0, stream, (TY*)out, out_stride, (const TY*)gate_up, gu_stride, n, I, limit, alpha, scale)
 #define CALL(TY)                                                                                                                          \
     if (act == 0) { CALL_ACT(TY, 0); } else { CALL_ACT(TY, 1); }
     CVB_DISPATCH_DTYPE(dtype, CALL);

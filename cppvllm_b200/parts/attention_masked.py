@@ -7,7 +7,7 @@
                                               with ``v_mix = "first"`` (that layer keeps its values for the step); the mixed
                                               value is what the cache holds
     s_ij = scale q_i . k_j;  s <- c tanh(s / c) (``softcap`` = c);  s <- s - r1_h ln(1 + r2_h (i - j)) (``distance_bias``)
-    visible: j <= i and  same chunk of ``chunk`` positions  |  i - j < ``window``  |  all;  with ``pool`` = P beside a window
+    visible: j <= i and  same chunk of ``chunk`` positions  |  i - j < ``window`` or j < ``keep_first``  |  all;  with ``pool`` = P beside a window
              also one key and value per block of P positions that lies wholly before the window (the means of the block's
              cached keys and values), in the same softmax
     softmax, with exp(sink_h) added to the denominator (``sink``);  o_h <- o_h sigmoid((Wg x)_h) (``head_gate``), or
@@ -31,7 +31,7 @@ from .base import CacheSpec, Mixer, WeightSpec, register_part
 @register_part("mixer", "masked_attention")
 class MaskedAttention(Mixer):
     def __init__(self, runtime, prefix="", names=None, *, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int,
-                 scale: float, eps: float, qk_norm: bool = True, position=None, chunk: int = 0, window: int = 0, pool: int = 0,
+                 scale: float, eps: float, qk_norm: bool = True, position=None, chunk: int = 0, window: int = 0, pool: int = 0, keep_first: int = 0,
                  softcap: float = 0.0, distance_bias: bool = False, sink: bool = False, head_gate: bool = False,
                  v_mix: str = "none", qkv_bias: bool = False, element_gate: bool = False, force_general: bool = False):
         super().__init__(runtime, prefix, names)
@@ -39,14 +39,15 @@ class MaskedAttention(Mixer):
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} key/value heads")
         if v_mix not in ("none", "first", "mix"):
             raise ValueError(f"v_mix is 'none', 'first' or 'mix', got {v_mix!r}")
-        if min(chunk, window, pool) < 0 or (pool and not window):
-            raise ValueError("chunk, window and pool are not negative, and pooled blocks stand beside a window")
+        if min(chunk, window, pool, keep_first) < 0 or ((pool or keep_first) and not window):
+            raise ValueError("chunk, window, pool and keep_first are not negative; pooled blocks and kept first tokens stand beside a window")
         if head_gate and element_gate:
             raise ValueError("the output has one gate: per head or per element")
         self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
         self.dim, self.vdim, self.scale, self.eps = int(dim), int(vdim), float(scale), float(eps)
         self.qk_norm, self.position = bool(qk_norm), position
         self.chunk, self.window, self.pool, self.softcap = int(chunk), int(window), int(pool), float(softcap or 0.0)
+        self.keep_first = int(keep_first)
         self.distance_bias, self.sink, self.head_gate, self.v_mix = bool(distance_bias), bool(sink), bool(head_gate), v_mix
         self.qkv_bias, self.element_gate = bool(qkv_bias), bool(element_gate)
         self.core_width = self.num_heads * self.vdim
@@ -60,7 +61,8 @@ class MaskedAttention(Mixer):
     def cache_spec(self) -> CacheSpec:
         if self.planes == 2:
             return CacheSpec((2, self.num_kv_heads, self.dim + self.vdim), token_axis=2)
-        return CacheSpec((self.num_kv_heads, self.dim + self.vdim), token_axis=1)
+        # pages wholly behind the window are given back, but for those of the kept first tokens
+        return CacheSpec.key_with_value(self.num_kv_heads, self.dim, self.vdim, window=self.window, keep_first=self.keep_first)
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         D, H, G, dk, dv = self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim
@@ -159,16 +161,16 @@ class MaskedAttention(Mixer):
                 if self.chunk:
                     seen = min(seen, self.chunk)
                 if self.window:
-                    seen = min(seen, self.window + (ctx.max_kv_len // self.pool if self.pool else 0))
+                    seen = min(seen, self.window + self.keep_first + (ctx.max_kv_len // self.pool if self.pool else 0))
                 splits = ops.attn_masked_decode_splits(ctx.num_seqs, G, seen)
                 if splits > 1:
                     most = ops.attn_keys_scratch_floats(self.rt.workspace.max_seqs, G, dv, 8)
                     scratch = self.rt.workspace.flat(f"attn_masked_parts_{G}_{dv}", most, torch.float32)
             ops.attn_masked_bf16(att, q, cache.pages, g.block_tables, ctx.cu_seqlens, ctx.positions, ctx.num_seqs,
                                  ops.attn_keys_tiles(q_lens, H, G), H, G, dk, dv, g.page_size, self.scale, planes=self.planes,
-                                 chunk=self.chunk, window=self.window, pool=self.pool, softcap=self.softcap, r1=self.r1, r2=self.r2,
+                                 chunk=self.chunk, window=self.window, pool=self.pool, keep_first=self.keep_first, softcap=self.softcap, r1=self.r1, r2=self.r2,
                                  sink=self.sinks, gate=gate, all_single=single, splits=splits, scratch=scratch, out_scale=out_scale)
             return
         ops.attn_masked_general(att, q, cache.pages, g.block_tables, ctx.seq_of_token, ctx.positions, ctx.num_tokens, H, G, dk, dv,
-                                g.page_size, self.scale, planes=self.planes, chunk=self.chunk, window=self.window, pool=self.pool,
+                                g.page_size, self.scale, planes=self.planes, chunk=self.chunk, window=self.window, pool=self.pool, keep_first=self.keep_first,
                                 softcap=self.softcap, r1=self.r1, r2=self.r2, sink=self.sinks, gate=gate, out_scale=out_scale)

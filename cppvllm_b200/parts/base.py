@@ -53,6 +53,10 @@ def part_class(category: str, kind: str) -> type:
                          f"{sorted(_REGISTRY.get(category, {}))}") from None
 
 
+def has_part(category: str, kind: str) -> bool:
+    return kind in _REGISTRY.get(category, {})
+
+
 def build_part(category: str, spec, runtime, **extra):
     cls = part_class(category, spec.kind)
     return cls(runtime, prefix=spec.prefix, names=dict(spec.names), **spec.params, **extra)
@@ -86,6 +90,10 @@ class CacheSpec:
     @staticmethod
     def keys_and_values(num_kv_heads: int, head_dim: int, window: int = 0) -> "CacheSpec":
         return CacheSpec((2, int(num_kv_heads), int(head_dim)), token_axis=2, window=int(window))
+
+    @staticmethod
+    def key_with_value(num_kv_heads: int, dim: int, vdim: int, window: int = 0, keep_first: int = 0) -> "CacheSpec":
+        return CacheSpec((int(num_kv_heads), int(dim) + int(vdim)), token_axis=1, window=int(window), keep_first=int(keep_first))
 
     @staticmethod
     def keys_only(num_kv_heads: int, head_dim: int, window: int = 0, keep_first: int = 0) -> "CacheSpec":
@@ -232,7 +240,14 @@ class Mixer(Part):
 
 
 class FeedForward(Part):
+    """A feed-forward keeps nothing between steps; asked like a mixer (a member of a ``side_by_side`` group) it says so."""
     category = "ffn"
+
+    def cache_spec(self) -> Optional[CacheSpec]:
+        return None
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return None
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         raise NotImplementedError

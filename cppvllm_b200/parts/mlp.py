@@ -5,7 +5,7 @@ gu = x Wgu^T with Wgu = rows(gate_proj) over rows(up_proj); act = T( rnd(silu(g)
 
 ``gated_mlp``: y = Wdown (act(Wgate x) * (Wup x)), act = "gelu_tanh" (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))); tensors
 ``gate|up|down`` (the names are parameters), no biases.  Prompt portions that fill the SMs take the product whose tcgen05 epilogue is
-the gated activation."""
+the gated activation.  As a member of ``side_by_side`` it offers what lies between its products (``core``)."""
 from __future__ import annotations
 
 from typing import Dict
@@ -92,7 +92,8 @@ class GatedMLP(FeedForward):
             raise ValueError(f"activation '{activation}' is not built; built: gelu_tanh")
         self.hidden_size, self.intermediate_size, self.activation = int(hidden_size), int(intermediate_size), activation
         self.gate_name, self.up_name, self.down_name = gate_name, up_name, down_name
-        self.w_gate_up = self.w_down = None
+        self.core_width = self.intermediate_size
+        self.w_in = self.w_o = None               # gate rows over up rows; the down projection
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         D, I = self.hidden_size, self.intermediate_size
@@ -103,22 +104,25 @@ class GatedMLP(FeedForward):
         g, u = tensors[self.full_name(self.gate_name)], tensors[self.full_name(self.up_name)]
         if g.dtype != u.dtype:
             g, u = g.float(), u.float()
-        self.w_gate_up = torch.cat([g, u], dim=0).contiguous()
-        self.w_down = tensors[self.full_name(self.down_name)]
+        self.w_in = torch.cat([g, u], dim=0).contiguous()
+        self.w_o = tensors[self.full_name(self.down_name)]
 
     def weight_bytes(self) -> int:
-        return sum(w.numel() * w.element_size() for w in (self.w_gate_up, self.w_down))
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o))
 
     def _project(self, x, w, out, rows):
         return ops.linear(x, w, out=out) if self.rt.plain_kernels else ops.project_rows(x, w, out, rows)
+
+    def core(self, packed, out, scale, ctx, cache, state):
+        return ops.geglu(out, packed, scale)
 
     def forward(self, x, ctx):
         T = x.shape[0]
         ws = self.rt.workspace
         act = ws.rows("ffn_act", T, self.intermediate_size, x.dtype)
-        if not self.rt.plain_kernels and ops.gated_product_fused(x.dtype, self.w_gate_up, T):
-            ops.gemm_bf16_tcgen05(act, x, self.w_gate_up, geglu=True)        # gate and up never travel through memory
+        if not self.rt.plain_kernels and ops.gated_product_fused(x.dtype, self.w_in, T):
+            ops.gemm_bf16_tcgen05(act, x, self.w_in, geglu=True)             # gate and up never travel through memory
         else:
-            gu = self._project(x, self.w_gate_up, ws.rows("ffn_gate_up", T, 2 * self.intermediate_size, x.dtype), T)
+            gu = self._project(x, self.w_in, ws.rows("ffn_gate_up", T, 2 * self.intermediate_size, x.dtype), T)
             ops.geglu(act, gu)
-        return self._project(act, self.w_down, ws.rows("ffn_out", T, self.hidden_size, x.dtype), T)
+        return self._project(act, self.w_o, ws.rows("ffn_out", T, self.hidden_size, x.dtype), T)

@@ -13,7 +13,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..csrc import ops
-from .base import CacheSpec, Runtime, StateSpec, WeightSpec, build_part, part_class
+from .base import CacheSpec, Runtime, StateSpec, WeightSpec, build_part, has_part, part_class
 from .spec import ModelSpec, RunEntry
 
 
@@ -39,7 +39,8 @@ class CausalLM:
         self._check_shared_caches()
 
     def _build_mixer(self, spec):
-        """A mixer from its spec: a position encoding it names is handed over, and mixers it is made of (``members``) are built first."""
+        """A mixer from its spec: a position encoding it names is handed over, and what it is made of (``members``: mixers, or feed-forwards
+        that run beside them) is built first."""
         params = dict(spec.params)
         pos_name = params.pop("position", None)
         if pos_name is not None:
@@ -48,7 +49,8 @@ class CausalLM:
             params["position"] = self.positions[pos_name]
         if "members" in params:
             params["members"] = [self._build_mixer(m) for m in params["members"]]
-        return part_class("mixer", spec.kind)(self.rt, prefix=spec.prefix, names=dict(spec.names), **params)
+        category = "mixer" if has_part("mixer", spec.kind) or not has_part("ffn", spec.kind) else "ffn"
+        return part_class(category, spec.kind)(self.rt, prefix=spec.prefix, names=dict(spec.names), **params)
 
     @property
     def capturable(self) -> bool:

@@ -18,6 +18,11 @@ type; only the projections around them are products in the activations' type.
   S <- diag(g) S + k v^T;  o = S^T q;  y = Wo concat_h(RMSNorm(o_h) * w * silu(Wg x)_h), w shared by the heads.  State per request:
   [H, dim, vdim].  A step of decoded tokens is one kernel between the projections.  The inner size of the low-rank projection is
   whatever the checkpoint holds.
+* ``ssd``: [z | u | dt] = Win x;  [x | B | C] = silu(causal convolution of u over time per channel + bias);  dt <- softplus(dt + dt_bias) per head;
+  S <- exp(-exp(A_h) dt) S + dt B x^T  ([state, vdim], B and C of group h / (heads / groups));  y = S^T C + D_h x;
+  out = Wo (RMSNorm_parts(y * silu(z)) * w), the norm over ``norm_parts`` equal parts of the row, the gate in front of it.  State per
+  request: S of every head and behind it a ring of the last ``taps`` inputs of the convolution.  Portions in bf16 run in chunks on the tensor
+  cores, decoded tokens in one kernel and the norm; float32 and other sizes take the token-by-token scan (csrc/ssd.cu, csrc/recurrent.cu).
 """
 from __future__ import annotations
 
@@ -286,3 +291,81 @@ class GatedLinearMixer(Mixer):
         if self._scaled[0] != scale:                      # the constant rides on the norm's weight
             self._scaled = (scale, (self.w_norm * scale).contiguous())
         return ops.gated_norm(out, o, packed[:, g_off:g_off + H * dv], self._scaled[1], H, self.eps, gate_act="silu")
+
+
+@register_part("mixer", "ssd")
+class StateSpaceMixer(Mixer):
+    def __init__(self, runtime, prefix="", names=None, *, hidden_size: int, num_heads: int, groups: int, state: int, vdim: int, taps: int,
+                 norm_parts: int, eps: float):
+        super().__init__(runtime, prefix, names)
+        self.hidden_size, self.num_heads, self.groups, self.dim, self.vdim = int(hidden_size), int(num_heads), int(groups), int(state), int(vdim)
+        self.taps, self.norm_parts, self.eps = int(taps), int(norm_parts), float(eps)
+        if self.num_heads % self.groups:
+            raise ValueError(f"{self.num_heads} heads are not a multiple of {self.groups} groups")
+        self.inner = self.num_heads * self.vdim
+        if self.inner % self.norm_parts:
+            raise ValueError(f"{self.inner} columns do not fall into {self.norm_parts} equal parts")
+        if self.taps < 1:
+            raise ValueError("a convolution has at least one tap")
+        if self.dim > 512:
+            raise ValueError("the scan kernel keeps at most 512 rows of a state")
+        self.channels = self.inner + 2 * self.groups * self.dim
+        self.core_width = self.inner
+        self.w_in = self.w_o = None
+
+    def state_spec(self) -> StateSpec:
+        n = self.num_heads * self.dim * self.vdim + (self.taps * self.channels if self.taps > 1 else 0)
+        return StateSpec((-(-n // 4) * 4,), torch.float32)           # whole 16-byte pieces: every slot's matrices start on one
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        D, H, C = self.hidden_size, self.num_heads, self.channels
+        f = self.full_name
+        return {f("in"): WeightSpec((self.inner + C + H, D)), f("conv"): WeightSpec((C, self.taps), role="vector"), f("conv.b"): WeightSpec((C,), role="vector"),
+                f("dt_bias"): WeightSpec((H,), role="vector"), f("A_log"): WeightSpec((H,), role="vector"), f("D"): WeightSpec((H,), role="vector", init="norm"),
+                f("norm"): WeightSpec((self.inner,), role="vector", init="norm"), f("o"): WeightSpec((D, self.inner))}
+
+    def bind(self, tensors) -> None:
+        t = lambda n: tensors[self.full_name(n)]          # noqa: E731
+        self.w_in, self.w_o = t("in"), t("o")
+        self.conv_w, self.conv_b = t("conv").t().contiguous(), t("conv.b").contiguous()
+        self.dt_bias, self.neg_a, self.skip, self.w_norm = t("dt_bias").contiguous(), (-torch.exp(t("A_log"))).contiguous(), t("D").contiguous(), t("norm").contiguous()
+
+    def weight_bytes(self) -> int:
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o))
+
+    def forward(self, x, ctx, cache, state):
+        T = x.shape[0]
+        ws = self.rt.workspace
+        packed = _project(self.rt, x, self.w_in, ws.rows("rec_in", T, self.w_in.shape[0], x.dtype), T)
+        y = self.core(packed, ws.rows("rec_y", T, self.core_width, x.dtype), 1.0, ctx, cache, state)
+        return _project(self.rt, y, self.w_o, ws.rows("attn_proj", T, self.hidden_size, x.dtype), T)
+
+    def core(self, packed, out, scale, ctx, cache, state):
+        T, S = packed.shape[0], ctx.num_seqs
+        sizes = (self.num_heads, self.groups, self.dim, self.vdim)
+        H, G, N, P = sizes
+        ws, f32 = self.rt.workspace, torch.float32
+        u_off, dt_off = self.inner, self.inner + self.channels
+        y = ws.rows("rec_o", T, self.inner, f32)
+        if ctx.all_decode and T == S and not self.rt.plain_kernels and ops.ssd_step_supported(N, P):
+            ops.ssd_step(y, packed, u_off, dt_off, self.conv_w, self.conv_b, self.dt_bias, self.neg_a, self.skip, state, ctx.cu_seqlens,
+                         ctx.state_slots, ctx.positions, S, *sizes)
+        else:
+            q_lens = ctx.q_lens if ctx.q_lens is not None else [1] * S
+            chunks = not self.rt.plain_kernels and ops.ssd_chunks_supported(packed.dtype, N, P)
+            u = ws.rows("ssd_u", T, self.channels, packed.dtype if chunks else f32)
+            dt, la = ws.rows("ssd_dt", T, H, f32), ws.rows("ssd_log_decay", T, H, f32)
+            ops.ssd_prep(u, dt, la, packed, u_off, dt_off, self.conv_w, self.conv_b, self.dt_bias, self.neg_a, state, ctx.seq_of_token,
+                         ctx.cu_seqlens, ctx.state_slots, ctx.positions, *sizes)
+            ops.ssd_ring(state, packed, u_off, dt_off, self.taps, ctx.cu_seqlens, ctx.state_slots, ctx.positions, S, *sizes)
+            if chunks:
+                ends = decays = None
+                if max(q_lens) > ops.SSD_CHUNK:
+                    held = ops.ssd_held_chunks(ws.max_tokens)
+                    ends = ws.flat(f"ssd_ends_{H}_{N}_{P}", held * H * N * P, f32)
+                    decays = ws.flat(f"ssd_decays_{H}", held * H, f32)
+                ops.ssd_chunks(y, u, dt, la, self.skip, state, ctx.cu_seqlens, ctx.state_slots, q_lens, *sizes, ends=ends, decays=decays)
+            else:
+                i, n = self.inner, G * N
+                ops.skip_scan(y, u[:, i + n:], u[:, i:i + n], u[:, :i], la, dt, self.skip, state, ctx.cu_seqlens, ctx.state_slots, S, H, G, N, P)
+        return ops.gate_norm(out, y, packed[:, :self.inner], self.w_norm, self.norm_parts, self.eps, scale)

@@ -1,4 +1,5 @@
-"""Mixer ``side_by_side``: several mixers that read the same input, their outputs added up with a constant each:
+"""Mixer ``side_by_side``: several mixers (or mixers and a feed-forward: a layer whose two sublayers share one norm) that read the same
+input, their outputs added up with a constant each:
 
     y = sum_m scale_m mixer_m(x)
 
@@ -21,7 +22,7 @@ from ..csrc import ops
 from .base import Mixer, WeightSpec, register_part
 from .recurrent import _cat_rows, _project
 
-ROW_STEP = 8        # the joined input projection's rows are padded to whole 16-byte chunks of bf16 outputs
+ROW_STEP = 8        # every member's rows of the joined input projection are padded to whole 16-byte chunks of bf16 outputs
 
 
 @register_part("mixer", "side_by_side")
@@ -61,15 +62,16 @@ class SideBySideMixer(Mixer):
 
     def bind(self, tensors) -> None:
         self.in_cols = []
-        col = 0
+        col, rows = 0, []
         for m in self.members:
             m.bind(tensors)
-            self.in_cols.append((col, col + m.w_in.shape[0]))
-            col += m.w_in.shape[0]
-        rows = [m.w_in for m in self.members]
-        pad = -col % ROW_STEP
-        if pad:
-            rows.append(torch.zeros(pad, self.hidden_size, dtype=rows[0].dtype, device=rows[0].device))
+            n = m.w_in.shape[0]
+            self.in_cols.append((col, col + n))
+            rows.append(m.w_in)
+            pad = -n % ROW_STEP
+            if pad:
+                rows.append(torch.zeros(pad, self.hidden_size, dtype=m.w_in.dtype, device=m.w_in.device))
+            col += n + pad
         self.w_in = _cat_rows(rows)
         outs = [m.w_o for m in self.members]
         if len({o.dtype for o in outs}) > 1:

@@ -14,6 +14,10 @@ where a norm hands it to a matrix product.
 * block ``parallel``: x = norm(h);  h <- h + (mixer(x) + ffn(x)).  One norm; both sublayers read its output; a layer may
   have no feed-forward.  The two outputs leave the block as pending deltas, so that the next block's norm (or the final
   norm) adds them: a layer costs one elementwise kernel.
+* norm ``dynamic_tanh``: y = T(tanh(alpha x) * w + b), element by element, no statistics; alpha is one learned number.  ``add_forward`` as
+  above.
+* input ``concat_input``: in front of a run of layers, h <- W [h ; embedded] (W [D, 2 D]); pending deltas are folded in by the kernel
+  that lays the two side by side, and the product's float sums are the new stream.
 * input ``pass_input``: in front of pass number t of a repeated run of layers, h <- (h + embedded) + step[t] (the
   embedding output only from the second pass on); pending deltas are folded in by the same kernel.
 """
@@ -126,6 +130,35 @@ class WideRMSNorm(Norm):
         return ops.resid_update(residual, _as_tuple(delta), norm_weight=self.weight, eps=self.eps, out=self._out(residual, out))
 
 
+@register_part("norm", "dynamic_tanh")
+class DynamicTanh(Norm):
+    """Tensors <prefix><name>, <name>.alpha (a scalar) and <name>.b."""
+
+    def __init__(self, runtime, prefix="", names=None, *, size: int, weight_name: str = "weight", buffer: str = "normed"):
+        super().__init__(runtime, prefix, names)
+        self.size, self.weight_name, self.buffer = int(size), weight_name, buffer
+        self.scale = self.shift = self.alpha = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        n = self.full_name(self.weight_name)
+        return {n: WeightSpec((self.size,), role="vector", init="norm"), n + ".b": WeightSpec((self.size,), role="vector"),
+                n + ".alpha": WeightSpec((), role="vector", init="norm")}
+
+    def bind(self, tensors) -> None:
+        n = self.full_name(self.weight_name)
+        self.scale, self.shift, self.alpha = tensors[n].contiguous(), tensors[n + ".b"].contiguous(), tensors[n + ".alpha"].reshape(1).contiguous()
+
+    def weight_bytes(self) -> int:
+        return 2 * self.size * self.scale.element_size()
+
+    def forward(self, x, out=None):
+        return self.add_forward(x, None, out)
+
+    def add_forward(self, residual, delta, out=None):
+        out = out if out is not None else self.rt.workspace.rows(self.buffer, residual.shape[0], self.size, self.rt.dtype)
+        return ops.tanh_update(residual, _as_tuple(delta), self.alpha, self.scale, self.shift, out)
+
+
 @register_part("embedding", "normed_tokens")
 class NormedTokenEmbedding(Part):
     category = "embedding"
@@ -233,4 +266,29 @@ class PassInput(StreamInput):
         if rows is not None and rows.data_ptr() == h.data_ptr():
             raise ValueError("the embedding output was not kept apart from the residual stream")
         ops.resid_update(h, _as_tuple(pending), rows=rows, vector=self.steps[index])
+        return h, None
+
+
+@register_part("input", "concat_input")
+class ConcatInput(StreamInput):
+    def __init__(self, runtime, prefix="", names=None, *, hidden_size: int, weight_name: str = "in"):
+        super().__init__(runtime, prefix, names)
+        self.hidden_size, self.weight_name = int(hidden_size), weight_name
+        self.weight: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {self.full_name(self.weight_name): WeightSpec((self.hidden_size, 2 * self.hidden_size))}
+
+    def bind(self, tensors) -> None:
+        self.weight = tensors[self.full_name(self.weight_name)]
+
+    def weight_bytes(self) -> int:
+        return self.weight.numel() * self.weight.element_size()
+
+    def forward(self, h, pending, embedded, index: int):
+        if embedded.data_ptr() == h.data_ptr():
+            raise ValueError("the embedding output was not kept apart from the residual stream")
+        T, D = h.shape
+        both = ops.stream_concat(self.rt.workspace.rows("stream_both", T, 2 * D, self.rt.dtype), h, _as_tuple(pending), embedded)
+        ops.linear(both, self.weight, out=h, out_dtype=torch.float32)
         return h, None
