@@ -50,6 +50,17 @@ from the best group.  Whole models stand beside Lorulix (the closest existing mo
 and its value, a mixer with a matrix of state per head, dense and routed feed-forwards) and Qwen3; its kernels beside the like kernels
 of Rumurax (attention, the projection's epilogue, the router), Dugulorn and Lorulix (scans, convolution, preparation), Givirax
 (experts), Qwen3 (the gated product) and the weight-streaming product (the recurrence of decoded tokens, which reads gate matrices).
+
+    python bench.py --design legalix
+
+The Legalix model of a size has the same width, heads and head size and a dense tanh-GELU feed-forward of the same inner size in every
+layer, beside the mixer; its layers repeat the pattern [state-space recurrence, attention behind a window of 1,024 tokens with 4 kept first
+tokens and capped scores, attention over a latent of 96 + 32 elements with a sink, state-space recurrence], and a loop goes through the middle
+layers twice, so that as many layers RUN as the compared models have: recurrences of inner size twice the width in heads of 64, 128 rows
+of state, 8 groups, 4 taps, a norm in 8 parts.  Whole models stand beside Sumevik (the closest existing model: a float32 stream, attention
+over entries of a key and its value, a recurrence with a matrix of state per head) and Qwen3; its kernels beside the like kernels of
+Sumevik and Rumurax (attention, the projection's epilogue, the recurrence, the norm behind it, the convolution), Dugulorn (latent attention)
+and Givirax (the stream's norm and the input of a repeated pass).
 """
 from __future__ import annotations
 
@@ -157,6 +168,24 @@ def sumevik_config(s, max_positions):
                 "router": {"experts": EXPERTS, "top": TOP, "groups": {"count": 2, "keep": 1}, "identity": SV_IDENTITY}}}
     return {"architecture": "Sumevik", "vocab": s["vocab"], "width": D, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
             "layers": [(recurrence, pair)[i % 2] for i in range(s["layers"])]}
+
+
+LG_WINDOW, LG_KEEP, LG_CAP, LG_STATE, LG_VDIM, LG_GROUPS = 1024, 4, 30.0, 128, 64, 8
+
+
+def legalix_config(s, max_positions):
+    D, H, hd = s["width"], s["heads"], s["dim"]
+    ssd = {"type": "mamba2", "mixer": {"heads": 2 * D // LG_VDIM, "vdim": LG_VDIM, "state": LG_STATE, "groups": LG_GROUPS, "conv": 4, "norm_groups": 8}}
+    window = {"type": "attention", "mixer": {"heads": H, "kv_heads": s["kv_heads"], "dim": hd, "vdim": hd, "scale": 1.0 / math.sqrt(hd), "softcap": LG_CAP,
+                                             "mask": {"size": LG_WINDOW, "keep_first": LG_KEEP}, "rot": {"dims": hd, "base": 1.0e6}}}
+    latent = {"type": "latent_attention", "mixer": {"heads": H, "dim": hd, "rot_dim": 32, "vdim": hd, "q_rank": 3 * D // 8, "kv_rank": 96,
+                                                    "scale": 1.0 / math.sqrt(hd + 32), "rot": {"dims": 32, "base": 1.0e4}}}
+    # as many layers run as the others have: the middle ones (a quarter of them) twice
+    loop = s["layers"] // 4
+    pattern = [ssd, window, latent, ssd]
+    layers = [dict(pattern[i % 4], mlp={"kind": "dense", "ff": s["ff"]}) for i in range(s["layers"] - loop)]
+    return {"architecture": "Legalix", "vocab": s["vocab"], "width": D, "embedding": {"scale": math.sqrt(D)}, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "layers": layers, "loop": {"start": 1, "stop": 1 + loop, "times": 2}}
 
 
 def qwen3_config(s, max_positions):
@@ -1040,9 +1069,181 @@ def sumevik_kernel_pairs(s, pk):
     return out
 
 
+def legalix_kernel_pairs(s, pk):
+    """Each kernel of the Legalix parts beside the like kernel of the closest designs at the same sizes (see kernel_pairs)."""
+    from .csrc import ops
+    d = torch.device("cuda:0")
+    g = torch.Generator(device="cuda").manual_seed(0)
+    bf, f32, i32 = torch.bfloat16, torch.float32, torch.int32
+    D, H, KV, hd, I = s["width"], s["heads"], s["kv_heads"], s["dim"], s["ff"]
+    page, out = 32, {}
+    hbm, flop = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+
+    def rnd(*shape, scale=1.0, dtype=bf):
+        return (torch.randn(*shape, generator=g, device=d, dtype=f32) * scale).to(dtype)
+
+    def pair(name, new_us, new_work, like_us, like_work, unit, like, note=None):
+        peak = hbm if unit == "bytes" else flop
+        fn, fl = new_work / (new_us * 1e-6) / peak, like_work / (like_us * 1e-6) / peak
+        out[name] = {"new_us": round(new_us, 2), "new_frac": round(fn, 4), "like_us": round(like_us, 2), "like_frac": round(fl, 4),
+                     "gap": round(fl / fn, 2), "roofline": "copy bandwidth" if unit == "bytes" else "bf16 peak", "like": like}
+        if note:
+            out[name]["note"] = note
+
+    # -- windowed attention: a prompt of 2,048 tokens, 8 decoded tokens -----------------------------------------------------
+    T, B = 2048, 8
+    n_pages = T // page
+    tables = torch.arange(n_pages, dtype=i32, device=d).view(1, n_pages)
+    cu, pos, slot0 = torch.tensor([0, T], dtype=i32, device=d), torch.arange(T, dtype=i32, device=d), torch.zeros(1, dtype=i32, device=d)
+    seq_of = torch.zeros(T, dtype=i32, device=d)
+    cu_b, pos_b = torch.arange(0, B + 1, dtype=i32, device=d), torch.full((B,), 4095, dtype=i32, device=d)
+    slots_b = torch.arange(0, B, dtype=i32, device=d)
+    scale = 1 / math.sqrt(hd)
+    q, att, gate_e = rnd(T, H * hd), torch.empty(T, H * hd, dtype=bf, device=d), rnd(T, H * hd)
+    tiles = ops.attn_keys_tiles([T], H, KV)
+    ent = rnd(n_pages + 1, KV, page, 2 * hd)
+    kw, kw_like = dict(window=LG_WINDOW, keep_first=LG_KEEP, softcap=LG_CAP), dict(chunk=SV_CHUNK)
+    new = _us(lambda i: ops.attn_masked_bf16(att, q, ent, tables, cu, pos, 1, tiles, H, KV, hd, hd, page, scale, out_scale=0.5, **kw))
+    like = _us(lambda i: ops.attn_masked_bf16(att, q, ent, tables, cu, pos, 1, tiles, H, KV, hd, hd, page, scale, gate=gate_e, out_scale=0.7, **kw_like))
+    seen = sum(min(p + 1, LG_WINDOW + min(LG_KEEP, max(0, p + 1 - LG_WINDOW))) for p in range(T))
+    pair("attention_window_prefill_2048", new, 4.0 * H * hd * seen, like, 4.0 * H * hd * sum(p % SV_CHUNK + 1 for p in range(T)), "flops",
+         "Sumevik attn_masked_kernel, chunks of 1,024, gate per element", note="a cap on every score")
+    copies, ctx = 4, 4096
+    pps = ctx // page
+    tabs = [torch.randperm(B * pps, generator=g, device=d).to(i32).view(B, pps).contiguous() for _ in range(copies)]
+    ents = [rnd(B * pps + 1, KV, page, 2 * hd) for _ in range(copies)]
+    z = ops.attn_masked_decode_splits(B, KV, LG_WINDOW + LG_KEEP)
+    parts = torch.empty(max(1, ops.attn_keys_scratch_floats(B, KV, hd, 8)), dtype=f32, device=d)
+    run = lambda **k: _us(lambda i: ops.attn_masked_bf16(att[:B], q[:B], ents[i % copies], tabs[i % copies], cu_b, pos_b, B, B, H, KV, hd, hd,   # noqa: E731
+                                                         page, scale, all_single=True, splits=z, scratch=parts, **k))
+    new, like = run(**kw), run(gate=gate_e[:B], **kw_like)
+    pair("attention_window_decode_b8", new, B * (LG_WINDOW + LG_KEEP) * KV * hd * 4.0, like, B * SV_CHUNK * KV * hd * 4.0, "bytes",
+         "Sumevik attn_masked_decode_kernel, chunks of 1,024, gate per element")
+    del ents
+    packed, q_out, w1 = rnd(T, (H + 2 * KV) * hd), torch.empty(T, H * hd, dtype=bf, device=d), torch.ones(hd, device=d)
+    cos, sin = torch.rand(T, hd // 2, generator=g, device=d), torch.rand(T, hd // 2, generator=g, device=d)
+    prep = lambda half, w: _us(lambda i: ops.masked_qkv_prep(q_out, packed, H, KV, hd, hd, 1e-5, q_weight=w, k_weight=w, cos=cos, sin=sin, rot=hd,   # noqa: E731
+                                                             interleaved=not half, positions=pos, pages=ent, slots=pos, page_size=page))
+    new, like = prep(True, None), prep(False, w1)
+    moved = T * (H + 2 * KV) * hd * 4.0
+    pair("projection_epilogue_2048_tokens", new, moved, like, moved, "bytes", "Rumurax masked_qkv_prep, with norms", note="pairs (i, i + dims / 2)")
+
+    # -- latent attention with a sink --------------------------------------------------------------------------------------
+    R, dr = 96, 32
+    HD = R + dr
+    q_lat, o_lat, sink = rnd(T, H * HD), torch.empty(T, H * R, dtype=bf, device=d), rnd(H, dtype=f32)
+    lat = rnd(n_pages + 1, page, HD)
+    ltiles = ops.attn_keys_tiles([T], H, 1)
+    run = lambda sk: _us(lambda i: ops.attn_keys_bf16(o_lat, q_lat, lat, tables, cu, pos, 1, ltiles, H, 1, HD, page, 0.09, value_dim=R, sink=sk))   # noqa: E731
+    new, like = run(sink), run(None)
+    flops = 2.0 * H * (HD + R) * T * (T + 1) / 2
+    pair("latent_attention_prefill_2048", new, flops, like, flops, "flops", "Dugulorn attn_keys_kernel, no sink")
+    lats = [rnd(B * pps + 1, page, HD) for _ in range(16)]
+    groups = min(n for n in range(1, H + 1) if H % n == 0 and H // n <= 16)
+    zl = ops.attn_keys_decode_splits(B, groups, ctx)
+    lparts = torch.empty(ops.attn_keys_scratch_floats(B, groups, HD, 8), dtype=f32, device=d)
+    run = lambda sk: _us(lambda i: ops.attn_keys_bf16(o_lat[:B], q_lat[:B], lats[i % 16], tabs[i % copies], cu_b, pos_b, B, B, H, groups, HD, page, 0.09,   # noqa: E731
+                                                      all_single=True, splits=zl, scratch=lparts, value_dim=R, kv_heads_in_pages=1, sink=sk))
+    new, like = run(sink), run(None)
+    pair("latent_attention_decode_b8", new, B * ctx * HD * 2.0, like, B * ctx * HD * 2.0, "bytes", "Dugulorn attn_keys_decode_kernel, no sink")
+    del lats
+    q_up, q_abs = rnd(T, H * (hd + dr)), rnd(H, T, R)
+    cl, sl = torch.rand(T, dr // 2, generator=g, device=d), torch.rand(T, dr // 2, generator=g, device=d)
+    new = _us(lambda i: ops.latent_q_turn(q_lat, q_up, H, hd, R, dr, dr, cl, sl, pos))
+    like = _us(lambda i: ops.latent_q_assemble(q_lat, q_abs, q_up, H, hd, R, dr, dr, cl, sl, pos))
+    pair("latent_queries_2048_tokens", new, T * H * dr * 4.0, like, T * H * HD * 4.0, "bytes", "latent_q_assemble (a copy of q_abs beside the turn)",
+         note="the batched product writes q_abs to its place")
+
+    # -- state-space recurrence ------------------------------------------------------------------------------------------------
+    HS, P, N, G = 2 * D // LG_VDIM, LG_VDIM, LG_STATE, LG_GROUPS
+    inner, C = HS * P, HS * P + 2 * G * N
+    sizes = (HS, G, N, P)
+    lin = rnd(T, inner + C + HS)
+    conv_w, conv_b, dt_b, neg_a, skip = rnd(4, C, dtype=f32), rnd(C, dtype=f32), rnd(HS, dtype=f32), -torch.rand(HS, generator=g, device=d), rnd(HS, dtype=f32)
+    sfloats = HS * N * P + 4 * C
+    st = torch.zeros(2, sfloats, dtype=f32, device=d)
+    u, dt, la = torch.empty(T, C, dtype=bf, device=d), torch.empty(T, HS, device=d), torch.empty(T, HS, device=d)
+    y32, wn, y = torch.empty(T, inner, device=d), torch.ones(inner, device=d), torch.empty(T, inner, dtype=bf, device=d)
+    held = ops.ssd_held_chunks(T)
+    ends, decays = torch.empty(held * HS * N * P, device=d), torch.empty(held * HS, device=d)
+    prep = lambda: ops.ssd_prep(u, dt, la, lin, inner, inner + C, conv_w, conv_b, dt_b, neg_a, st, seq_of, cu, slot0, pos, *sizes)      # noqa: E731
+    scan = lambda: ops.ssd_chunks(y32, u, dt, la, skip, st, cu, slot0, [T], *sizes, ends=ends, decays=decays)                             # noqa: E731
+    norm = lambda: ops.gate_norm(y, y32, lin[:, :inner], wn, 8, 1e-5)                                                                  # noqa: E731
+
+    def core(i):
+        prep()
+        ops.ssd_ring(st, lin, inner, inner + C, 4, cu, slot0, pos, 1, *sizes)
+        scan()
+        norm()
+    new = _us(core)
+    # Sumevik's gated linear attention over its own heads, from the packed projection to the normed output
+    dk, HK, HV, RK = hd // 2, H * hd // 2, H * hd, 16
+    gla = rnd(T, 2 * HK + 2 * HV + RK)
+    wa2, ab, wl = rnd(HK, RK, scale=0.1), rnd(HK, dtype=f32), torch.ones(hd, device=d)
+    zz, o32, y_lin = torch.empty(T, HK, device=d), torch.empty(T, HV, device=d), torch.empty(T, HV, dtype=bf, device=d)
+    st_l = torch.zeros(2, H * dk * hd, device=d)
+    chunk, held_l = ops.linear_chunk_tokens(T, H, dk, hd), ops.linear_held_chunks(T, H, dk, hd)
+    ends_l, dec_l = torch.empty(held_l * H * dk * hd, device=d), torch.empty(held_l * H * dk, device=d)
+    lscan = lambda: ops.linear_scan(o32, gla, 0, HK, 2 * HK, dk ** -0.5, zz, st_l, cu, slot0, [T], H, dk, hd, chunk, ends_l, dec_l)      # noqa: E731
+
+    def core_like(i):
+        ops.linear(gla[:, 2 * HK + 2 * HV:], wa2, out=zz, out_dtype=f32)
+        ops.linear_decay(zz, ab, 16.0)
+        lscan()
+        ops.gated_norm(y_lin, o32, gla[:, 2 * HK + HV:2 * HK + 2 * HV], wl, H, 1e-5, gate_act="silu")
+    like = _us(core_like)
+    pair("recurrence_core_2048_tokens", new, 4.0 * HS * N * P * T, like, 4.0 * H * dk * hd * T, "flops", "Sumevik gated linear attention, the same span",
+         note="from the packed projection to the gated, normed output; four flops an element of state and token")
+    new, like = _us(lambda i: scan()), _us(lambda i: lscan())
+    pair("recurrence_scan_2048_tokens", new, 4.0 * HS * N * P * T, like, 4.0 * H * dk * hd * T, "flops", "Sumevik linear_scan")
+    new = _us(lambda i: prep())
+    W, PW = D, D // SV_PART
+    lru_in, u_l, st_r = rnd(T, 2 * W), torch.empty(T, W, dtype=bf, device=d), torch.zeros(2, 5 * W, device=d)
+    bx, cb, cw = rnd(W, dtype=f32), rnd(W, dtype=f32), rnd(4, W, dtype=f32)
+    like = _us(lambda i: ops.lru_conv(u_l, lru_in, 0, W, PW, bx, cw, cb, st_r, seq_of, cu, slot0, pos))
+    pair("convolution_2048_tokens", new, T * (C * 4.0 + HS * 10.0), like, T * W * 4.0, "bytes", "Sumevik lru_conv", note="with silu, step sizes and decays")
+    new = _us(lambda i: norm())
+    like = _us(lambda i: ops.gated_norm(y_lin, o32, gla[:, 2 * HK + HV:2 * HK + 2 * HV], wl, H, 1e-5, gate_act="silu"))
+    pair("gate_and_norm_2048_tokens", new, T * inner * 8.0, like, T * HV * 8.0, "bytes", "Sumevik gated_norm")
+    n_copy = max(2, int(300e6 // (B * sfloats * 4)) + 1)
+    states = [torch.zeros(B + 1, sfloats, device=d) for _ in range(n_copy)]
+
+    def step(i):
+        ops.ssd_step(y32[:B], lin[:B], inner, inner + C, conv_w, conv_b, dt_b, neg_a, skip, states[i % n_copy], cu_b, slots_b, pos_b, B, *sizes)
+        ops.gate_norm(y[:B], y32[:B], lin[:B, :inner], wn, 8, 1e-5)
+    new = _us(step)
+    n_l = max(2, int(300e6 // (B * H * dk * hd * 4)) + 1)
+    states_l = [torch.zeros(B + 1, H * dk * hd, device=d) for _ in range(n_l)]
+    like = _us(lambda i: ops.linear_step(y_lin[:B], gla[:B], 0, HK, 2 * HK, 2 * HK + HV, 2 * HK + 2 * HV, wa2, ab, dk ** -0.5, 16.0, wl, 1e-5, 0.9,
+                                         states_l[i % n_l], cu_b, slots_b, B, H, dk, hd))
+    pair("recurrence_decode_b8", new, B * (HS * N * P * 8.0 + C * 20.0), like, B * H * dk * hd * 8.0, "bytes", "Sumevik linear_step",
+         note="state and ring read and written; with the norm behind it")
+    del states, states_l
+
+    # -- norm, feed-forward, the input of a pass ---------------------------------------------------------------------------------
+    h, delta, x_out = rnd(T, D, dtype=f32), rnd(T, D), torch.empty(T, D, dtype=bf, device=d)
+    alpha, w_d, b_d = torch.full((1,), 0.5, device=d), torch.ones(D, device=d), torch.zeros(D, device=d)
+    new = _us(lambda i: ops.tanh_update(h, (delta,), alpha, w_d, b_d, x_out))
+    like = _us(lambda i: ops.resid_update(h, (delta,), norm_weight=w_d, eps=1e-5, out=x_out))
+    pair("norm_2048_tokens", new, T * D * 12.0, like, T * D * 12.0, "bytes", "Givirax resid_update (RMS norm)")
+    new8, like8 = _us(lambda i: ops.tanh_update(h[:B], (delta[:B],), alpha, w_d, b_d, x_out[:B])), _us(
+        lambda i: ops.resid_update(h[:B], (delta[:B],), norm_weight=w_d, eps=1e-5, out=x_out[:B]))
+    pair("norm_8_decoded_tokens", new8, B * D * 12.0, like8, B * D * 12.0, "bytes", "Givirax resid_update (RMS norm)")
+    both, emb = torch.empty(T, 2 * D, dtype=bf, device=d), rnd(T, D, dtype=f32)
+    new = _us(lambda i: ops.stream_concat(both, h, (delta,), emb))
+    like = _us(lambda i: ops.resid_update(h, (delta,), rows=emb, vector=b_d))
+    pair("pass_input_2048_tokens", new, T * D * 14.0, like, T * D * 14.0, "bytes", "Givirax resid_update (embedding and vector added)")
+    wide = rnd(T, (H + 2 * KV) * hd + 2 * I)
+    joined = torch.empty(T, H * hd + I, dtype=bf, device=d)
+    gu, act = rnd(T, 2 * I), torch.empty(T, I, dtype=bf, device=d)
+    new, like = _us(lambda i: ops.geglu(joined[:, H * hd:], wide[:, (H + 2 * KV) * hd:], 0.5)), _us(lambda i: ops.swiglu(act, gu))
+    pair("activation_2048_tokens", new, T * I * 6.0, like, T * I * 6.0, "bytes", "Qwen3 swiglu", note="columns of wider rows")
+    return out
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="design_bench", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--design", default="givirax", choices=["givirax", "dugulorn", "lorulix", "rumurax", "sumevik"])
+    ap.add_argument("--design", default="givirax", choices=["givirax", "dugulorn", "lorulix", "rumurax", "sumevik", "legalix"])
     ap.add_argument("--sizes", default="small,large")
     ap.add_argument("--steps", type=int, default=48)
     ap.add_argument("--no-kernels", action="store_true", help="whole models only")
@@ -1063,23 +1264,27 @@ def main(argv=None) -> int:
         result.update(closest="Givirax", window=RX_WINDOW, pool=RX_POOL, chunk=RX_CHUNK, streams=2, experts=EXPERTS, top=TOP)
     if a.design == "sumevik":
         result.update(closest="Lorulix", chunk=SV_CHUNK, part=SV_PART, experts=EXPERTS, identity=SV_IDENTITY, top=TOP)
+    if a.design == "legalix":
+        result.update(closest="Sumevik", window=LG_WINDOW, keep_first=LG_KEEP, state=LG_STATE, state_vdim=LG_VDIM, state_groups=LG_GROUPS)
     for name in a.sizes.split(","):
         s = SIZES[name]
         entry = {"shape": s}
         if not a.no_models:
             t0 = time.time()
             design_config = {"givirax": givirax_config, "dugulorn": dugulorn_config, "lorulix": lorulix_config, "rumurax": rumurax_config,
-                             "sumevik": sumevik_config}[a.design]
+                             "sumevik": sumevik_config, "legalix": legalix_config}[a.design]
             entry[a.design] = model_points(design_config(s, 4160), 2048, 8, 4096, a.steps)
             if a.design in ("lorulix", "rumurax"):
                 entry["givirax"] = model_points(givirax_config(s, 4160), 2048, 8, 4096, a.steps)
             if a.design == "sumevik":
                 entry["lorulix"] = model_points(lorulix_config(s, 4160), 2048, 8, 4096, a.steps)
+            if a.design == "legalix":
+                entry["sumevik"] = model_points(sumevik_config(s, 4160), 2048, 8, 4096, a.steps)
             entry["qwen3"] = model_points(qwen3_config(s, 4160), 2048, 8, 4096, a.steps)
             entry["seconds"] = round(time.time() - t0, 1)
         if not a.no_kernels:
             entry["kernels"] = {"givirax": kernel_pairs, "dugulorn": dugulorn_kernel_pairs, "lorulix": lorulix_kernel_pairs,
-                                "rumurax": rumurax_kernel_pairs, "sumevik": sumevik_kernel_pairs}[a.design](s, pk)
+                                "rumurax": rumurax_kernel_pairs, "sumevik": sumevik_kernel_pairs, "legalix": legalix_kernel_pairs}[a.design](s, pk)
         result["sizes"][name] = entry
     print(json.dumps(result))
     return 0
