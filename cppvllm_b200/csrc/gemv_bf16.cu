@@ -776,6 +776,7 @@ constexpr size_t kRingSmem = 128 + static_cast<size_t>(kRingStages) * kRingStage
 
 struct RingParams {
     __nv_bfloat16* out;            // [M, N]
+    float* out32;                  // instead of out: the float sums, unrounded
     const __nv_bfloat16* x;        // [M, K]
     const __nv_bfloat16* W;        // [N, K]
     int* err;
@@ -891,7 +892,9 @@ gemv_ring_kernel(const RingParams p) {
                 float sum = 0.f;
 #pragma unroll
                 for (int w = 0; w < kRingConsumers; ++w) sum += red[w * 128 + row * 8 + m];
-                p.out[static_cast<int64_t>(m) * p.N + row0 + tile * 16 + row] = __float2bfloat16_rn(sum);
+                const int64_t at = static_cast<int64_t>(m) * p.N + row0 + tile * 16 + row;
+                if (p.out32 != nullptr) p.out32[at] = sum;
+                else p.out[at] = __float2bfloat16_rn(sum);
             }
         }
         asm volatile("bar.sync 1, %0;\n" ::"n"(kRingConsumers * 32) : "memory");      // `red` is free again
@@ -1013,7 +1016,8 @@ extern "C" int cvb_gemv_splitk_bf16(void* out, const void* x, const void* W, int
 
 // out[:M] = x[:M] W^T for up to 8 rows and a weight of any size, streamed through a ring of shared-memory stages by one
 // block per SM (see gemv_ring_kernel).  `dependent`: launch with the programmatic-dependent-launch attribute.
-extern "C" int cvb_gemv_ring_bf16(void* out, const void* x, const void* W, int M, int N, int K, int dependent, int* err,
+// `out_float`: out is float and receives the sums unrounded.
+extern "C" int cvb_gemv_ring_bf16(void* out, const void* x, const void* W, int M, int N, int K, int out_float, int dependent, int* err,
                                   cudaStream_t stream) {
     if (M == 0) return CVB_OK;
     if (M < 0 || M > kBatch || N <= 0 || K <= 0) return CVB_E_SIZE;
@@ -1034,7 +1038,8 @@ extern "C" int cvb_gemv_ring_bf16(void* out, const void* x, const void* W, int M
         set = true;
     }
     RingParams p{};
-    p.out = (__nv_bfloat16*)out; p.x = (const __nv_bfloat16*)x; p.W = (const __nv_bfloat16*)W; p.err = err;
+    p.out = out_float ? nullptr : (__nv_bfloat16*)out; p.out32 = out_float ? (float*)out : nullptr;
+    p.x = (const __nv_bfloat16*)x; p.W = (const __nv_bfloat16*)W; p.err = err;
     p.M = M; p.N = N; p.K = K;
     const int blocks = min(sms > 0 ? sms : 148, N);
     launch_kernel_dependent(gemv_ring_kernel, dim3(blocks), dim3(kRingThreads), kRingSmem, stream, dependent != 0, p);

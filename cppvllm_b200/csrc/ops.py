@@ -2041,17 +2041,17 @@ def gemv_ring_supported(x_dtype: torch.dtype, weight: torch.Tensor, rows: int) -
 
 def gemv_ring_bf16(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, rows: int, dependent: bool = False) -> torch.Tensor:
     """out[:rows] = x[:rows] @ weight^T for up to 8 rows: one block per SM streams its share of the weight's rows through a
-    ring of shared-memory stages filled by bulk copies."""
+    ring of shared-memory stages filled by bulk copies.  A float32 `out` receives the sums unrounded."""
     lib = _gemv_lib()
     _cuda(out, x, weight)
     _contig(out, x, weight)
     N, K = weight.shape
-    if x.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or x.shape[1] != K:
-        raise KernelError("gemv_ring_bf16: x [M, K], weight [N, K] and out must be bf16")
+    if x.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16 or out.dtype not in (torch.bfloat16, torch.float32) or x.shape[1] != K:
+        raise KernelError("gemv_ring_bf16: x [M, K] and weight [N, K] must be bf16, out bf16 or float32")
     if out.shape[1] != N or out.shape[0] < rows or x.shape[0] < rows:
         raise KernelError("gemv_ring_bf16: out must be [M, N]")
-    _check(lib.cvb_gemv_ring_bf16(_ptr(out), _ptr(x), _ptr(weight), c_int(rows), c_int(N), c_int(K), c_int(1 if dependent else 0),
-                                  _ptr(error_flag(x.device)), _stream()), "gemv_ring_bf16")
+    _check(lib.cvb_gemv_ring_bf16(_ptr(out), _ptr(x), _ptr(weight), c_int(rows), c_int(N), c_int(K), c_int(1 if out.dtype == torch.float32 else 0),
+                                  c_int(1 if dependent else 0), _ptr(error_flag(x.device)), _stream()), "gemv_ring_bf16")
     return out
 
 

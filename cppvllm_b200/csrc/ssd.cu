@@ -572,23 +572,27 @@ ssd_step_kernel(float* __restrict__ y, const T* __restrict__ packed, const float
 
 constexpr int kNormQuads = 8;                            // four-element pieces a thread keeps in registers
 
-// A block per (token, part); rows in pieces of four that start on 16 bytes (8 bytes of bf16 rows) stay in registers.
+// A block (up to 512 elements: a warp, four to a block) per (token, part); rows in pieces of four that start on 16 bytes (8 bytes of bf16
+// rows) stay in registers.
 template <typename T, int THREADS>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(THREADS < 128 ? 128 : THREADS)
 ssd_norm_vec_kernel(T* __restrict__ out, int out_stride, const float* __restrict__ y, const T* __restrict__ z, int z_stride, const float* __restrict__ w,
-                    int parts, int n, float eps, float scale) {
+                    int64_t rows, int parts, int n, float eps, float scale) {
     pdl_trigger();
     pdl_wait();
     __shared__ float scratch[32];
-    const int64_t t = blockIdx.x;
-    const int c0 = blockIdx.y * n;
+    constexpr int kPer = THREADS < 128 ? 128 / THREADS : 1, kQuads = THREADS < 128 ? 4 : kNormQuads;
+    const int64_t row = static_cast<int64_t>(blockIdx.x) * kPer + threadIdx.x / THREADS;
+    if (row >= rows) return;
+    const int64_t t = row / parts;
+    const int c0 = static_cast<int>(row - t * parts) * n, lane = threadIdx.x % THREADS;
     const float* yr = y + t * parts * n + c0;
     const T* zr = z + t * z_stride + c0;
-    float4 v[kNormQuads];
+    float4 v[kQuads];
     float ss = 0.f;
 #pragma unroll
-    for (int k = 0; k < kNormQuads; ++k) {
-        const int j = (threadIdx.x + k * THREADS) * 4;
+    for (int k = 0; k < kQuads; ++k) {
+        const int j = (lane + k * THREADS) * 4;
         if (j < n) {
             v[k] = *reinterpret_cast<const float4*>(yr + j);
             float g[4];
@@ -608,8 +612,8 @@ ssd_norm_vec_kernel(T* __restrict__ out, int out_stride, const float* __restrict
     const float inv = scale / sqrtf(ss / static_cast<float>(n) + eps);
     T* dst = out + t * out_stride + c0;
 #pragma unroll
-    for (int k = 0; k < kNormQuads; ++k) {
-        const int j = (threadIdx.x + k * THREADS) * 4;
+    for (int k = 0; k < kQuads; ++k) {
+        const int j = (lane + k * THREADS) * 4;
         if (j < n) {
             const float4 ww = *reinterpret_cast<const float4*>(w + c0 + j);
             const float r[4] = {v[k].x * inv * ww.x, v[k].y * inv * ww.y, v[k].z * inv * ww.z, v[k].w * inv * ww.w};
@@ -782,15 +786,17 @@ extern "C" int cvb_ssd_norm(void* out, int out_stride, const float* y, const voi
                             float eps, float scale, int dtype, cudaStream_t stream) {
     if (T == 0) return CVB_OK;
     if (T < 0 || parts <= 0 || parts > 65535 || n <= 0) return CVB_E_SIZE;
+    const int64_t rows = static_cast<int64_t>(T) * parts;
+    if (rows > 2147483647LL) return CVB_E_SIZE;
     if (out_stride < parts * n || z_stride < parts * n) return CVB_E_SHAPE;
     const uintptr_t ab = dtype == CVB_DTYPE_BF16 ? 7 : 15;
     const bool vec = n % 4 == 0 && n <= 256 * kNormQuads * 4 && out_stride % 4 == 0 && z_stride % 4 == 0 && ssd_al16(y) && ssd_al16(w)
                      && ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & ab) == 0;
-#define CALL_N(TY, TH) launch_kernel(ssd_norm_vec_kernel<TY, TH>, dim3(T, parts), dim3(TH), 0, stream, (TY*)out, out_stride, y, (const TY*)z, z_stride, w, \
-                                     parts, n, eps, scale)
+#define CALL_N(TY, TH) launch_kernel(ssd_norm_vec_kernel<TY, TH>, dim3(static_cast<unsigned>(TH < 128 ? (rows + 3) / 4 : rows)), dim3(TH < 128 ? 128 : TH), 0, \
+                                     stream, (TY*)out, out_stride, y, (const TY*)z, z_stride, w, rows, parts, n, eps, scale)
 #define CALL(TY)                                                                                                              \
-    if (vec && n <= 256) { CALL_N(TY, 32); }                                                                                  \
-    else if (vec && n <= 2048) { CALL_N(TY, 128); }                                                                           \
+    if (vec && n <= 512) { CALL_N(TY, 32); }                                                                                  \
+    else if (vec && n <= 4096) { CALL_N(TY, 128); }                                                                           \
     else if (vec) { CALL_N(TY, 256); }                                                                                        \
     else launch_kernel(ssd_norm_kernel<TY>, dim3(T, parts), dim3(kSsdThreads), 0, stream, (TY*)out, out_stride, y, (const TY*)z, z_stride, w, \
                        parts, n, eps, scale)

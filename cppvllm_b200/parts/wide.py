@@ -290,5 +290,8 @@ class ConcatInput(StreamInput):
             raise ValueError("the embedding output was not kept apart from the residual stream")
         T, D = h.shape
         both = ops.stream_concat(self.rt.workspace.rows("stream_both", T, 2 * D, self.rt.dtype), h, _as_tuple(pending), embedded)
-        ops.linear(both, self.weight, out=h, out_dtype=torch.float32)
+        if not self.rt.plain_kernels and ops.gemv_ring_supported(both.dtype, self.weight, T):
+            ops.gemv_ring_bf16(h, both, self.weight, T)        # a few decoded tokens: the weight is a stream
+        else:
+            ops.linear(both, self.weight, out=h, out_dtype=torch.float32)
         return h, None
