@@ -9,8 +9,8 @@
 // the kernel for decoded tokens write its input while other blocks still read the others; inputs before position 0 are zeros by
 // their position.
 //
-//   ssd_prep    : x, B, C, dt and a of every token.  By vectors where the channels allow it: a thread owns eight channels over eight
-//                 tokens and slides a window of K rows along.
+//   ssd_prep    : x, B, C, dt and a of every token.  By vectors where the channels allow it: a thread owns eight channels over four
+//                 tokens and asks for all their rows together.
 //   ssd_ring    : the last K - 1 raw inputs of every portion into the ring (behind ssd_prep, which reads the older ones).
 //   ssd_scan    : portions in chunks of 64 tokens on the tensor cores (bf16 x, B, C; `mma.sync.m16n8k16`, float accumulation).  With
 //                 l the running sum of a inside a chunk (never positive differences, so nothing overflows) and S0 the state in front:
@@ -39,10 +39,15 @@ struct SsdShape {
 };
 
 __device__ __forceinline__ float ssd_silu(float z) { return z / (1.f + expf(-z)); }
+// with bf16 activations through the hardware's exponential and division
+template <typename T> __device__ __forceinline__ float ssd_silu_of(float z) {
+    if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
+    else return ssd_silu(z);
+}
 __device__ __forceinline__ float ssd_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 constexpr int kSsdThreads = 128;
-constexpr int kPrepRun = 8;                              // tokens per thread of the vector form
+constexpr int kPrepRun = 4;                              // tokens per thread of the vector form
 
 // The convolution of channel c for the token at packed row t: `local` tokens of its portion lie before it, it sits at position pos.
 template <typename T>
@@ -90,8 +95,25 @@ ssd_prep_kernel(U* __restrict__ u, float* __restrict__ dt, float* __restrict__ l
     const int local = static_cast<int>(t) - cu_seqlens[s], pos = positions[t];
     const float* ring = state + static_cast<int64_t>(slot) * sh.state_floats + static_cast<int64_t>(sh.H) * sh.N * sh.P;
     for (int c = blockIdx.y * kSsdThreads + threadIdx.x; c < sh.C; c += gridDim.y * kSsdThreads)
-        u[t * sh.C + c] = from_float<U>(ssd_silu(ssd_conv_of(packed, conv_w, conv_b, ring, sh, t, local, pos, c)));
+        u[t * sh.C + c] = from_float<U>(ssd_silu_of<U>(ssd_conv_of(packed, conv_w, conv_b, ring, sh, t, local, pos, c)));
 }
+
+// eight elements of a row as they lie in memory
+template <typename T> struct Row8;
+template <> struct Row8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = *reinterpret_cast<const float4*>(p); b = *reinterpret_cast<const float4*>(p + 4); }
+    __device__ __forceinline__ void get(float (&f)[8]) const { f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w; }
+};
+template <> struct Row8<__nv_bfloat16> {
+    uint4 r;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { r = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void get(float (&f)[8]) const {
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&r);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { const float2 v = __bfloat1622float2(h[i]); f[2 * i] = v.x; f[2 * i + 1] = v.y; }
+    }
+};
 
 template <typename T, typename U, int K>
 __global__ void __launch_bounds__(kSsdThreads)
@@ -114,39 +136,51 @@ ssd_prep_vec_kernel(U* __restrict__ u, float* __restrict__ dt, float* __restrict
     }
     const int c = (blockIdx.y * kSsdThreads + threadIdx.x) * 8;
     if (c >= sh.C) return;
-    float w[K][8], b[8], x[K][8];
+    const T* base = packed + sh.u_off + c;
+    Row8<T> x[K - 1 + kPrepRun];                          // rows t0 - K + 1 .. t1 - 1, asked for together
+#pragma unroll
+    for (int i = 0; i < K - 1 + kPrepRun; ++i) x[i].load(base + static_cast<int64_t>(min(max(t0 - K + 1 + i, 0), t1 - 1)) * sh.stride);
+    int seq[kPrepRun], first[kPrepRun];
+#pragma unroll
+    for (int i = 0; i < kPrepRun; ++i) seq[i] = seq_of_token[min(t0 + i, t1 - 1)];
+#pragma unroll
+    for (int i = 0; i < kPrepRun; ++i) first[i] = cu_seqlens[seq[i]];
+    float w[K][8], b[8];
     load8(b, conv_b + c);
 #pragma unroll
     for (int m = 0; m < K; ++m) load8(w[m], conv_w + static_cast<int64_t>(m) * sh.C + c);
-    const T* base = packed + sh.u_off + c;
 #pragma unroll
-    for (int m = 1; m < K; ++m) load8(x[m], base + static_cast<int64_t>(max(t0 - K + m, 0)) * sh.stride);   // rows t0 - K + 1 .. t0 - 1
-    for (int t = t0; t < t1; ++t) {
-#pragma unroll
-        for (int m = 0; m + 1 < K; ++m)
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[m][e] = x[m + 1][e];
-        load8(x[K - 1], base + static_cast<int64_t>(t) * sh.stride);
-        const int s = seq_of_token[t], local = t - cu_seqlens[s];
+    for (int i = 0; i < kPrepRun; ++i) {
+        const int t = t0 + i, local = t - first[i];
+        if (t >= t1) break;
         float y[8];
         if (local >= K - 1) {
 #pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                float acc = b[e];
+            for (int e = 0; e < 8; ++e) y[e] = b[e];
 #pragma unroll
-                for (int m = 0; m < K; ++m) acc = fmaf(w[m][e], x[m][e], acc);
-                y[e] = ssd_silu(acc);
+            for (int m = 0; m < K; ++m) {
+                float v[8];
+                x[i + m].get(v);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) y[e] = fmaf(w[m][e], v[e], y[e]);
             }
         } else {                                          // the window reaches back before the portion
-            const int slot = state_slots[s];
+            const int slot = state_slots[seq[i]];
             if (slot < 0 || slot >= sh.num_slots) {
                 atomicExch(err, 2);
                 continue;
             }
             const float* ring = state + static_cast<int64_t>(slot) * sh.state_floats + static_cast<int64_t>(sh.H) * sh.N * sh.P;
+#pragma unroll 1
+            for (int e = 0; e < 8; ++e) {
+                const float v = ssd_conv_of(packed, conv_w, conv_b, ring, sh, t, local, positions[t], c + e);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[e] = ssd_silu(ssd_conv_of(packed, conv_w, conv_b, ring, sh, t, local, positions[t], c + e));
+                for (int k = 0; k < 8; ++k)
+                    if (k == e) y[k] = v;
+            }
         }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = ssd_silu_of<U>(y[e]);
         store8(u + static_cast<int64_t>(t) * sh.C + c, y);
     }
 }
@@ -174,6 +208,7 @@ ssd_ring_kernel(float* __restrict__ state, const T* __restrict__ packed, const i
 
 constexpr int kChunk = 64;                               // tokens per chunk
 constexpr int kCols = 64;                                // columns of S per block
+constexpr int kOutThreads = 256;                         // pass 3: two warps per 16 tokens, 32 columns each
 constexpr int kLdX = kCols + 8;                          // padded row of a tile of columns, in elements
 
 struct SsdChunk { int seq, k, n_chunks, buf, begin, n; };
@@ -225,7 +260,7 @@ __device__ __forceinline__ void chunk_sums(float* l, float* d, const float* __re
 // `width` columns (a multiple of 8) of a chunk's rows into shared rows of ld elements; rows past the chunk are zeros.
 __device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int ld, const __nv_bfloat16* __restrict__ src, int64_t stride, int n, int width) {
     const int per = width >> 3;
-    for (int i = threadIdx.x; i < kChunk * per; i += kSsdThreads) {
+    for (int i = threadIdx.x; i < kChunk * per; i += blockDim.x) {
         const int r = i / per, c = (i - r * per) * 8;
         cp_async16(dst + r * ld + c, r < n ? src + r * stride + c : src, r < n);
     }
@@ -234,7 +269,7 @@ __device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int ld, const __n
 // x times e^(l_last - l_s) dt_s, in two bf16 addends
 __device__ __forceinline__ void weigh_rows(__nv_bfloat16* hi, __nv_bfloat16* lo, const __nv_bfloat16* x, const float* l, const float* d, int width) {
     const float last = l[kChunk - 1];
-    for (int i = threadIdx.x; i < kChunk * (width >> 1); i += kSsdThreads) {
+    for (int i = threadIdx.x; i < kChunk * (width >> 1); i += blockDim.x) {
         const int r = i / (width >> 1), c = (i - r * (width >> 1)) * 2;
         const float w = expf(last - l[r]) * d[r];
         float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x + r * kLdX + c));
@@ -246,11 +281,11 @@ __device__ __forceinline__ void weigh_rows(__nv_bfloat16* hi, __nv_bfloat16* lo,
     }
 }
 
-// What the chunk adds to S: sum_s B_s xw_s^T; a warp takes every fourth slab of 16 rows of S.  put(row, column, two values).
+// What the chunk adds to S: sum_s B_s xw_s^T; the block's warps take slabs of 16 rows of S in turn.  put(row, column, two values).
 template <typename F>
 __device__ __forceinline__ void chunk_state(const __nv_bfloat16* sB, int ldb, const __nv_bfloat16* hi, const __nv_bfloat16* lo, int N, int width, F put) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int m0 = warp * 16; m0 < N; m0 += 64) {
+    for (int m0 = warp * 16; m0 < N; m0 += static_cast<int>(blockDim.x >> 5) * 16) {
         float acc[kCols / 8][4];
 #pragma unroll
         for (int i = 0; i < kCols / 8; ++i) { acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f; }
@@ -350,8 +385,8 @@ ssd_carry_kernel(float* __restrict__ ends, const float* __restrict__ decays, con
     }
 }
 
-// Pass 3.  A warp owns 16 tokens of the chunk.
-__global__ void __launch_bounds__(kSsdThreads)
+// Pass 3.  A warp owns 16 tokens of the chunk and half the block's columns; both warps of a pair make the 16 tokens' C . B.
+__global__ void __launch_bounds__(kOutThreads)
 ssd_out_kernel(float* __restrict__ y, const __nv_bfloat16* __restrict__ u, const float* __restrict__ dt, const float* __restrict__ la,
                const float* __restrict__ D, const float* __restrict__ ends, float* __restrict__ state, const int* __restrict__ cu_seqlens,
                const int* __restrict__ state_slots, int S, SsdShape sh, int* __restrict__ err) {
@@ -368,7 +403,7 @@ ssd_out_kernel(float* __restrict__ y, const __nv_bfloat16* __restrict__ u, const
     __shared__ float l[kChunk], d[kChunk];
     const int h = blockIdx.y, p0 = blockIdx.z * kCols, width = min(kCols, sh.P - p0);
     const int g = h / (sh.H / sh.G), N = sh.N, ldb = N + 8;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3, col0 = (threadIdx.x >> 7) * (kCols / 2);
     const int s_rows = N > kChunk ? N : kChunk;           // the room of S0 also takes the chunk's weighted rows
     __nv_bfloat16* sC = reinterpret_cast<__nv_bfloat16*>(smem_raw);
     __nv_bfloat16* sB = sC + kChunk * ldb;
@@ -384,7 +419,7 @@ ssd_out_kernel(float* __restrict__ y, const __nv_bfloat16* __restrict__ u, const
     float* st = state + static_cast<int64_t>(slot) * sh.state_floats + h * mat + p0;
     const float* from = ck.n_chunks > 1 ? ends + (static_cast<int64_t>(ck.buf + ck.k) * sh.H + h) * mat + p0 : st;
     const int quads = width >> 2;
-    for (int i = threadIdx.x; i < N * quads; i += kSsdThreads) {
+    for (int i = threadIdx.x; i < N * quads; i += kOutThreads) {
         const int r = i / quads, c = (i - r * quads) * 4;
         const float4 v = *reinterpret_cast<const float4*>(from + static_cast<int64_t>(r) * sh.P + c);
         const __nv_bfloat162 h0 = __floats2bfloat162_rn(v.x, v.y), h1 = __floats2bfloat162_rn(v.z, v.w);
@@ -400,20 +435,20 @@ ssd_out_kernel(float* __restrict__ y, const __nv_bfloat16* __restrict__ u, const
     __syncthreads();
 
     const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;  // the two tokens whose rows this thread holds
-    float o[kCols / 8][4];
+    float o[kCols / 16][4];
 #pragma unroll
-    for (int i = 0; i < kCols / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    for (int i = 0; i < kCols / 16; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m[kChunk / 8][4];
 #pragma unroll
     for (int i = 0; i < kChunk / 8; ++i) { m[i][0] = m[i][1] = m[i][2] = m[i][3] = 0.f; }
-    if (warp * 16 < ck.n) {
+    if (warp * 16 < ck.n && col0 < width) {
         for (int ks = 0; ks < N / 16; ++ks) {
             uint32_t a[4];
             ldm_x4(a, sC + (warp * 16 + (lane & 15)) * ldb + ks * 16 + (lane >> 4) * 8);
 #pragma unroll
-            for (int dp = 0; dp < kCols / 16; ++dp) {     // S0^T C
-                if (dp * 16 >= width) break;
-                const int at = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdX + dp * 16 + ((lane >> 4) & 1) * 8;
+            for (int dp = 0; dp < kCols / 32; ++dp) {     // S0^T C
+                if (col0 + dp * 16 >= width) break;
+                const int at = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdX + col0 + dp * 16 + ((lane >> 4) & 1) * 8;
                 uint32_t b[4];
                 ldm_x4_trans(b, hi + at);
                 mma_16816(o[dp * 2], a, b[0], b[1]);
@@ -433,7 +468,7 @@ ssd_out_kernel(float* __restrict__ y, const __nv_bfloat16* __restrict__ u, const
         }
         const float l0 = l[r0], l1 = l[r1], e0 = expf(l0), e1 = expf(l1);
 #pragma unroll
-        for (int i = 0; i < kCols / 8; ++i) { o[i][0] *= e0; o[i][1] *= e0; o[i][2] *= e1; o[i][3] *= e1; }
+        for (int i = 0; i < kCols / 16; ++i) { o[i][0] *= e0; o[i][1] *= e0; o[i][2] *= e1; o[i][3] *= e1; }
 #pragma unroll
         for (int nt = 0; nt < kChunk / 8; ++nt) {
             if (nt > warp * 2 + 1) break;
@@ -456,10 +491,10 @@ ssd_out_kernel(float* __restrict__ y, const __nv_bfloat16* __restrict__ u, const
                 al[q] = pack2(v0 - f.x, v1 - f.y);
             }
 #pragma unroll
-            for (int dp = 0; dp < kCols / 16; ++dp) {
-                if (dp * 16 >= width) break;
+            for (int dp = 0; dp < kCols / 32; ++dp) {
+                if (col0 + dp * 16 >= width) break;
                 uint32_t b[4];
-                ldm_x4_trans(b, sX + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdX + dp * 16 + ((lane >> 4) & 1) * 8);
+                ldm_x4_trans(b, sX + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdX + col0 + dp * 16 + ((lane >> 4) & 1) * 8);
                 mma_16816(o[dp * 2], ah, b[0], b[1]);
                 mma_16816(o[dp * 2 + 1], ah, b[2], b[3]);
                 mma_16816(o[dp * 2], al, b[0], b[1]);
@@ -473,9 +508,9 @@ ssd_out_kernel(float* __restrict__ y, const __nv_bfloat16* __restrict__ u, const
             if (r >= ck.n) continue;
             float* dst = y + (static_cast<int64_t>(ck.begin + r) * sh.H + h) * sh.P + p0;
 #pragma unroll
-            for (int i = 0; i < kCols / 8; ++i) {
-                if (i * 8 >= width) break;
-                const int c = i * 8 + ((lane & 3) << 1);
+            for (int i = 0; i < kCols / 16; ++i) {
+                if (col0 + i * 8 >= width) break;
+                const int c = col0 + i * 8 + ((lane & 3) << 1);
                 const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + r * kLdX + c));
                 *reinterpret_cast<float2*>(dst + c) = make_float2(fmaf(skip, x.x, o[i][half * 2]), fmaf(skip, x.y, o[i][half * 2 + 1]));
             }
@@ -527,6 +562,18 @@ ssd_step_kernel(float* __restrict__ y, const T* __restrict__ packed, const float
     float* row = state + static_cast<int64_t>(slot) * sh.state_floats;
     float* ring = row + static_cast<int64_t>(sh.H) * N * P;
     const bool first_of_group = h % per == 0;             // writes the group's B and C into the ring
+    float* st = row + static_cast<int64_t>(h) * N * P;
+    const int rg = narrow ? tid / nvec : 0;
+    // the thread's first rows of S are on their way before the convolutions
+    constexpr int kAhead = V == 4 ? 8 : 1;
+    float4 ahead[kAhead];
+    if constexpr (V == 4) {
+        if (narrow && rg < R) {
+#pragma unroll
+            for (int k = 0; k < kAhead; ++k)
+                if (rg + k * R < N) ahead[k] = *reinterpret_cast<const float4*>(st + static_cast<int64_t>(rg + k * R) * P + (tid - rg * nvec) * 4);
+        }
+    }
     for (int c = tid; c < P + 2 * N; c += kStepThreads) {
         const int ch = c < P ? h * P + c : (c < P + N ? HP + g * N + c - P : HP + (sh.G + g) * N + c - P - N);
         smf[c] = ssd_silu(ssd_conv_of(packed, conv_w, conv_b, ring, sh, t, 0, pos, ch));
@@ -535,15 +582,27 @@ ssd_step_kernel(float* __restrict__ y, const T* __restrict__ packed, const float
     }
     const float dt = ssd_dt(packed, dt_bias, sh, t, h), a = expf(neg_a[h] * dt), skip = D[h];
     __syncthreads();
-    float* st = row + static_cast<int64_t>(h) * N * P;
-    const int rg = narrow ? tid / nvec : 0;
     for (int cv = narrow ? tid - rg * nvec : tid; cv < nvec; cv += (narrow ? nvec : kStepThreads)) {
         if (rg >= R) break;
         float v[V], o[V];
 #pragma unroll
         for (int j = 0; j < V; ++j) { v[j] = dt * xs[cv * V + j]; o[j] = 0.f; }
+        int i = rg;
+        if constexpr (V == 4) {
+            if (narrow) {
+#pragma unroll
+                for (int k = 0; k < kAhead; ++k, i += R) {
+                    if (i >= N) break;
+                    const float b = bs[i], q = cs[i];
+                    float4 x = ahead[k];
+                    x.x = fmaf(a, x.x, b * v[0]); x.y = fmaf(a, x.y, b * v[1]); x.z = fmaf(a, x.z, b * v[2]); x.w = fmaf(a, x.w, b * v[3]);
+                    o[0] = fmaf(q, x.x, o[0]); o[1] = fmaf(q, x.y, o[1]); o[2] = fmaf(q, x.z, o[2]); o[3] = fmaf(q, x.w, o[3]);
+                    *reinterpret_cast<float4*>(st + static_cast<int64_t>(i) * P + cv * V) = x;
+                }
+            }
+        }
 #pragma unroll 8
-        for (int i = rg; i < N; i += R) {
+        for (; i < N; i += R) {
             float* p = st + static_cast<int64_t>(i) * P + cv * V;
             const float k = bs[i], q = cs[i];
             if constexpr (V == 4) {
@@ -604,7 +663,7 @@ ssd_norm_vec_kernel(T* __restrict__ out, int out_stride, const float* __restrict
                 const float4 a = *reinterpret_cast<const float4*>(zr + j);
                 g[0] = a.x; g[1] = a.y; g[2] = a.z; g[3] = a.w;
             }
-            v[k].x *= ssd_silu(g[0]); v[k].y *= ssd_silu(g[1]); v[k].z *= ssd_silu(g[2]); v[k].w *= ssd_silu(g[3]);
+            v[k].x *= ssd_silu_of<T>(g[0]); v[k].y *= ssd_silu_of<T>(g[1]); v[k].z *= ssd_silu_of<T>(g[2]); v[k].w *= ssd_silu_of<T>(g[3]);
             ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
         }
     }
@@ -642,13 +701,13 @@ ssd_norm_kernel(T* __restrict__ out, int out_stride, const float* __restrict__ y
     const T* zr = z + t * z_stride + c0;
     float ss = 0.f;
     for (int j = threadIdx.x; j < n; j += kSsdThreads) {
-        const float v = yr[j] * ssd_silu(to_float(zr[j]));
+        const float v = yr[j] * ssd_silu_of<T>(to_float(zr[j]));
         ss = fmaf(v, v, ss);
     }
     ss = block_sum(ss, scratch);
     const float inv = scale / sqrtf(ss / static_cast<float>(n) + eps);
     for (int j = threadIdx.x; j < n; j += kSsdThreads)
-        out[t * out_stride + c0 + j] = from_float<T>(yr[j] * ssd_silu(to_float(zr[j])) * inv * w[c0 + j]);
+        out[t * out_stride + c0 + j] = from_float<T>(yr[j] * ssd_silu_of<T>(to_float(zr[j])) * inv * w[c0 + j]);
 }
 
 static bool ssd_al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
@@ -755,7 +814,7 @@ extern "C" int cvb_ssd_chunks(float* y, const void* u, const float* dt, const fl
         launch_kernel(ssd_carry_kernel, dim3(S, H, static_cast<unsigned>(zs < 64 ? zs : 64)), dim3(256), 0, stream, ends, decays, state, cu_seqlens,
                       state_slots, S, sh, err_flag);
     }
-    launch_kernel(ssd_out_kernel, dim3(chunks, H, slices), dim3(kSsdThreads), smem3, stream, y, (const __nv_bfloat16*)u, dt, la, D, ends, state,
+    launch_kernel(ssd_out_kernel, dim3(chunks, H, slices), dim3(kOutThreads), smem3, stream, y, (const __nv_bfloat16*)u, dt, la, D, ends, state,
                   cu_seqlens, state_slots, S, sh, err_flag);
     return launch_status();
 }

@@ -130,8 +130,14 @@ class LatentAttention(Mixer):
         # the batched products write straight to their places inside wider rows: q_abs in front of the turned part, and (without a
         # gate) the heads side by side
         q_att = ws.rows("lat_qatt", T, H * (R + dr), dt)
-        torch.bmm(q.view(T, H, dn + dr)[:, :, :dn].transpose(0, 1), self.w_uk, out=q_att.view(T, H, R + dr)[:, :, :R].transpose(0, 1))
-        ops.latent_q_turn(q_att, q, H, dn, R, dr, self.rot, pos.cos, pos.sin, ctx.positions)
+        q_nope = q.view(T, H, dn + dr)[:, :, :dn].transpose(0, 1)
+        if self.rt.plain_kernels:
+            q_abs = ws.rows("lat_qabs", T, H * R, dt).view(H, T, R)
+            torch.bmm(q_nope, self.w_uk, out=q_abs)
+            ops.latent_q_assemble(q_att, q_abs, q, H, dn, R, dr, self.rot, pos.cos, pos.sin, ctx.positions)
+        else:
+            torch.bmm(q_nope, self.w_uk, out=q_att.view(T, H, R + dr)[:, :, :R].transpose(0, 1))
+            ops.latent_q_turn(q_att, q, H, dn, R, dr, self.rot, pos.cos, pos.sin, ctx.positions)
         o_lat = ws.rows("lat_o", T, H * R, dt)
         self.attend(o_lat, q_att, ctx, cache, g, scale)
         lat_heads = o_lat.view(T, H, R).transpose(0, 1)
