@@ -80,7 +80,7 @@ def test_gated_activation_on_columns_of_wider_rows(dtype, T, I, lead):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,G,dk,dv,rot,normed", [(4, 2, 64, 64, 32, False), (3, 1, 32, 16, 32, True), (2, 2, 18, 7, 4, False), (2, 1, 48, 48, 12, False),
-                                                  (4, 4, 128, 48, 32, False)])
+                                                  (6, 3, 128, 80, 64, False)])
 def test_projection_epilogue_with_pairs_across_the_rotation(dtype, H, G, dk, dv, rot, normed):
     """Pairs (i, i + rot / 2): by 16 bytes where half the rotation is whole chunks, element by element elsewhere; with and without norms."""
     from cppvllm_b200.csrc import ops
@@ -112,7 +112,7 @@ def test_projection_epilogue_with_pairs_across_the_rotation(dtype, H, G, dk, dv,
 
 
 @pytest.mark.parametrize("dtype,kernel", [("float32", "general"), ("bfloat16", "general"), ("bfloat16", "portion"), ("bfloat16", "decode"), ("bfloat16", "split")])
-@pytest.mark.parametrize("H,G,dk,dv,window,keep,page", [(4, 2, 64, 64, 24, 5, 16), (6, 2, 32, 96, 70, 20, 32), (2, 1, 128, 48, 7, 100, 16), (16, 1, 16, 16, 1, 1, 32),
+@pytest.mark.parametrize("H,G,dk,dv,window,keep,page", [(4, 2, 64, 64, 24, 5, 16), (6, 2, 32, 96, 70, 20, 32), (2, 1, 128, 80, 7, 100, 16), (16, 1, 16, 16, 1, 1, 32),
                                                         (4, 2, 64, 32, 64, 64, 64), (2, 2, 32, 32, 33, 0, 16)])
 def test_attention_behind_a_window_with_kept_first_tokens(dtype, kernel, H, G, dk, dv, window, keep, page):
     """Requests of unequal length whose pages behind the window (but for those of the kept tokens) have been given back: their entries in
